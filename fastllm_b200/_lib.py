@@ -11,7 +11,8 @@ import os
 HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(HERE, "libfastllm_b200.so")
 
-FL_ARCH = {"llama": 0, "mistral": 1, "qwen2": 2, "mixtral": 3, "bert": 4, "nifunex": 5, "rofetar": 6, "tozarax": 7, "medulorn": 8}
+FL_ARCH = {"llama": 0, "mistral": 1, "qwen2": 2, "mixtral": 3, "bert": 4, "nifunex": 5, "rofetar": 6, "tozarax": 7, "medulorn": 8,
+           "latodra": 9}
 FL_MIXER = {"gla": 0, "latent_attention": 1, "attention": 2, "mamba2": 3, "delta": 4, "lightning": 5}
 FL_ACT = {"swish_clamp": 0, "gelu_tanh": 1, "relu2": 2, "relu": 3}
 FL_ROT_SCALE = {"yarn": 0, "bands": 1}
@@ -41,7 +42,8 @@ class FlLayerDesc(C.Structure):
                 ("no_qk_norm", C.c_int32), ("beside", C.c_int32), ("router", C.c_int32), ("route_groups", C.c_int32),
                 ("route_keep", C.c_int32), ("qkv_bias", C.c_int32), ("qk_norm_whole", C.c_int32), ("mask_chunk", C.c_int32),
                 ("keep_first", C.c_int32), ("rot_scaling", C.c_int32), ("out_scale", C.c_float), ("pair_sum", C.c_int32),
-                ("router_bias", C.c_int32), ("shared_plain", C.c_int32), ("reserved", C.c_int32 * 2)]
+                ("router_bias", C.c_int32), ("shared_plain", C.c_int32), ("q_rank", C.c_int32), ("out_gate", C.c_int32),
+                ("reserved", C.c_int32 * 2)]
 
 
 class FlStackConfig(C.Structure):
@@ -49,7 +51,9 @@ class FlStackConfig(C.Structure):
                 ("compute_dtype", C.c_int32), ("norm_plain", C.c_int32), ("no_pre_norm", C.c_int32), ("no_post_norm", C.c_int32),
                 ("max_positions", C.c_int32), ("canon_taps", C.c_int32), ("gated_residual", C.c_int32), ("depth_avg", C.c_int32),
                 ("post_sum_norm", C.c_int32), ("residual_alpha", C.c_float), ("norm_scalar", C.c_int32), ("embed_scale", C.c_float),
-                ("logit_softcap", C.c_float), ("token_shift", C.c_int32), ("reserved", C.c_int32 * 3)]
+                ("logit_softcap", C.c_float), ("token_shift", C.c_int32), ("embed_norm", C.c_int32), ("layer_scale", C.c_int32),
+                ("tied_head", C.c_int32), ("loop_start", C.c_int32), ("loop_stop", C.c_int32), ("loop_times", C.c_int32),
+                ("loop_reinject", C.c_int32), ("loop_step", C.c_int32), ("reserved", C.c_int32 * 3)]
 
 
 class FastllmError(RuntimeError):

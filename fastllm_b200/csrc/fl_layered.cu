@@ -1,4 +1,4 @@
-// Layered decoders (FL_ARCH_NIFUNEX, FL_ARCH_ROFETAR, FL_ARCH_TOZARAX, FL_ARCH_MEDULORN): weight layout + ingest, pooled cache (pages of latents or keys | values +
+// Layered decoders (FL_ARCH_NIFUNEX, FL_ARCH_ROFETAR, FL_ARCH_TOZARAX, FL_ARCH_MEDULORN, FL_ARCH_LATODRA): weight layout + ingest, pooled cache (pages of latents or keys | values +
 // recurrent-state slots), and the step function for mixed batches (portions of prompts beside single decoded tokens).
 #include <cmath>
 #include <map>
@@ -62,6 +62,7 @@ static void check_mixer(const LayeredModel& m, int i, const fl_layer_desc& d, bo
                  at + "latent attention: kv_rank <= 512 and rot_dim <= 128");
         FL_CHECK(d.rot_dims >= 0 && d.rot_dims <= d.rot_dim && d.rot_dims % 2 == 0, FL_ERR_INVALID, at + "rotated channels must be even and <= rot_dim");
         FL_CHECK(d.window >= 0, FL_ERR_INVALID, at + "negative window");
+        FL_CHECK(d.q_rank >= 0 && d.sink >= 0 && d.sink <= 2, FL_ERR_INVALID, at + "bad query latent size / sink kind");
         if (d.kv_from >= 0) {
             FL_CHECK(d.kv_from < i, FL_ERR_INVALID, at + "kv_from must name an earlier layer");
             const fl_layer_desc& s = m.layers[d.kv_from].d;
@@ -133,7 +134,8 @@ static void check_layer(const LayeredModel& m, int i, const fl_layer_desc& d) {
 
 void layered_build(LayeredModel& m, const fl_layer_desc* descs) {
     const fl_stack_config& c = m.cfg;
-    FL_CHECK(c.arch == FL_ARCH_NIFUNEX || c.arch == FL_ARCH_ROFETAR || c.arch == FL_ARCH_TOZARAX || c.arch == FL_ARCH_MEDULORN, FL_ERR_INVALID,
+    FL_CHECK(c.arch == FL_ARCH_NIFUNEX || c.arch == FL_ARCH_ROFETAR || c.arch == FL_ARCH_TOZARAX || c.arch == FL_ARCH_MEDULORN ||
+                 c.arch == FL_ARCH_LATODRA, FL_ERR_INVALID,
              "layered models: unknown arch");
     FL_CHECK(c.vocab >= 1 && c.width >= 1 && c.n_layers >= 1 && c.n_layers <= 4096, FL_ERR_INVALID, "layered models: sizes must be positive");
     FL_CHECK(c.compute_dtype == FL_DTYPE_BF16 || c.compute_dtype == FL_DTYPE_F32, FL_ERR_INVALID, "compute_dtype must be bf16 or f32");
@@ -146,13 +148,36 @@ void layered_build(LayeredModel& m, const fl_layer_desc* descs) {
     FL_CHECK(!(c.token_shift && c.canon_taps > 0), FL_ERR_UNSUPPORTED, "a stack has a token shift or input convolutions, not both");
     FL_CHECK(!c.token_shift || c.no_pre_norm, FL_ERR_UNSUPPORTED, "the token shift is built for stacks whose mixers read the stream itself");
     FL_CHECK(c.logit_softcap >= 0.f, FL_ERR_INVALID, "negative logit cap");
+    const bool both_norms = !c.no_pre_norm && !c.no_post_norm && !c.post_sum_norm;
+    FL_CHECK(!c.layer_scale || both_norms, FL_ERR_UNSUPPORTED, "layer scales are built for stacks with a norm before and after every sublayer");
+    FL_CHECK(!(c.tied_head && c.max_positions > 0), FL_ERR_UNSUPPORTED, "a tied output projection with a position table is not built");
+    if (c.loop_times > 0) {
+        FL_CHECK(c.loop_start >= 0 && c.loop_stop > c.loop_start && c.loop_stop <= c.n_layers && c.loop_times <= 4096, FL_ERR_INVALID, "bad loop span");
+        FL_CHECK(both_norms || !(c.loop_reinject || c.loop_step), FL_ERR_UNSUPPORTED,
+                 "what a loop adds between its passes is built for stacks with a norm before and after every sublayer");
+        FL_CHECK(!c.depth_avg, FL_ERR_UNSUPPORTED, "a loop and a depth average do not go together");
+    } else {
+        FL_CHECK(c.loop_times == 0 && !c.loop_reinject && !c.loop_step, FL_ERR_INVALID, "loop options without a loop");
+    }
     m.W = c.width; m.V = c.vocab; m.L = c.n_layers; m.f32 = c.compute_dtype == FL_DTYPE_F32;
     m.layers.resize(m.L);
     struct Reg { void** pp; size_t bytes; };
     std::vector<Reg> regs;
     auto reg = [&](auto** pp, size_t bytes) { regs.push_back({(void**)pp, bytes}); };
     const size_t W = m.W;
-    reg(&m.embed, (size_t)m.V * W * 2); reg(&m.head, (size_t)m.V * W * 2); reg(&m.final_norm, W * 4);
+    reg(&m.embed, (size_t)m.V * W * 2); reg(&m.final_norm, W * 4);
+    if (!c.tied_head) reg(&m.head, (size_t)m.V * W * 2);
+    if (c.embed_norm) reg(&m.embed_norm, W * 4);
+    if (c.loop_step) reg(&m.loop_step, (size_t)c.loop_times * W * 4);
+    // the order of computation: the layers before the loop, its passes, the layers behind it
+    const bool loop = c.loop_times > 0;
+    auto passes = [&](int i) { return loop && i >= c.loop_start && i < c.loop_stop ? c.loop_times : 1; };
+    for (int i = 0; i < m.L; ++i) {
+        if (!loop || i != c.loop_start) { m.runs.push_back({i, 0, false}); continue; }
+        for (int t = 0; t < c.loop_times; ++t)
+            for (int k = c.loop_start; k < c.loop_stop; ++k) m.runs.push_back({k, t, k == c.loop_start});
+        i = c.loop_stop - 1;
+    }
     if (c.max_positions > 0) reg(&m.pos, (size_t)c.max_positions * W * 2);
     auto pad8 = [](int n) { return (n + 7) / 8 * 8; };
     // one mixer: its rows inside the layer's stacked input matrix start at `base`; registers its side tables and its cache / state
@@ -161,7 +186,7 @@ void layered_build(LayeredModel& m, const fl_layer_desc* descs) {
         const size_t H = d.heads, D = d.dim, Dv = d.vdim;
         auto recurrent = [&]() {                        // a per-slot state [heads][rows][vdim] + the per-head decay parameters
             lw.gla_index = (int)m.gla_layers.size();
-            m.gla_layers.push_back(&lw);
+            m.gla_layers.insert(m.gla_layers.end(), passes(i), &lw);
             m.max_heads = std::max<int>(m.max_heads, (int)H);
         };
         auto rope = [&]() {
@@ -185,8 +210,9 @@ void layered_build(LayeredModel& m, const fl_layer_desc* descs) {
                 if (!d.no_qk_norm) reg(&lw.knorm, (d.qk_norm_whole ? G * D : D) * 4);
                 lw.kv_owner = i;
                 lw.kv_index = (int)m.kv_layers.size();
-                m.kv_layers.push_back(&lw);
+                m.kv_layers.insert(m.kv_layers.end(), passes(i), &lw);
             } else {
+                FL_CHECK(passes(i) == 1 && passes(d.kv_from) == 1, FL_ERR_UNSUPPORTED, "kv_from is not built for layers of a loop");
                 lw.kv_owner = d.kv_from;
                 lw.kv_index = m.layers[d.kv_from].kv_index;
             }
@@ -224,22 +250,30 @@ void layered_build(LayeredModel& m, const fl_layer_desc* descs) {
             lw.n_in = lw.off_a + d.decay_rank;
             reg(&lw.a2, H * D * d.decay_rank * 2); reg(&lw.a2b, H * D * 4); reg(&lw.hnorm, Dv * 4);
             lw.gla_index = (int)m.gla_layers.size();
-            m.gla_layers.push_back(&lw);
+            m.gla_layers.insert(m.gla_layers.end(), passes(i), &lw);
             m.max_hd = std::max<int>(m.max_hd, (int)(H * D));
         } else {
-            const size_t R = d.rot_dim, C = d.kv_rank;
-            lw.off_q = 0; lw.n_in = (int)(H * (D + R));
-            lw.off_dkv = -1;
+            const size_t R = d.rot_dim, C = d.kv_rank, Q = d.q_rank;
+            lw.off_q = 0; lw.n_in = (int)(Q > 0 ? Q : H * (D + R));
+            if (Q > 0) {
+                reg(&lw.dq_norm, Q * 4); reg(&lw.uq, H * (D + R) * Q * 2);
+                m.max_qr = std::max<int>(m.max_qr, (int)Q); m.max_q = std::max<int>(m.max_q, (int)(H * (D + R)));
+            }
+            lw.off_dkv = -1; lw.off_g = -1;
             if (d.kv_from < 0) {
                 lw.off_dkv = lw.n_in; lw.n_in += (int)(C + R);
                 reg(&lw.dkv_norm, C * 4);
                 lw.kv_owner = i;
                 lw.kv_index = (int)m.kv_layers.size();
-                m.kv_layers.push_back(&lw);
+                m.kv_layers.insert(m.kv_layers.end(), passes(i), &lw);
             } else {
+                FL_CHECK(passes(i) == 1 && passes(d.kv_from) == 1, FL_ERR_UNSUPPORTED, "kv_from is not built for layers of a loop");
                 lw.kv_owner = d.kv_from;
                 lw.kv_index = m.layers[d.kv_from].kv_index;
             }
+            if (d.out_gate) { lw.off_g = lw.n_in; lw.n_in += (int)(H * Dv); }
+            if (Q > 0 || d.out_gate) lw.n_in = pad8(lw.n_in);
+            if (d.sink == 2) reg(&lw.sinkv, H * 4);
             reg(&lw.uk_t, H * C * D * 2); reg(&lw.uv, H * Dv * C * 2);
             rope();
             m.max_hc = std::max<int>(m.max_hc, (int)(H * C));
@@ -262,6 +296,7 @@ void layered_build(LayeredModel& m, const fl_layer_desc* descs) {
         const bool pre = !c.no_pre_norm, post = !c.no_post_norm;
         if (pre) reg(&lw.norm1, W * 4);
         if (post) reg(&lw.norm1b, W * 4);
+        if (c.layer_scale) reg(&lw.ls1, W * 4);
         if (c.token_shift) reg(&lw.shift, W * 4);
         build_mixer(lw, i, 0);
         if (d.beside) {
@@ -278,12 +313,13 @@ void layered_build(LayeredModel& m, const fl_layer_desc* descs) {
         }
         reg(&lw.w_in, (size_t)lw.n_in * W * 2);
         m.max_in = std::max(m.max_in, lw.n_in);
-        if (c.canon_taps > 0) { reg(&lw.canon1, W * c.canon_taps * 4); lw.canon_index = i; }
+        if (c.canon_taps > 0) reg(&lw.canon1, W * c.canon_taps * 4);
         if (c.gated_residual) { reg(&lw.rg1, W * W * 2); reg(&lw.rg1b, W * 4); }
         if (c.depth_avg) reg(&lw.dwa, (size_t)(i + 2) * 4);
         if (d.ffn != FL_FFN_NONE) {
             if (pre) reg(&lw.norm2, W * 4);
             if (post) reg(&lw.norm2b, W * 4);
+            if (c.layer_scale) reg(&lw.ls2, W * 4);
             if (c.canon_taps > 0) reg(&lw.canon2, W * c.canon_taps * 4);
             if (c.gated_residual) { reg(&lw.rg2, W * W * 2); reg(&lw.rg2b, W * 4); }
             if (d.ffn == FL_FFN_DENSE && d.ffn_bias) { reg(&lw.b_gu, (size_t)2 * d.ff * 4); reg(&lw.b_down, W * 4); }
@@ -309,7 +345,8 @@ void layered_build(LayeredModel& m, const fl_layer_desc* descs) {
     m.slab.alloc(total, /*zero=*/true);
     size_t off = 0;
     for (const Reg& r : regs) { *r.pp = m.slab.p + off; off += up256(r.bytes); }
-    m.weight_bytes = total - up256((size_t)m.V * W * 2) - (c.max_positions > 0 ? up256((size_t)c.max_positions * W * 2) : 0);
+    if (c.tied_head) m.head = m.embed;
+    m.weight_bytes = total - (c.tied_head ? 0 : up256((size_t)m.V * W * 2)) - (c.max_positions > 0 ? up256((size_t)c.max_positions * W * 2) : 0);
 
     // names -> destinations
     LayeredRoutes R;
@@ -319,7 +356,10 @@ void layered_build(LayeredModel& m, const fl_layer_desc* descs) {
     auto vec = [&](const std::string& n, float* base, int64_t rows, int64_t cols) { R.r[n] = LyRoute{LyRoute::F32, base, rows, cols, 0}; };
     // a layer norm's weight: [W], or one number for all channels (norm_scalar), kept as W equal floats so that the kernels index it alike
     auto normw = [&](const std::string& n, float* base) { R.r[n] = LyRoute{c.norm_scalar ? LyRoute::F32_FILL : LyRoute::F32, base, (int64_t)W, 1, 0}; };
-    mat("embed", m.embed, 0, m.V, W); mat("head", m.head, 0, m.V, W); normw("final.norm", m.final_norm);
+    mat("embed", m.embed, 0, m.V, W); normw("final.norm", m.final_norm);
+    if (!c.tied_head) mat("head", m.head, 0, m.V, W);
+    if (m.embed_norm != nullptr) normw("embed.norm", m.embed_norm);
+    if (m.loop_step != nullptr) vec("loop.step", m.loop_step, c.loop_times, W);
     if (m.pos != nullptr) mat("pos", m.pos, 0, c.max_positions, W);
     // the tensors of one mixer, named p + "q" and so on (p = "l<i>.mix." or "l<i>.mix.left." / "l<i>.mix.right.")
     auto route_mixer = [&](const LayeredLayerW& lw, const std::string& p) {
@@ -360,8 +400,14 @@ void layered_build(LayeredModel& m, const fl_layer_desc* descs) {
             mat(p + "a1", lw.w_in, lw.off_a, d.decay_rank, W);
             mat(p + "a2", lw.a2, 0, H * D, d.decay_rank); vec(p + "a2.b", lw.a2b, H * D, 1); vec(p + "norm", lw.hnorm, Dv, 1);
         } else {
-            const int64_t Rr = d.rot_dim, C = d.kv_rank;
-            mat(p + "q", lw.w_in, lw.off_q, H * (D + Rr), W);
+            const int64_t Rr = d.rot_dim, C = d.kv_rank, Q = d.q_rank;
+            if (Q > 0) {
+                mat(p + "dq", lw.w_in, lw.off_q, Q, W); vec(p + "dq.norm", lw.dq_norm, Q, 1); mat(p + "uq", lw.uq, 0, H * (D + Rr), Q);
+            } else {
+                mat(p + "q", lw.w_in, lw.off_q, H * (D + Rr), W);
+            }
+            if (d.out_gate) mat(p + "g", lw.w_in, lw.off_g, H * Dv, W);
+            if (d.sink == 2) vec(p + "sink", lw.sinkv, H, 1);
             if (d.kv_from < 0) { mat(p + "dkv", lw.w_in, lw.off_dkv, C + Rr, W); vec(p + "dkv.norm", lw.dkv_norm, C, 1); }
             R.r[p + "uk"] = LyRoute{LyRoute::UK_T, lw.uk_t, H * D, C, (int)H};
             mat(p + "uv", lw.uv, 0, H * Dv, C);
@@ -376,6 +422,8 @@ void layered_build(LayeredModel& m, const fl_layer_desc* descs) {
         if (pre && post) { normw(p + "norm1", lw.norm1); normw(p + "norm1b", lw.norm1b); }
         else normw(p + "norm1", pre ? lw.norm1 : lw.norm1b);
         if (lw.shift) vec(p + "shift", lw.shift, W, 1);
+        if (lw.ls1) vec(p + "ls1", lw.ls1, W, 1);
+        if (lw.ls2) vec(p + "ls2", lw.ls2, W, 1);
         if (lw.side) {
             lw.side->w_in = lw.w_in;
             route_mixer(lw, p + "mix.left."); route_mixer(*lw.side, p + "mix.right.");
@@ -481,10 +529,10 @@ void layered_random_init(LayeredModel& m, uint64_t seed, float stdv) {
         if (r->kind == LyRoute::F32 || r->kind == LyRoute::F32_RAW || r->kind == LyRoute::F32_FILL) {
             auto ends = [&](const char* t) { const size_t k = std::strlen(t); return n.size() >= k && n.compare(n.size() - k, k, t) == 0; };
             // a plain norm weight sits around one, a zero-centred one around zero
-            const bool around_one = ends("mix.norm") || ends("left.norm") || ends("right.norm") || ends("dkv.norm") || ends("q.norm") || ends("k.norm") || ends("mix.D") || ends("left.out") || ends("right.out") ||
+            const bool around_one = ends("mix.norm") || ends("left.norm") || ends("right.norm") || ends("dkv.norm") || ends("dq.norm") || n == "embed.norm" || ends(".ls1") || ends(".ls2") || ends("q.norm") || ends("k.norm") || ends("mix.D") || ends("left.out") || ends("right.out") ||
                                     (m.cfg.norm_plain && (ends("norm1") || ends("norm2") || ends("norm1b") || ends("norm2b") || n == "final.norm"));
             const bool is_mat = n.find("router") != std::string::npos || n.find("mix.a2") != std::string::npos || n.find("shared.sg") != std::string::npos ||
-                                ends(".conv") || ends(".canon1") || ends(".canon2");
+                                ends(".conv") || ends(".canon1") || ends(".canon2") || n == "loop.step";
             const bool is_bias = n.size() >= 4 && n.compare(n.size() - 4, 4, "a2.b") == 0;
             if (around_one) fill_f32_kernel<<<8, 256>>>((float*)r->dst, numel, 1.0f);
             else if (ends(".decay")) fill_f32_kernel<<<8, 256>>>((float*)r->dst, numel, 0.96875f);
@@ -494,7 +542,7 @@ void layered_random_init(LayeredModel& m, uint64_t seed, float stdv) {
             else if (is_mat) synth_fill_f32_kernel<<<kNumSMs, 256>>>((float*)r->dst, numel, ts, stdv, ident);
             else fill_f32_kernel<<<8, 256>>>((float*)r->dst, numel, 0.0f);
         } else {
-            synth_fill_bf16_kernel<<<kNumSMs * 8, 256>>>((uint16_t*)r->dst, 1, numel, numel, ts, n == "embed" ? 1.0f : stdv, ident);
+            synth_fill_bf16_kernel<<<kNumSMs * 8, 256>>>((uint16_t*)r->dst, 1, numel, numel, ts, n == "embed" && !m.cfg.tied_head ? 1.0f : stdv, ident);
         }
         g_launches.fetch_add(1);
         m.have.insert(n);
@@ -522,6 +570,12 @@ void layered_finalize(LayeredModel& m) {
             const fl_layer_desc& d = lw.d;
             map(lw.w_in, lw.n_in, m.W, lw.tm_in, lw.tc_in);
             map(lw.w_o, m.W, d.heads * d.vdim, lw.tm_o, lw.tc_o);
+            // (a query latent may end inside a k block: the tensor maps fill its rest with zeros)
+            lw.tc_uq = lw.uq != nullptr && d.q_rank % 8 == 0 && d.heads * (d.dim + d.rot_dim) % 8 == 0;
+            if (lw.tc_uq) {
+                const uint64_t nq = (uint64_t)d.heads * (d.dim + d.rot_dim), Q = d.q_rank;
+                lw.tm_uq = make_tmap_bf16(lw.uq, nq, Q, Q, 128);
+            }
             if (lw.side) map(lw.side->w_o, m.W, lw.side->d.heads * lw.side->d.vdim, lw.side->tm_o, lw.side->tc_o);
             map(lw.rg1, m.W, m.W, lw.tm_rg1, lw.tc_rg1); map(lw.rg2, m.W, m.W, lw.tm_rg2, lw.tc_rg2);
             const int GF = d.ffn_act == FL_ACT_RELU2 ? d.ff : 2 * d.ff;       // rows of the first feed-forward matrix: up, or gate | up
@@ -617,12 +671,12 @@ void layered_cache_create(fl_cache& c, int max_slots, int max_seq, int pool_toke
         if (lw.conv_ch > 0 && d.conv > 1) y.conv_state[k].alloc((size_t)max_slots * (d.conv - 1) * lw.conv_ch, true);
     }
     if (m.cfg.canon_taps > 1) {
-        y.canon_state.resize(m.L);
-        for (int i = 0; i < m.L; ++i) y.canon_state[i].alloc((size_t)2 * max_slots * (m.cfg.canon_taps - 1) * m.W, true);
+        y.canon_state.resize(m.runs.size());
+        for (size_t i = 0; i < m.runs.size(); ++i) y.canon_state[i].alloc((size_t)2 * max_slots * (m.cfg.canon_taps - 1) * m.W, true);
     }
     if (m.cfg.token_shift) {
-        y.shift_state.resize(m.L);
-        for (int i = 0; i < m.L; ++i) y.shift_state[i].alloc((size_t)max_slots * m.W, true);
+        y.shift_state.resize(m.runs.size());
+        for (size_t i = 0; i < m.runs.size(); ++i) y.shift_state[i].alloc((size_t)max_slots * m.W, true);
     }
     y.rope_cos.resize(m.ropes.size()); y.rope_sin.resize(m.ropes.size());
     for (size_t k = 0; k < m.ropes.size(); ++k) {
@@ -670,6 +724,8 @@ static void ensure_ws(fl_cache& c, size_t T, size_t n_want) {
         if (m.cfg.canon_taps > 0 || m.cfg.token_shift) y.hc.alloc(R * W);
         if (m.cfg.gated_residual) y.gz.alloc(R * W);
         if (m.cfg.depth_avg) y.xs.alloc((size_t)(m.L + 1) * R * W);
+        else if (m.cfg.loop_reinject) y.xs.alloc(R * W);
+        if (m.max_qr > 0) { y.cq.alloc(R * m.max_qr); y.qx.alloc(R * m.max_q); }
         for (const LayeredLayerW& lw : m.layers)
             if (lw.side && y.y2.n < R * W) y.y2.alloc(R * W);
         y.qa.alloc(R * std::max(m.max_hc, 1)); y.ol.alloc(R * std::max(m.max_hc, 1));
@@ -679,10 +735,11 @@ static void ensure_ws(fl_cache& c, size_t T, size_t n_want) {
         y.pair_row.alloc(P); y.pair_of.alloc(P); y.grp_off.alloc((size_t)m.max_experts + 2);
         if (!m.f32) {
             y.h_hi.alloc(R * W); y.h_lo.alloc(R * W);
+            if (m.max_qr > 0) { y.cq_hi.alloc(R * m.max_qr); y.cq_lo.alloc(R * m.max_qr); }
             y.u_hi.alloc(R * std::max(m.max_hv, 1)); y.u_lo.alloc(R * std::max(m.max_hv, 1));
             y.act_hi.alloc(R * std::max(m.max_ff, 1)); y.act_lo.alloc(R * std::max(m.max_ff, 1));
             // split-K slices of a tensor-core GEMM with <= 128 rows: ks * rows <= 256 (see pick_ksplit)
-            const size_t nmax = std::max<size_t>(std::max<size_t>(m.max_in, W), std::max<size_t>(2 * (size_t)m.max_ff, m.V));
+            const size_t nmax = std::max<size_t>(std::max<size_t>(std::max(m.max_in, m.max_q), W), std::max<size_t>(2 * (size_t)m.max_ff, m.V));
             size_t need = 256 * nmax;
             size_t gx_rows = 0;
             for (const LayeredLayerW& lw : m.layers) {          // grouped expert GEMMs: [slices][experts * cap rows][2 ff | W]
@@ -858,7 +915,7 @@ static void latent_attn_tc(fl_cache& c, LaunchCtx& lc, const LayeredLayerW& lw, 
         dense_gemm(c, lc, "gemm_tc_attn_scores", rows, nkp, Ep, tk, y.at_s.p, y.at_qhi.p, y.at_qlo.p);
         const int keep = std::min(nkp, kSoftmaxKeep);
         launch(lc, "attn_softmax", 0, ly_attn_softmax_kernel, dim3(rows), dim3(256), (size_t)keep * 4, (const float*)y.at_s.p, a.row_pos, r0 + f, H, k_lo, 0, nk, nkp,
-               a.window, 0, 0, 0.f, 0, (const float*)nullptr, keep, y.at_phi.p, y.at_plo.p);
+               a.window, 0, 0, 0.f, a.sink, a.sinkv, keep, y.at_phi.p, y.at_plo.p);
         const CUtensorMap tv = make_tmap_bf16(y.at_kct.p, (uint64_t)C, (uint64_t)nkp, (uint64_t)nkp, 128);
         dense_gemm(c, lc, "gemm_tc_attn_values", rows, C, nkp, tv, a.ol + (size_t)(r0 + f) * H * C, y.at_phi.p, y.at_plo.p);
     }
@@ -1024,20 +1081,21 @@ void layered_forward(fl_cache& c, const int* slots, const int* counts, int n, co
     for (int i = 0; i < n; ++i) c.slot_len[slots[i]] += counts[i];
 }
 
-// One mixer over all rows of the step: reads its columns of the projected buffer y.proj (row stride lw.n_in), its cache pages / state
+// One mixer over all rows of the step (`pass`: which pass of a loop, 0 elsewhere -- its own cache and state): reads its columns of the projected buffer y.proj (row stride lw.n_in), its cache pages / state
 // slots, and leaves the mixer's inner output (what its output projection reads) in y.u with the hi | lo halves when that
 // projection runs on the tensor cores.
-static void run_mixer(fl_cache& c, LaunchCtx& lc, const StepTab& st, const LayeredLayerW& lw, const int* slots, const int* counts, int n,
+static void run_mixer(fl_cache& c, LaunchCtx& lc, const StepTab& st, const LayeredLayerW& lw, int pass, const int* slots, const int* counts, int n,
                       const int* h_row0, const int* h_pos0) {
     const LayeredModel& m = *c.lm;
     LayeredCache& y = *c.ly;
     const fl_layer_desc& d = lw.d;
     const int Ti = st.T, H = d.heads, D = d.dim, Dv = d.vdim;
     const float eps = m.cfg.norm_eps;
+    const int kv_index = lw.kv_index + pass, gla_index = lw.gla_index + pass;
     uint16_t *uhi = m.f32 ? nullptr : y.u_hi.p, *ulo = m.f32 ? nullptr : y.u_lo.p;
     if (d.mixer == FL_MIXER_ATTN) {
         const int G = d.kv_heads;
-        AttnPrepArgs pa{y.proj.p, lw.n_in, lw.off_q, lw.off_k, lw.off_v, lw.qnorm, lw.knorm, eps, y.kv_pool[lw.kv_index], y.page_table.p,
+        AttnPrepArgs pa{y.proj.p, lw.n_in, lw.off_q, lw.off_k, lw.off_v, lw.qnorm, lw.knorm, eps, y.kv_pool[kv_index], y.page_table.p,
                         c.pages_per_seq, st.row_seq, st.row_pos, st.seq_slot, y.rope_cos[lw.rope_index].p, y.rope_sin[lw.rope_index].p,
                         H, G, D, Dv, d.rot_dims, d.rot_halves, lw.bq, lw.bk, lw.bv, d.qk_norm_whole};
         // eight warps per block take the heads in turn; steps of few rows spread a row's heads over up to four blocks (not with a
@@ -1046,7 +1104,7 @@ static void run_mixer(fl_cache& c, LaunchCtx& lc, const StepTab& st, const Layer
         const int heads_all = H + (lw.off_k >= 0 ? G : 0), py = (Ti <= 64 && !d.qk_norm_whole) ? std::max(1, std::min(4, (heads_all + 7) / 8)) : 1;
         if (m.f32) launch(lc, "attn_prep", 0, ly_attn_prep_kernel<float>, dim3(Ti, py), dim3(256), psm, pa);
         else launch(lc, "attn_prep", 0, ly_attn_prep_kernel<uint16_t>, dim3(Ti, py), dim3(256), psm, pa);
-        GqaAttnArgs at{y.proj.p, lw.n_in, lw.off_q, y.kv_pool[lw.kv_index], y.page_table.p, c.pages_per_seq, st.row_seq, st.row_pos, st.seq_slot,
+        GqaAttnArgs at{y.proj.p, lw.n_in, lw.off_q, y.kv_pool[kv_index], y.page_table.p, c.pages_per_seq, st.row_seq, st.row_pos, st.seq_slot,
                        y.u.p, lw.tc_o ? uhi : (uint16_t*)nullptr, ulo, H, G, D, Dv, d.window, d.scale, d.softcap, d.sink, 0, y.at_part.p,
                        d.keep_first, d.mask_chunk, lw.sinkv};
         // a step of single tokens is replayed from a captured graph whatever the contexts' lengths: its split count must not follow them
@@ -1080,7 +1138,7 @@ static void run_mixer(fl_cache& c, LaunchCtx& lc, const StepTab& st, const Layer
     } else if (d.mixer == FL_MIXER_MAMBA2 || d.mixer == FL_MIXER_DELTA) {
         const bool delta = d.mixer == FL_MIXER_DELTA;
         const int G = delta ? d.kv_heads : d.groups, rows = delta ? D : d.state;
-        float* cstate = d.conv > 1 ? y.conv_state[lw.gla_index].p : nullptr;
+        float* cstate = d.conv > 1 ? y.conv_state[gla_index].p : nullptr;
         ConvArgs ca{y.proj.p, lw.n_in, lw.conv_off, lw.conv_w, lw.conv_b, cstate, st.row_seq, st.row_pos, st.seq_row0, st.seq_slot, st.seq_pos0,
                     lw.conv_ch, d.conv, y.cv.p};
         // channel chunks per row: whole q / k heads for the delta rule (they are normalised inside one block)
@@ -1094,7 +1152,7 @@ static void run_mixer(fl_cache& c, LaunchCtx& lc, const StepTab& st, const Layer
         if (d.conv > 1) launch(lc, "conv_state", 0, ly_conv_state_kernel, dim3(n, (lw.conv_ch + 127) / 128), dim3(128), 0, ca);
         // column offsets inside cv (the convolved span starts at conv_off)
         RecArgs ra{y.cv.p, lw.conv_ch, lw.off_q - lw.conv_off, lw.off_k - lw.conv_off, lw.off_v - lw.conv_off, y.rs.p,
-                   delta ? (const float*)nullptr : (const float*)lw.dskip, y.go.p, y.gla_state[lw.gla_index].p, st.seq_row0, st.seq_slot, st.seq_pos0,
+                   delta ? (const float*)nullptr : (const float*)lw.dskip, y.go.p, y.gla_state[gla_index].p, st.seq_row0, st.seq_slot, st.seq_pos0,
                    H, G, rows, Dv};
         if (delta) {
             launch_rec_scan<true>(lc, ra, n);
@@ -1112,7 +1170,7 @@ static void run_mixer(fl_cache& c, LaunchCtx& lc, const StepTab& st, const Layer
         launch(lc, "lightning_prep", 0, ly_lightning_prep_kernel, dim3(Ti, nchunk), dim3(256), 0, (const float*)y.proj.p, lw.n_in, lw.conv_off, lw.conv_ch, chunk,
                (const float*)lw.decay, H, y.cv.p, y.rs.p);
         RecArgs ra{y.cv.p, lw.conv_ch, lw.off_q - lw.conv_off, lw.off_k - lw.conv_off, lw.off_v - lw.conv_off, y.rs.p, (const float*)nullptr, y.go.p,
-                   y.gla_state[lw.gla_index].p, st.seq_row0, st.seq_slot, st.seq_pos0, H, H, D, Dv};
+                   y.gla_state[gla_index].p, st.seq_row0, st.seq_slot, st.seq_pos0, H, H, D, Dv};
         launch_rec_scan<false>(lc, ra, n);
         const bool v4 = ((inner | lw.n_in | lw.off_g) & 3) == 0;       // four channels per thread
         launch(lc, "gated_group_norm", 0, ly_gated_group_norm_kernel, dim3(Ti, 1), dim3(std::min(v4 ? 256 : 1024, std::max(64, ((v4 ? inner / 4 : inner) + 31) / 32 * 32))), 0,
@@ -1121,22 +1179,33 @@ static void run_mixer(fl_cache& c, LaunchCtx& lc, const StepTab& st, const Layer
     } else if (d.mixer == FL_MIXER_GLA) {
         // decay pre-activation through the rank-r bottleneck: z = W_a2 a (the bias and the sigmoid^(1/tau) are applied by the scan)
         gemm(lc, "gemm_gla_decay", y.proj.p + lw.off_a, lw.n_in, lw.a2, H * D, d.decay_rank, y.la.p, H * D, Ti);
-        GlaArgs ga{y.proj.p, lw.n_in, lw.off_q, lw.off_k, lw.off_v, y.la.p, lw.a2b, 1.f / d.tau, y.go.p, y.gla_state[lw.gla_index].p, st.seq_row0,
+        GlaArgs ga{y.proj.p, lw.n_in, lw.off_q, lw.off_k, lw.off_v, y.la.p, lw.a2b, 1.f / d.tau, y.go.p, y.gla_state[gla_index].p, st.seq_row0,
                    st.seq_slot, st.seq_pos0, H, D, Dv, (float)(1.0 / std::sqrt((double)D))};
         launch_gla_scan(lc, ga, n);
         launch(lc, "gla_out", 0, ly_gla_out_kernel, dim3((Ti * H + 7) / 8), dim3(256), 0, (const float*)ga.o, (const float*)y.proj.p, lw.n_in, lw.off_g,
                (const float*)lw.hnorm, eps, Ti, H, Dv, y.u.p, lw.tc_o ? uhi : (uint16_t*)nullptr, ulo);
     } else {
-        const int R = d.rot_dim, C = d.kv_rank;
-        LatentAppendArgs aa{y.proj.p, lw.n_in, lw.off_q, lw.off_dkv, lw.dkv_norm, eps, y.kv_pool[lw.kv_index], y.page_table.p, c.pages_per_seq,
-                            st.row_seq, st.row_pos, st.seq_slot, y.rope_cos[lw.rope_index].p, y.rope_sin[lw.rope_index].p, H, D, R, C, d.rot_dims};
+        const int R = d.rot_dim, C = d.kv_rank, Q = d.q_rank;
+        LatentAppendArgs aa{y.proj.p, lw.n_in, lw.off_q, lw.off_dkv, lw.dkv_norm, eps, y.kv_pool[kv_index], y.page_table.p, c.pages_per_seq,
+                            st.row_seq, st.row_pos, st.seq_slot, y.rope_cos[lw.rope_index].p, y.rope_sin[lw.rope_index].p, H, D, R, C, d.rot_dims, lw.off_q, Q, lw.dq_norm, y.cq.p,
+                            lw.tc_uq ? y.cq_hi.p : (uint16_t*)nullptr, y.cq_lo.p};
         if (m.f32) launch(lc, "latent_append", 0, ly_latent_append_kernel<float>, dim3(Ti), dim3(128), 0, aa);
         else launch(lc, "latent_append", 0, ly_latent_append_kernel<uint16_t>, dim3(Ti), dim3(128), 0, aa);
+        // queries [T][H][D + R]: columns of the projected buffer, or expanded from the normed query latent
+        float* q = y.proj.p + lw.off_q;
+        int ldq = lw.n_in;
+        if (Q > 0) {
+            q = y.qx.p; ldq = H * (D + R);
+            gemm_tc_or_exact(c, lc, "gemm_q_up", y.cq.p, y.cq_hi.p, y.cq_lo.p, lw.uq, lw.tm_uq, lw.tc_uq, ldq, Q, q, Ti);
+            if (d.rot_dims > 0)
+                launch(lc, "rotate_q", 0, ly_rotate_q_kernel, dim3(Ti), dim3(128), 0, q, ldq, st.row_pos, (const float*)y.rope_cos[lw.rope_index].p,
+                       (const float*)y.rope_sin[lw.rope_index].p, H, D, R, d.rot_dims);
+        }
         // q~[row, h, :] = W_uk[h]^T q_plain[row, h, :]: the score against the latent needs no per-head keys
-        LyGemm qa{y.proj.p + lw.off_q, D + R, lw.n_in, nullptr, lw.uk_t, (long long)C * D, C, D, y.qa.p, C, H * C, nullptr, Ti};
+        LyGemm qa{q, D + R, ldq, nullptr, lw.uk_t, (long long)C * D, C, D, y.qa.p, C, H * C, nullptr, Ti};
         gemm_groups(lc, "gemm_q_absorb", qa, H, Ti);
-        LatentAttnArgs at{y.qa.p, y.proj.p, lw.n_in, lw.off_q, y.kv_pool[lw.kv_index], y.page_table.p, c.pages_per_seq, st.row_seq, st.row_pos,
-                          st.seq_slot, y.ol.p, H, D, R, C, d.window, d.scale, 0};
+        LatentAttnArgs at{y.qa.p, q, ldq, 0, y.kv_pool[kv_index], y.page_table.p, c.pages_per_seq, st.row_seq, st.row_pos,
+                          st.seq_slot, y.ol.p, H, D, R, C, d.window, d.scale, 0, d.sink, lw.sinkv};
         // long portions (serving precision): scores and weighted sums as tensor-core GEMMs over the gathered window; everything
         // else (decoded tokens, short portions, the exact mode) on the per-(row, head) kernel.  Rows are taken in order.
         static const bool tc_attn_off = env_flag("FL_LAYERED_NO_TC_ATTN");
@@ -1158,8 +1227,11 @@ static void run_mixer(fl_cache& c, LaunchCtx& lc, const StepTab& st, const Layer
         // value expansion after the softmax: out[row, h, :] = W_uv[h] (sum_j p_j c_j)
         LyGemm ov{y.ol.p, C, H * C, nullptr, lw.uv, (long long)Dv * C, Dv, C, y.u.p, Dv, H * Dv, nullptr, Ti};
         gemm_groups(lc, "gemm_v_expand", ov, H, Ti);
-        if (lw.tc_o) {
-            const size_t nu = (size_t)Ti * H * Dv;
+        const size_t nu = (size_t)Ti * H * Dv;
+        if (d.out_gate) {
+            launch(lc, "out_gate", 0, ly_out_gate_kernel, dim3((unsigned)std::min<size_t>(4 * kNumSMs, (nu + 255) / 256)), dim3(256), 0, y.u.p, (const float*)y.proj.p,
+                   lw.n_in, lw.off_g, H * Dv, Ti, lw.tc_o ? uhi : (uint16_t*)nullptr, ulo);
+        } else if (lw.tc_o) {
             launch(lc, "split_hi_lo", 0, ly_split_kernel, dim3((unsigned)std::min<size_t>(4 * kNumSMs, (nu + 255) / 256)), dim3(256), 0,
                    (const float*)y.u.p, nu, uhi, ulo);
         }
@@ -1187,17 +1259,17 @@ static void enqueue_step(fl_cache& c, LaunchCtx& lc, const StepTab& st, const in
     const float* sub_in = canon ? y.hc.p : norm_out;            // what the sublayer's own matrices read
     const size_t hist_stride = y.rows * (size_t)W;
     launch(lc, "embed_norm", 0, ly_embed_norm_kernel, dim3(Ti), dim3(nthr), 0, (const uint16_t*)m.embed, st.tok, W,
-           pre ? (const float*)m.layers[0].norm1 : (const float*)nullptr, eps, plain, (const uint16_t*)m.pos, st.row_pos, m.cfg.embed_scale, y.x.p,
-           depth ? y.xs.p : (float*)nullptr, y.h.p, hhi, hlo);
+           pre ? (const float*)m.layers[0].norm1 : (const float*)nullptr, eps, plain, (const uint16_t*)m.pos, st.row_pos, m.cfg.embed_scale, (const float*)m.embed_norm,
+           m.runs[0].pass_start ? (const float*)m.loop_step : (const float*)nullptr, y.x.p, depth || m.cfg.loop_reinject ? y.xs.p : (float*)nullptr, y.h.p, hhi, hlo);
     // in front of a sublayer: the gate's pre-activation from the normed input, then the input convolution (and its carried inputs)
-    auto sublayer_front = [&](const LayeredLayerW& lw, int sub) {
+    auto sublayer_front = [&](const LayeredLayerW& lw, int run, int sub) {
         if (gated) {
             const uint16_t* rg = sub == 0 ? lw.rg1 : lw.rg2;
             gemm_tc_or_exact(c, lc, "gemm_gate", norm_out, hhi, hlo, rg, sub == 0 ? lw.tm_rg1 : lw.tm_rg2, sub == 0 ? lw.tc_rg1 : lw.tc_rg2, W, W, y.gz.p, Ti);
         }
         if (canon) {
             const int taps = m.cfg.canon_taps;
-            float* cs = taps > 1 ? y.canon_state[lw.canon_index].p + (size_t)sub * c.max_batch * (taps - 1) * W : nullptr;
+            float* cs = taps > 1 ? y.canon_state[run].p + (size_t)sub * c.max_batch * (taps - 1) * W : nullptr;
             ConvArgs ca{norm_out, W, 0, sub == 0 ? lw.canon1 : lw.canon2, nullptr, cs, st.row_seq, st.row_pos, st.seq_row0, st.seq_slot, st.seq_pos0, W, taps, nullptr};
             // few rows: one row per block; long steps: a block walks 8 rows with its taps staged once
             const int rpb = Ti >= 1024 ? 8 : 1;
@@ -1213,8 +1285,8 @@ static void enqueue_step(fl_cache& c, LaunchCtx& lc, const StepTab& st, const in
     // stacks with a token shift: the mixer reads hc = x + (x_prev - x) * shift (x_prev from the row before, or the slot's carried
     // row); the slot then keeps this step's last row of x.  The shift kernel rewrites the hi | lo halves with those of hc.
     const bool shifted = m.cfg.token_shift != 0, sum_norm = m.cfg.post_sum_norm != 0;
-    auto shift_front = [&](const LayeredLayerW& lw, int li) {
-        ConvArgs ca{y.x.p, W, 0, nullptr, nullptr, y.shift_state[li].p, st.row_seq, st.row_pos, st.seq_row0, st.seq_slot, st.seq_pos0, W, 2, nullptr};
+    auto shift_front = [&](const LayeredLayerW& lw, int run) {
+        ConvArgs ca{y.x.p, W, 0, nullptr, nullptr, y.shift_state[run].p, st.row_seq, st.row_pos, st.seq_row0, st.seq_slot, st.seq_pos0, W, 2, nullptr};
         if (W % 4 == 0)
             launch(lc, "token_shift", 0, ly_token_shift_kernel<4>, dim3(Ti, (W / 4 + 127) / 128), dim3(128), 0, ca, (const float*)lw.shift, y.hc.p, hhi, hlo);
         else
@@ -1240,34 +1312,42 @@ static void enqueue_step(fl_cache& c, LaunchCtx& lc, const StepTab& st, const in
             launch(lc, "join", 0, ly_join_kernel<1>, dim3(Ti), dim3(nthr), 0, y.x.p, (const float*)y.y.p, y2, wa, wb, gz, gate_bias, y.xs.p, hist_stride,
                    hist_slot, dw, wnext, eps, W, plain, y.h.p, hhi, hlo);
     };
-    for (int li = 0; li < m.L; ++li) {
+    const int n_runs = (int)m.runs.size();
+    for (int run = 0; run < n_runs; ++run) {
+        const int li = m.runs[run].layer, pass = m.runs[run].pass;
         const LayeredLayerW& lw = m.layers[li];
         const fl_layer_desc& d = lw.d;
         const int H = d.heads, Dv = d.vdim;
-        sublayer_front(lw, 0);
-        if (shifted) shift_front(lw, li);
+        sublayer_front(lw, run, 0);
+        if (shifted) shift_front(lw, run);
         gemm_tc_or_exact(c, lc, "gemm_mix_in", shifted ? (const float*)y.hc.p : sub_in, hhi, hlo, lw.w_in, lw.tm_in, lw.tc_in, lw.n_in, W, y.proj.p, Ti);
-        run_mixer(c, lc, st, lw, slots, counts, n, h_row0, h_pos0);
+        run_mixer(c, lc, st, lw, pass, slots, counts, n, h_row0, h_pos0);
         gemm_tc_or_exact(c, lc, "gemm_mix_out", y.u.p, uhi, ulo, lw.w_o, lw.tm_o, lw.tc_o, W, H * Dv, y.y.p, Ti);
         if (lw.side) {
             const LayeredLayerW& sw = *lw.side;
-            run_mixer(c, lc, st, sw, slots, counts, n, h_row0, h_pos0);
+            run_mixer(c, lc, st, sw, pass, slots, counts, n, h_row0, h_pos0);
             gemm_tc_or_exact(c, lc, "gemm_mix_out", y.u.p, uhi, ulo, sw.w_o, sw.tm_o, sw.tc_o, W, sw.d.heads * sw.d.vdim, y.y2.p, Ti);
         }
-        const float* next1 = (pre && li + 1 < m.L) ? m.layers[li + 1].norm1 : nullptr;
-        const int more = li + 1 < m.L ? split_x : 0;       // whether another sublayer reads x after this layer
-        const bool has_ff = d.ffn != FL_FFN_NONE;
+        const bool last = run + 1 == n_runs, has_ff = d.ffn != FL_FFN_NONE;
+        const float* next1 = (pre && !last) ? m.layers[m.runs[run + 1].layer].norm1 : nullptr;
+        const int more = last ? 0 : split_x;               // whether another sublayer reads x after this layer
+        // what joins the stream between this layer and the next run when that one starts a pass of the loop
+        const bool into_pass = !last && m.runs[run + 1].pass_start;
+        const int next_pass = into_pass ? m.runs[run + 1].pass : 0;
+        const float* again = (into_pass && next_pass > 0 && m.cfg.loop_reinject) ? (const float*)y.xs.p : (const float*)nullptr;
+        const float* pstep = (into_pass && m.cfg.loop_step) ? (const float*)m.loop_step + (size_t)next_pass * W : (const float*)nullptr;
         if (sum_norm)
             sum_norm_join(nullptr, lw.side ? (const float*)y.y2.p : (const float*)nullptr, lw.side ? d.out_scale : 1.f, lw.side ? lw.side->d.out_scale : 0.f,
                           lw.norm1b, (has_ff || !shifted) ? (has_ff ? split_x : more) : 0);
         else if (post)
             launch(lc, "post_norm", 0, ly_post_norm_kernel, dim3(Ti), dim3(nthr), 0, y.x.p, (const float*)y.y.p, (const float*)nullptr, (const float*)lw.norm1b,
-                   has_ff ? (const float*)lw.norm2 : next1, eps, W, plain, has_ff ? split_x : more, y.h.p, hhi, hlo);
+                   has_ff ? (const float*)lw.norm2 : next1, (const float*)lw.ls1, has_ff ? (const float*)nullptr : again, has_ff ? (const float*)nullptr : pstep, eps, W, plain,
+                   has_ff ? split_x : more, y.h.p, hhi, hlo);
         else
             join(lw.side ? (const float*)y.y2.p : (const float*)nullptr, lw.pair_wa, lw.pair_wb, lw.rg1b, (depth && !has_ff) ? li + 1 : -1, lw.dwa,
                  has_ff ? (const float*)lw.norm2 : next1);
         if (!has_ff) continue;
-        sublayer_front(lw, 1);
+        sublayer_front(lw, run, 1);
         const int F = d.ff, act = d.ffn_act, GF = act == FL_ACT_RELU2 ? F : 2 * F;
         if (d.ffn == FL_FFN_DENSE) {
             gemm_tc_or_exact(c, lc, "gemm_ff_in", sub_in, hhi, hlo, lw.w_gu, lw.tm_gu, lw.tc_gu, GF, W, y.gu.p, Ti);
@@ -1339,7 +1419,7 @@ static void enqueue_step(fl_cache& c, LaunchCtx& lc, const StepTab& st, const in
             sum_norm_join(lw.b_down, nullptr, 1.f, 0.f, lw.norm2b, shifted ? 0 : more);
         else if (post)
             launch(lc, "post_norm", 0, ly_post_norm_kernel, dim3(Ti), dim3(nthr), 0, y.x.p, (const float*)y.y.p, (const float*)lw.b_down, (const float*)lw.norm2b,
-                   next1, eps, W, plain, more, y.h.p, hhi, hlo);
+                   next1, (const float*)lw.ls2, again, pstep, eps, W, plain, more, y.h.p, hhi, hlo);
         else
             join(nullptr, nullptr, nullptr, lw.rg2b, depth ? li + 1 : -1, lw.dwa, next1);
     }

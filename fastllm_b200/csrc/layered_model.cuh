@@ -1,10 +1,10 @@
-// Layered decoders (FL_ARCH_NIFUNEX, FL_ARCH_ROFETAR, FL_ARCH_TOZARAX, FL_ARCH_MEDULORN): model / cache objects shared by fl_layered.cu and
-// fl_lib.cu.  A layer = one mixer (gated linear attention | latent attention | grouped-query attention | Mamba-2 | gated delta rule |
+// Layered decoders (FL_ARCH_NIFUNEX, FL_ARCH_ROFETAR, FL_ARCH_TOZARAX, FL_ARCH_MEDULORN, FL_ARCH_LATODRA): model / cache objects shared by
+// fl_layered.cu and fl_lib.cu.  A layer = one mixer (gated linear attention | latent attention | grouped-query attention | Mamba-2 | gated delta rule |
 // lightning attention), or two of them side by side, + an optional feed-forward (dense | MoE), each wrapped by a norm before and
 // after, after only (fl_stack_config.no_pre_norm), before only (no_post_norm), or a norm of the sum of stream and sublayer result
 // (post_sum_norm); optionally a learned position table, an input convolution in front of every sublayer, a token shift in front of
-// every mixer, a gate on every sublayer's contribution and an average over all earlier layers' outputs.  Sizes and constants
-// come from fl_layer_desc / fl_stack_config; nothing is fixed per model.
+// every mixer, a gate on every sublayer's contribution, an average over all earlier layers' outputs, a scale per channel on every
+// sublayer's normed result, and a span of layers that runs several times with the same weights.  Sizes and constants come from fl_layer_desc / fl_stack_config; nothing is fixed per model.
 #pragma once
 #include <cuda.h>
 
@@ -24,7 +24,7 @@ struct LayeredLayerW {
     fl_layer_desc d{};
     float *norm1 = nullptr, *norm1b = nullptr, *norm2 = nullptr, *norm2b = nullptr;     // [W] f32
     // mixer input projections stacked into ONE matrix [n_in, W] (one GEMM per layer):
-    //   GLA:     q | k | v | g | a1        latent attention:  q | dkv   (no dkv rows when kv_from >= 0)
+    //   GLA:     q | k | v | g | a1        latent attention:  q (or dq, with a query latent) | dkv (not when kv_from >= 0) | g (with a gate)
     //   attention:  q | k | v  (no k, v rows when kv_from >= 0)      Mamba-2:  z | x | B | C | dt      delta rule:  q | k | v | g | b | a
     // (rows padded with zeros to a multiple of 8 for the three newer mixers, so that the tensor-core GEMM's tiles fit)
     uint16_t* w_in = nullptr;
@@ -49,10 +49,14 @@ struct LayeredLayerW {
     float* dkv_norm = nullptr;          // [kv_rank]
     uint16_t* uk_t = nullptr;           // [heads][kv_rank, dim]: W_uk per head, transposed (q absorbs it: q~ = W_uk[h]^T q)
     uint16_t* uv = nullptr;             // [heads * vdim, kv_rank]
+    float* dq_norm = nullptr;           // query latent: [q_rank]
+    uint16_t* uq = nullptr;             // query latent: [heads * (dim + rot_dim), q_rank]
+    CUtensorMap tm_uq{};
+    bool tc_uq = false;
     int kv_owner = -1;                  // layer whose cache this layer reads (itself when it projects its own)
-    int kv_index = -1;                  // index of that cache among the model's latent caches
+    int kv_index = -1;                  // index of that cache among the model's paged caches (a looped layer: of its first pass; pass t adds t)
     int rope_index = -1;                // index into the model's distinct rotary tables
-    int gla_index = -1;                 // index among the model's recurrent layers (GLA, Mamba-2, delta rule)
+    int gla_index = -1;                 // index among the model's recurrent states (a looped layer: of its first pass)
     // feed-forward: groups 0..E-1 = experts (or the one dense block), `shared` separate
     uint16_t *w_gu = nullptr, *w_down = nullptr;        // [groups][2 ff, W] (gate rows then up rows), [groups][W, ff]
     uint16_t *s_gu = nullptr, *s_down = nullptr;        // shared expert
@@ -72,9 +76,9 @@ struct LayeredLayerW {
     uint16_t *rg1 = nullptr, *rg2 = nullptr;           // [W, W] gates of the two sublayers' contributions
     float *rg1b = nullptr, *rg2b = nullptr;            // [W]
     float* dwa = nullptr;                              // [layer index + 2] weights of the depth average
+    float *ls1 = nullptr, *ls2 = nullptr;              // [W] scales of the two sublayers' normed results
     CUtensorMap tm_rg1{}, tm_rg2{};
     bool tc_rg1 = false, tc_rg2 = false;
-    int canon_index = -1;               // index among the layers' input-convolution states
 };
 
 struct RopeSpec {                       // one distinct rotary configuration (tables are built per cache: they depend on max_seq)
@@ -88,15 +92,25 @@ struct RopeSpec {                       // one distinct rotary configuration (ta
     }
 };
 
+// One run of a layer: the stack in the order it is computed.  Without a loop every layer runs once.
+struct LayerRun {
+    int layer = 0;
+    int pass = 0;                       // which of the layer's caches / states this run uses
+    bool pass_start = false;            // the first layer of a pass of the loop
+};
+
 struct LayeredModel {
     fl_stack_config cfg{};
     int W = 0, V = 0, L = 0;
     bool f32 = false;                   // compute_dtype == FL_DTYPE_F32
     std::vector<LayeredLayerW> layers;
+    std::vector<LayerRun> runs;
     std::vector<RopeSpec> ropes;
-    std::vector<const LayeredLayerW*> kv_layers, gla_layers;   // mixers that own a paged cache (latent, or keys | values) / a recurrent state
+    std::vector<const LayeredLayerW*> kv_layers, gla_layers;   // mixers that own a paged cache (latent, or keys | values) / a recurrent state,
+                                                               // once per pass
     DevBuf<uint8_t> slab;
-    uint16_t *embed = nullptr, *head = nullptr, *pos = nullptr;    // pos: [max_positions, W] learned position vectors (or nullptr)
+    float *embed_norm = nullptr, *loop_step = nullptr;             // [W]; [loop_times, W]
+    uint16_t *embed = nullptr, *head = nullptr, *pos = nullptr;    // head: the same table as embed when tied; pos: [max_positions, W] learned position vectors (or nullptr)
     float* final_norm = nullptr;
     CUtensorMap tm_head{};
     bool tc_head = false;
@@ -106,7 +120,7 @@ struct LayeredModel {
     bool finalized = false;
     uint64_t weight_bytes = 0;
     // widest sizes over the layers (workspace planning)
-    int max_in = 0, max_hv = 0, max_hd = 0, max_hc = 0, max_ff = 0, max_top = 0, max_experts = 0, max_cv = 0, max_heads = 0, max_av = 0;    // max_av: widest value head of a grouped-query attention layer
+    int max_in = 0, max_hv = 0, max_hd = 0, max_hc = 0, max_ff = 0, max_top = 0, max_experts = 0, max_cv = 0, max_heads = 0, max_av = 0, max_qr = 0, max_q = 0;    // max_av: widest value head of a grouped-query attention layer; max_qr / max_q: widest query latent / queries expanded from one
     std::mutex mu;
 };
 
@@ -118,8 +132,8 @@ struct LayeredCache {
     std::vector<DevBuf<uint8_t>> kv_store;
     std::vector<DevBuf<float>> gla_state;          // per recurrent layer: [slots][heads][dim | state][vdim]
     std::vector<DevBuf<float>> conv_state;         // per recurrent layer: [slots][taps - 1][conv_ch] (empty without a convolution)
-    std::vector<DevBuf<float>> canon_state;        // input convolutions: per layer [2 sublayers][slots][taps - 1][W]
-    std::vector<DevBuf<float>> shift_state;        // token shift: per layer [slots][W], the mixer input of the slot's last position
+    std::vector<DevBuf<float>> canon_state;        // input convolutions: per layer run [2 sublayers][slots][taps - 1][W]
+    std::vector<DevBuf<float>> shift_state;        // token shift: per layer run [slots][W], the mixer input of the slot's last position
     std::vector<DevBuf<float>> rope_cos, rope_sin; // per RopeSpec: [max_seq][dims/2]
     DevBuf<int> page_table;             // [slots][pages_per_slot]
     DevBuf<int> step_tab;               // per-step integer tables (see StepTab in fl_layered.cu)
@@ -129,12 +143,14 @@ struct LayeredCache {
     size_t rows = 0, want_cap = 0;
     DevBuf<float> x, h, y, proj, la, u, go, qa, ol, gu, act, eo, sh_gu, sh_act, sh_o, route_w, sgate, hf, logits;
     DevBuf<float> hc, gz, y2, xs;       // convolved sublayer input; gate pre-activations; the second mixer's projected output;
-                                        // xs [L + 1][rows][W]: the embedding output and every layer's own result (depth average)
+                                        // xs [L + 1][rows][W]: the embedding output and every layer's own result (depth average); a
+                                        // loop that adds the embedding output again keeps just that, [rows][W]
+    DevBuf<float> cq, qx;               // query latents [rows, max_qr], the queries expanded from them [rows, max_q]
     DevBuf<float> cv, rs;               // recurrent mixers: convolved + activated columns [rows, max_cv]; per-head (decay, strength) [rows, 2 heads]
     DevBuf<int> route_sel, pair_row, pair_of, grp_off;
     PinnedBuf<float> h_logits;
     // serving precision: hi/lo halves of the activations that feed tensor-core GEMMs, and the split-K slices of their outputs
-    DevBuf<uint16_t> h_hi, h_lo, u_hi, u_lo, act_hi, act_lo, hf_hi, hf_lo;
+    DevBuf<uint16_t> h_hi, h_lo, cq_hi, cq_lo, u_hi, u_lo, act_hi, act_lo, hf_hi, hf_lo;
     DevBuf<float> gemm_out;
     DevBuf<uint16_t> gx_hi, gx_lo, ga_hi, ga_lo;        // grouped expert GEMMs: gathered inputs / activations, [experts * cap] rows
     DevBuf<int> grp_cnt;

@@ -110,23 +110,31 @@ __device__ __forceinline__ float norm_scale(const float* __restrict__ w, int c, 
 
 // x[row] = embed[tok[row]] (times escale when that is not 0) (+ pos_tab[row_pos[row]], a learned position vector);  h[row] = x / sqrt(mean x^2 + eps) * scale(w).
 // nw == nullptr (the first sublayer reads the stream itself): h is not written and the hi | lo halves are those of x.
-// x0 (optional): a second copy of x, the first entry of the depth average's history.
+// en (optional): the embedding row is RMS-normed first, scale(en).  x0 (optional): a second copy of x, the first entry of the depth
+// average's history or what a loop adds again; step (optional): a vector added to x behind that copy (a loop that starts with layer 0).
 static __global__ void ly_embed_norm_kernel(const uint16_t* __restrict__ embed, const int* __restrict__ tok, int W, const float* __restrict__ nw,
                                             float eps, int plain, const uint16_t* __restrict__ pos_tab, const int* __restrict__ row_pos,
-                                            float escale, float* __restrict__ x, float* __restrict__ x0, float* __restrict__ h,
-                                            uint16_t* __restrict__ hhi, uint16_t* __restrict__ hlo) {
+                                            float escale, const float* __restrict__ en, const float* __restrict__ step, float* __restrict__ x,
+                                            float* __restrict__ x0, float* __restrict__ h, uint16_t* __restrict__ hhi, uint16_t* __restrict__ hlo) {
     __shared__ float red[33];
     const int row = blockIdx.x;
     const uint16_t* e = embed + (size_t)tok[row] * W;
     const uint16_t* pe = pos_tab ? pos_tab + (size_t)row_pos[row] * W : nullptr;
     float* xr = x + (size_t)row * W;
-    float ss = 0.f;
+    float ss = 0.f, er = 1.f;
+    if (en != nullptr) {
+        float es = 0.f;
+        for (int c = threadIdx.x; c < W; c += blockDim.x) { const float v = __uint_as_float((uint32_t)e[c] << 16); es += v * v; }
+        er = 1.f / sqrtf(block_sum(es, red) / (float)W + eps);
+    }
     for (int c = threadIdx.x; c < W; c += blockDim.x) {
         float v = __uint_as_float((uint32_t)e[c] << 16);
+        if (en != nullptr) v *= er * norm_scale(en, c, plain);
         if (escale != 0.f) v *= escale;
         if (pe) v += __uint_as_float((uint32_t)pe[c] << 16);
-        xr[c] = v;
         if (x0) x0[(size_t)row * W + c] = v;
+        if (step) v += step[c];
+        xr[c] = v;
         ss += v * v;
         if (nw == nullptr) split_store(hhi, hlo, (size_t)row * W + c, v);
     }
@@ -141,10 +149,12 @@ static __global__ void ly_embed_norm_kernel(const uint16_t* __restrict__ embed, 
 }
 
 // x[row] += norm(y[row] + yb; wb);  then, if wnext, h[row] = norm(x[row]; wnext); else, if split_x, the hi | lo halves of x[row]
-// itself (the next sublayer reads the stream un-normed).  yb: optional bias of the projection that produced y.
+// itself (the next sublayer reads the stream un-normed).  yb: optional bias of the projection that produced y.  ls (optional) [W] scales
+// the normed result per channel.  Between two passes of a loop the stream then gains x0[row] (optional: the embedding output once
+// more) and step (optional [W]: the next pass's vector), in this order, before the next norm.
 static __global__ void ly_post_norm_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ yb, const float* __restrict__ wb,
-                                           const float* __restrict__ wnext, float eps, int W, int plain, int split_x, float* __restrict__ h,
-                                           uint16_t* __restrict__ hhi, uint16_t* __restrict__ hlo) {
+                                           const float* __restrict__ wnext, const float* __restrict__ ls, const float* __restrict__ x0, const float* __restrict__ step,
+                                           float eps, int W, int plain, int split_x, float* __restrict__ h, uint16_t* __restrict__ hhi, uint16_t* __restrict__ hlo) {
     __shared__ float red[33];
     const int row = blockIdx.x;
     const float* yr = y + (size_t)row * W;
@@ -157,7 +167,11 @@ static __global__ void ly_post_norm_kernel(float* __restrict__ x, const float* _
     const float r = 1.f / sqrtf(block_sum(ss, red) / (float)W + eps);
     float s2 = 0.f;
     for (int c = threadIdx.x; c < W; c += blockDim.x) {
-        const float v = xr[c] + (yr[c] + (yb ? yb[c] : 0.f)) * r * norm_scale(wb, c, plain);
+        float d = (yr[c] + (yb ? yb[c] : 0.f)) * r * norm_scale(wb, c, plain);
+        if (ls) d *= ls[c];
+        float v = xr[c] + d;
+        if (x0) v += x0[(size_t)row * W + c];
+        if (step) v += step[c];
         xr[c] = v;
         s2 += v * v;
         if (wnext == nullptr && split_x) split_store(hhi, hlo, (size_t)row * W + c, v);
@@ -505,6 +519,21 @@ static __global__ void ly_gla_out_kernel(const float* __restrict__ o, const floa
 }
 
 // ---- latent attention ------------------------------------------------------------------------------------------------------
+// turns pair i % half of head i / half: channels D + 2 (i % half) and the next of the head's D + R query channels
+__device__ __forceinline__ void turn_pair(float* q0, int D, int R, int half, int i, const float* cs, const float* sn) {
+    const int hd = i / half, pi = i % half;
+    float* q = q0 + (size_t)hd * (D + R) + D + 2 * pi;
+    const float u = q[0], v = q[1];
+    q[0] = u * cs[pi] - v * sn[pi];
+    q[1] = v * cs[pi] + u * sn[pi];
+}
+// The rotated parts of a row's queries [H][D + R] (expanded from a query latent) turn in place.
+static __global__ void ly_rotate_q_kernel(float* __restrict__ q, int ldq, const int* __restrict__ row_pos, const float* __restrict__ cosb,
+                                          const float* __restrict__ sinb, int H, int D, int R, int rdims) {
+    const int half = rdims / 2;
+    const size_t at = (size_t)row_pos[blockIdx.x] * half;
+    for (int i = threadIdx.x; i < H * half; i += blockDim.x) turn_pair(q + (size_t)blockIdx.x * ldq, D, R, half, i, cosb + at, sinb + at);
+}
 struct LatentAppendArgs {
     float* proj; int ldp, off_q, off_dkv;       // off_dkv < 0: the layer reads another layer's cache (queries are still rotated)
     const float* dkv_norm; float eps;
@@ -513,9 +542,11 @@ struct LatentAppendArgs {
     const int *row_seq, *row_pos, *seq_slot;
     const float *cosb, *sinb;                    // [max_seq][rdims / 2], already multiplied by the YaRN magnitude
     int H, D, R, C, rdims;
+    int off_dq, Q; const float* dq_norm;         // Q > 0: columns off_dq .. of proj are a query latent instead of queries
+    float* cq; uint16_t *cqhi, *cqlo;            // [T, Q] the normed query latent and its hi | lo halves
 };
 // Per row: the latent (RMS-normed, plain weight) and the rotated shared key part go into the row's cache page; the rotated part of
-// every head's query is turned in place.  Pairs (2i, 2i+1) of the first rdims channels turn by pos * f_i; the rest pass through.
+// every head's query is turned in place (with a query latent: the latent is normed instead, the queries do not exist yet).  Pairs (2i, 2i+1) of the first rdims channels turn by pos * f_i; the rest pass through.
 template <typename CT>
 static __global__ void ly_latent_append_kernel(LatentAppendArgs a) {
     __shared__ float red[33];
@@ -523,12 +554,18 @@ static __global__ void ly_latent_append_kernel(LatentAppendArgs a) {
     float* pr = a.proj + (size_t)row * a.ldp;
     const float* cs = a.cosb + (size_t)pos * (a.rdims / 2);
     const float* sn = a.sinb + (size_t)pos * (a.rdims / 2);
-    for (int i = threadIdx.x; i < a.H * (a.rdims / 2); i += blockDim.x) {
-        const int hd = i / (a.rdims / 2), pi = i % (a.rdims / 2);
-        float* q = pr + a.off_q + hd * (a.D + a.R) + a.D + 2 * pi;
-        const float u = q[0], v = q[1];
-        q[0] = u * cs[pi] - v * sn[pi];
-        q[1] = v * cs[pi] + u * sn[pi];
+    if (a.Q > 0) {
+        const float* dq = pr + a.off_dq;
+        float sq = 0.f;
+        for (int c = threadIdx.x; c < a.Q; c += blockDim.x) sq += dq[c] * dq[c];
+        const float rq = 1.f / sqrtf(block_sum(sq, red) / (float)a.Q + a.eps);
+        for (int c = threadIdx.x; c < a.Q; c += blockDim.x) {
+            const float v = dq[c] * rq * a.dq_norm[c];
+            a.cq[(size_t)row * a.Q + c] = v;
+            split_store(a.cqhi, a.cqlo, (size_t)row * a.Q + c, v);
+        }
+    } else {
+        for (int i = threadIdx.x; i < a.H * (a.rdims / 2); i += blockDim.x) turn_pair(pr + a.off_q, a.D, a.R, a.rdims / 2, i, cs, sn);
     }
     if (a.off_dkv < 0) return;
     const int slot = a.seq_slot[a.row_seq[row]];
@@ -561,6 +598,8 @@ struct LatentAttnArgs {
     int H, D, R, C, window;
     float scale;
     int row_base;               // first row of this launch (blockIdx.x counts from it)
+    int sink;                   // != 0: the denominator gets exp(sinkv[head]) more (exp(0) when sinkv is nullptr)
+    const float* sinkv;         // [H] or nullptr
 };
 // CPL consecutive cache elements starting at channel c0 of a key row, as f32; channels >= C read as zero.  16-byte loads when the
 // chunk is whole, inside the latent and aligned; single elements otherwise.
@@ -594,7 +633,7 @@ __device__ __forceinline__ void load_chunk(const uint16_t* kp, int c0, int C, fl
 
 constexpr int kLatWarps = 8;
 // One block per (row, head).  score_j = (q~ . c_j + q_rot . k_rot_j) * scale over the keys j the window admits (0 <= pos - j <
-// window), softmax in f32, out = sum_j p_j c_j.  Warp w of the eight folds keys j0 + w, j0 + w + 8, ... into an online softmax (lanes own
+// window), softmax in f32 with the optional sink, out = sum_j p_j c_j.  Warp w of the eight folds keys j0 + w, j0 + w + 8, ... into an online softmax (lanes own
 // channels); the eight partial results are merged at the end.  Which warp takes which key depends on the position alone.
 template <typename CT, int CPL>
 static __global__ void __launch_bounds__(kLatWarps * 32) ly_latent_attn_kernel(LatentAttnArgs a) {
@@ -654,10 +693,11 @@ static __global__ void __launch_bounds__(kLatWarps * 32) ly_latent_attn_kernel(L
     for (int i = 0; i < CPL; ++i) { const int c = lane * CPL + i; if (c < C) sacc[wid * C + c] = acc[i]; }
     if (lane == 0) { sml[2 * wid] = m; sml[2 * wid + 1] = l; }
     __syncthreads();
-    float M = -INFINITY;
+    const float sv = a.sinkv ? a.sinkv[hd] : 0.f;
+    float M = a.sink ? sv : -INFINITY;
 #pragma unroll
     for (int w = 0; w < kLatWarps; ++w) M = fmaxf(M, sml[2 * w]);
-    float f[kLatWarps], Lsum = 0.f;
+    float f[kLatWarps], Lsum = a.sink ? expf(sv - M) : 0.f;
 #pragma unroll
     for (int w = 0; w < kLatWarps; ++w) { f[w] = expf(sml[2 * w] - M); Lsum += sml[2 * w + 1] * f[w]; }
     const float inv = 1.f / Lsum;
@@ -772,6 +812,18 @@ static __global__ void ly_attn_softmax_kernel(const float* __restrict__ S, const
         else if (c >= b_lo && c < c_hi && c >= n_first && vis(c)) i = na + (c - b_lo);
         if (i >= 0) p = (kept ? srow[i] : expf(score(c) - m)) * inv;
         split_store(phi, plo, r * nkp + c, p);
+    }
+}
+
+// u[row, c] *= sigmoid(proj[row, off_g + c]): a gate on the concatenated heads, with the hi | lo halves of the product
+static __global__ void ly_out_gate_kernel(float* __restrict__ u, const float* __restrict__ proj, int ldp, int off_g, int n, int T,
+                                          uint16_t* __restrict__ uhi, uint16_t* __restrict__ ulo) {
+    const size_t total = (size_t)T * n;
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+        const size_t row = i / n;
+        const float v = u[i] * sigmoidf_(proj[row * ldp + off_g + (i - row * n)]);
+        u[i] = v;
+        split_store(uhi, ulo, i, v);
     }
 }
 

@@ -833,10 +833,59 @@ class MedulornWithConfig(_LayeredBase):
                 yield f"l{i}.mix.right.decay", np.asarray(l["mixer"]["right"]["decay"], dtype=np.float32)
 
 
+def _query_latent_desc(d, m: dict):
+    """the fields both latent attentions of the Latodra decoder share: sizes, the scale, a query that goes through its own latent"""
+    d.mixer, d.kv_from = _lib.FL_MIXER["latent_attention"], -1
+    d.heads, d.dim, d.vdim = int(m["heads"]), int(m["dim"]), int(m["vdim"])
+    d.kv_rank, d.q_rank = int(m["kv_rank"]), int(m["q_rank"])
+    d.scale = float(m["scale"])
+
+
+def latodra_layer_descs(config: dict):
+    """config.json of the Latodra decoder -> ctypes array of FlLayerDesc (every size and constant comes from the file)."""
+    layers = config["layers"]
+    arr = (_lib.FlLayerDesc * len(layers))()
+    for i, l in enumerate(layers):
+        d, m, kind = arr[i], l["mixer"], l["type"]
+        _query_latent_desc(d, m)
+        if kind == "latent_attention":          # a rotated shared key part, a learned sink per head
+            d.rot_dim, d.sink = int(m["rot_dim"]), 2
+            _rotary_desc(d, m.get("rot") or {}, d.rot_dim)
+        elif kind == "latent_attention_2":      # no positions, gated heads
+            d.out_gate = 1
+        else:
+            raise FastllmError(-1, f"layer {i}: unknown mixer type {kind!r}")
+        _ffn_desc(d, i, l.get("mlp"), act="gelu_tanh")
+        if d.ffn == _lib.FL_FFN["moe"]:
+            raise FastllmError(-1, f"layer {i}: this design has dense feed-forwards only")
+    return arr
+
+
+class LatodraWithConfig(_LayeredBase):
+    """The Latodra decoder (no reference path): latent attention with a query latent, either with a YaRN-rotated shared key part and
+    a learned sink per head or without positions and with gated heads; a tanh-gelu gated feed-forward; norms (plain weight) before
+    and after every sublayer and a scale per channel on what joins the stream; a span of layers that runs several times with the
+    same weights, each pass with its own cache; a normed embedding whose table is the output projection too."""
+    arch, family, architectures = "latodra", "Latodra", ("Latodra",)
+    norm_plain = True
+
+    @classmethod
+    def stack_options(cls, config: dict, sc) -> None:
+        sc.embed_norm, sc.layer_scale, sc.tied_head = 1, 1, 1
+        loop = config.get("loop")
+        if loop:
+            sc.loop_start, sc.loop_stop, sc.loop_times = int(loop["start"]), int(loop["stop"]), int(loop["times"])
+            sc.loop_reinject, sc.loop_step = 1, 1
+
+    @classmethod
+    def layer_descs(cls, config: dict, tensor_shapes: dict):
+        return latodra_layer_descs(config)
+
+
 # every adapter, in the order the registry tries them (model_registry.rs:169-182 keeps the same kind of list)
 def registered_models():
     return (LlamaWithConfig, MistralWithConfig, QwenWithConfig, MixtralWithConfig, NifunexWithConfig, RofetarWithConfig, TozaraxWithConfig,
-            MedulornWithConfig)
+            MedulornWithConfig, LatodraWithConfig)
 
 
 def model_class_for(config: dict):

@@ -75,10 +75,14 @@ typedef enum fl_arch {
     FL_ARCH_TOZARAX = 7,   /* layered decoder (no reference path): learned positions; pre-normed sublayers that read their input through a
                               short causal convolution, gate their contribution and average over all earlier layers' outputs; two mixers
                               side by side (windowed attention without rotation | gated delta rule); sigmoid-routed squared-relu experts */
-    FL_ARCH_MEDULORN = 8   /* layered decoder (no reference path): x <- norm(alpha x + sub(x)) with one number as the norm's weight
+    FL_ARCH_MEDULORN = 8,  /* layered decoder (no reference path): x <- norm(alpha x + sub(x)) with one number as the norm's weight
                               (fl_stack_config.post_sum_norm); mixers read x through a token shift; chunk-masked attention with biased
                               projections | sliding-window attention with kept first tokens and a learned sink beside lightning attention;
                               relu-gated dense feed-forward or clamped-swish experts with a biased router; scaled embedding, capped logits */
+    FL_ARCH_LATODRA = 9    /* layered decoder (no reference path): latent attentions whose queries go through a latent of their own (one kind
+                              with a rotated shared key part and a learned softmax sink, one without positions and with a sigmoid gate on
+                              the heads); a scale per channel on every sublayer's normed result; a span of layers that runs several times
+                              with the same weights; a normed embedding that is also the output projection */
 } fl_arch;
 
 typedef enum fl_dtype { FL_DTYPE_F32 = 0, FL_DTYPE_BF16 = 1, FL_DTYPE_F16 = 2 } fl_dtype;
@@ -158,7 +162,10 @@ typedef struct fl_config {
  * rot_scaling = FL_ROT_SCALE_BANDS: frequencies whose wavelength is below yarn_original / yarn_fast stay, above yarn_original /
  * yarn_slow are divided by yarn_factor, between the two blend linearly in yarn_original / wavelength; cos and sin keep magnitude 1.
  * Feed-forward (ffn_act = FL_ACT_RELU): y = W_down (relu(W_gate h) * (W_up h)).  router_bias: "mlp.router.b" is added to the router
- * logits.  shared_plain: the shared expert's output is added as it is (no "mlp.shared.sg"). */
+ * logits.  shared_plain: the shared expert's output is added as it is (no "mlp.shared.sg").
+ * Latent attention with q_rank > 0: q = W_uq c_q, c_q = RMS norm of W_dq h (tensors "dq" [q_rank, width], "dq.norm" [q_rank], "uq"
+ * [heads * (dim + rot_dim), q_rank] instead of "q").  sink as for FL_MIXER_ATTN.  rot_dim = 0: no rotated part, only the latent is
+ * cached.  out_gate: the concatenated heads are multiplied by sigmoid(W_g h) before W_o (tensor "g" [heads * vdim, width]). */
 typedef enum fl_mixer_kind { FL_MIXER_GLA = 0, FL_MIXER_LATENT_ATTN = 1, FL_MIXER_ATTN = 2, FL_MIXER_MAMBA2 = 3, FL_MIXER_DELTA = 4, FL_MIXER_LIGHTNING = 5 } fl_mixer_kind;
 typedef enum fl_ffn_kind { FL_FFN_NONE = 0, FL_FFN_DENSE = 1, FL_FFN_MOE = 2 } fl_ffn_kind;
 typedef enum fl_ffn_act { FL_ACT_SWISH_CLAMP = 0, FL_ACT_GELU_TANH = 1, FL_ACT_RELU2 = 2, FL_ACT_RELU = 3 } fl_ffn_act;
@@ -188,7 +195,7 @@ typedef struct fl_layer_desc {
     int32_t conv;                      /* Mamba-2 / delta rule: taps of the short causal convolution */
     int32_t state, groups, norm_groups;/* Mamba-2: state size per head, B / C groups, parts of the gated output norm */
     float softcap;                     /* attention: score <- softcap * tanh(score / softcap); 0 = none */
-    int32_t sink;                      /* attention: 1 = one is added to the softmax denominator; 2 = exp(sink_h), a learned number per head */
+    int32_t sink;                      /* attention, latent attention: 1 = one is added to the softmax denominator; 2 = exp(sink_h), a learned number per head */
     int32_t rot_halves;                /* attention: 1 = rotary pairs are (i, i + rot_dims / 2), 0 = (2i, 2i + 1) */
     int32_t ffn_act, ffn_bias;         /* feed-forward: fl_ffn_act; dense: 1 = gate / up / down carry biases */
     int32_t no_qk_norm;                /* attention: 1 = queries and keys are used as projected (no per-head norm, no norm tensors) */
@@ -205,11 +212,13 @@ typedef struct fl_layer_desc {
     int32_t pair_sum;                  /* beside: 1 = the layer's mixer output is the out_scale-weighted sum of the two mixers' outputs */
     int32_t router_bias;               /* MoE, FL_ROUTER_SOFTMAX: 1 = the router logits carry a bias */
     int32_t shared_plain;              /* MoE: 1 = the shared expert is not gated */
+    int32_t q_rank;                    /* latent attention: > 0 = queries go through a normed latent of this width */
+    int32_t out_gate;                  /* latent attention: 1 = the concatenated heads are gated by sigmoid(W_g h) */
     int32_t reserved[2];
 } fl_layer_desc;
 
 typedef struct fl_stack_config {
-    int32_t arch;                      /* FL_ARCH_NIFUNEX */
+    int32_t arch;                      /* a layered fl_arch */
     int32_t vocab, width, n_layers;
     float norm_eps;
     int32_t compute_dtype;             /* FL_DTYPE_BF16: bf16 weights on the tensor-core path, bf16 cache; FL_DTYPE_F32: every product
@@ -234,6 +243,14 @@ typedef struct fl_stack_config {
     float logit_softcap;               /* > 0: logits <- cap tanh(logits / cap) */
     int32_t token_shift;               /* 1: a mixer reads h + (h_prev - h) * shift, h_prev = the previous token's mixer input of the same layer
                                           before this replacement, zeros at position 0 ("l<i>.shift" [width]); h_prev is kept per slot and layer */
+    int32_t embed_norm;                /* 1: the embedding row is RMS-normed with weight "embed.norm" [width] before it becomes the stream */
+    int32_t layer_scale;               /* 1: a sublayer's normed result is multiplied per channel by "l<i>.ls1" (mixer) / "l<i>.ls2" (feed-forward)
+                                          [width] (needs norms before and after the sublayers) */
+    int32_t tied_head;                 /* 1: the output projection is the embedding table (no "head" tensor) */
+    int32_t loop_start, loop_stop;     /* loop_times > 0: layers loop_start .. loop_stop - 1 run loop_times times in a row with the same weights, */
+    int32_t loop_times;                /*   each pass with its own cache / state; 0 = no loop */
+    int32_t loop_reinject;             /* 1: the embedding output is added to the stream before every pass but the first */
+    int32_t loop_step;                 /* 1: row t of "loop.step" [loop_times, width] is added to the stream before pass t (after loop_reinject's sum) */
     int32_t reserved[3];
 } fl_stack_config;
 

@@ -64,6 +64,10 @@ WORKLOADS = {
                             "shared expert) beside Tozarax (attention beside a delta rule in every layer, experts) and Rofetar (attention with q/k "
                             "norm, rotation and sink / delta rule alternating, dense feed-forward) at equal width / layers: 2048-token prefill and "
                             "batch-8 decode at 2k context, random weights"),
+    "latodra_vs_nifunex": ("latodra", 8, 2048, "layered decoder (Latodra: latent attention with query latents, rotated with a learned sink / without "
+                           "positions and gated, layer scales, looped middle layers, dense gelu feed-forward) beside Nifunex with latent attention in "
+                           "every layer and a dense feed-forward at equal width / ff / layers: 2048-token prefill and batch-8 decode at 2k context, "
+                           "random weights"),
 }
 QWEN_PREFILL_TFLOP_4K = 56.83         # 53.46 linear + 3.37 causal attention
 MINILM_FLOP_PER_TOKEN = 22.41e6      # 2 x 10.617 M linear + 4 T H 6 attention at T = 128
@@ -357,7 +361,8 @@ def run_reference(args, rank):
     if rank != 0:
         return
     arch, batch, ctx, desc = WORKLOADS[args.workload]
-    if args.workload in ("mixtral8x7b_b32", "qwen25_7b_prefill4k", "nifunex_vs_mixtral", "rofetar_vs_nifunex", "tozarax_vs_rofetar", "medulorn_vs_tozarax"):
+    if args.workload in ("mixtral8x7b_b32", "qwen25_7b_prefill4k", "nifunex_vs_mixtral", "rofetar_vs_nifunex", "tozarax_vs_rofetar", "medulorn_vs_tozarax",
+                         "latodra_vs_nifunex"):
         print(json.dumps({"impl": "reference", "unavailable": f"no CPU leg for workload {args.workload}: the reference does not wire Mixtral "
                           "and a 4096-token f32 prefill of a 7B model does not fit a bounded CPU sample; the decode workloads carry the CPU baseline"}),
               flush=True)
@@ -894,22 +899,11 @@ def run_layered_compare(args, local_rank):
     """--workload nifunex_vs_mixtral (one GPU): the layered decoder and Mixtral at the same width / experts / layer count, random
     weights -- one 2048-token prefill and batch-8 decode steps at a 2k context, through the public calls (host ids in, logits
     out), with the per-kernel CUDA-event profile of one call of each kind."""
-    import torch
     from fastllm_b200 import models
     batch, T, steps, warm = 8, 2048, max(4, min(args.steps, 32)), 3
     sizes = [("w1024", 1024, 2816, 4), ("w2048", 2048, 5632, 4), ("w4096", 4096, 14336, 4)]
     vocab, window = 32000, 1024
     results = {}
-
-    def timed(fn, n):
-        for _ in range(warm):
-            fn()
-        torch.cuda.synchronize()
-        t0 = time.perf_counter()
-        for _ in range(n):
-            fn()
-        torch.cuda.synchronize()
-        return (time.perf_counter() - t0) / n
 
     with ClockSampler(local_rank) as clk:
         t_wall0 = time.time()
@@ -924,7 +918,7 @@ def run_layered_compare(args, local_rank):
             def prefill():
                 cache.slot_reset(0)
                 cache.forward_ragged([0], [ids], None)
-            dt_p = timed(prefill, max(2, steps // 4))
+            dt_p = _timed(prefill, max(2, steps // 4), warm)
             models.prof_begin(); prefill(); prof_p = models.prof_end()
             for s in range(1, batch):
                 cache.forward_ragged([s], [ids], None)
@@ -932,7 +926,7 @@ def run_layered_compare(args, local_rank):
 
             def decode():
                 cache.forward_ragged(slots, [[7 + s] for s in slots], None)
-            dt_d = timed(decode, steps)
+            dt_d = _timed(decode, steps, warm)
             models.prof_begin(); decode(); prof_d = models.prof_end()
             rec["nifunex"] = {"prefill_tok_s": T / dt_p, "prefill_ms": dt_p * 1e3, "decode_tok_s": batch / dt_d, "decode_ms_per_step": dt_d * 1e3,
                               "weight_bytes": model.dev.streamed_bytes(), "prefill_kernels": _profile_table(prof_p), "decode_kernels": _profile_table(prof_d)}
@@ -946,7 +940,7 @@ def run_layered_compare(args, local_rank):
             def prefill_m():
                 mc.reset()
                 mc.forward_slots([0], ids2, [0])
-            dt_pm = timed(prefill_m, max(2, steps // 4))
+            dt_pm = _timed(prefill_m, max(2, steps // 4), warm)
             models.prof_begin(); prefill_m(); prof_pm = models.prof_end()
             for s in range(1, batch):
                 mc.forward_slots([s], ids2, [0])
@@ -956,7 +950,7 @@ def run_layered_compare(args, local_rank):
                 mc.forward_slots(slots, np.asarray([[7 + s] for s in slots], dtype=np.uint32), pos)
                 for i in range(batch):
                     pos[i] += 1
-            dt_dm = timed(decode_m, steps)
+            dt_dm = _timed(decode_m, steps, warm)
             models.prof_begin(); decode_m(); prof_dm = models.prof_end()
             rec["mixtral"] = {"prefill_tok_s": T / dt_pm, "prefill_ms": dt_pm * 1e3, "decode_tok_s": batch / dt_dm, "decode_ms_per_step": dt_dm * 1e3,
                               "weight_bytes": mx.dev.streamed_bytes(), "prefill_kernels": _profile_table(prof_pm), "decode_kernels": _profile_table(prof_dm)}
@@ -972,6 +966,45 @@ def run_layered_compare(args, local_rank):
                                  "(host ids in, f32 logits out) with a device synchronise on both sides; per-kernel figures are CUDA events",
                                  "l2": "weights of a step exceed L2 at every size"},
                       "clocks": clk.summary(t_wall0, t_wall1), "sizes": results}), flush=True)
+
+
+def _timed(fn, n, warm):
+    """wall-clock seconds per call of fn, a device synchronise on both sides"""
+    import torch
+    for _ in range(warm):
+        fn()
+    torch.cuda.synchronize()
+    t0 = time.perf_counter()
+    for _ in range(n):
+        fn()
+    torch.cuda.synchronize()
+    return (time.perf_counter() - t0) / n
+
+
+def _layered_record(cls, cfg, local_rank, batch, T, steps, warm, vocab, **hints):
+    """one layered model with random weights: a T-token prefill and batch decode steps at a T-token context through the public calls (host
+    ids in, logits out; wall clock with a device synchronise on both sides) and the per-kernel CUDA-event profile of one call of each"""
+    from fastllm_b200 import models
+
+    model, _ = cls.initialize_model(cfg, None, "bf16", local_rank, random_seed=0, std=0.02, **hints)
+    cache = model.new_device_cache(max_batch=batch, max_seq=T + 64, pool_tokens=batch * (T + 64))
+    ids = (np.arange(T, dtype=np.uint64) * 7919 % (vocab - 5) + 3).astype(np.uint32)
+
+    def prefill():
+        cache.slot_reset(0)
+        cache.forward_ragged([0], [ids], None)
+    dt_p = _timed(prefill, max(2, steps // 4), warm)
+    models.prof_begin(); prefill(); prof_p = models.prof_end()
+    for s in range(1, batch):
+        cache.forward_ragged([s], [ids], None)
+    slots = list(range(batch))
+
+    def decode():
+        cache.forward_ragged(slots, [[7 + s] for s in slots], None)
+    dt_d = _timed(decode, steps, warm)
+    models.prof_begin(); decode(); prof_d = models.prof_end()
+    return {"prefill_tok_s": T / dt_p, "prefill_ms": dt_p * 1e3, "decode_tok_s": batch / dt_d, "decode_ms_per_step": dt_d * 1e3,
+            "weight_bytes": model.dev.streamed_bytes(), "prefill_kernels": _profile_table(prof_p), "decode_kernels": _profile_table(prof_d)}
 
 
 def _rofetar_config(width, ff, layers, vocab):
@@ -1009,43 +1042,14 @@ def run_rofetar_compare(args, local_rank):
     """--workload rofetar_vs_nifunex (one GPU): Rofetar, Nifunex (dense feed-forward) and Mistral at the same width / ff / layer count,
     random weights -- one 2048-token prefill and batch-8 decode steps at a 2k context, through the public calls (host ids in,
     logits out), with the per-kernel CUDA-event profile of one call of each kind."""
-    import torch
     from fastllm_b200 import models
     batch, T, steps, warm = 8, 2048, max(4, min(args.steps, 32)), 3
     sizes = [("w1024", 1024, 2816, 4), ("w2048", 2048, 5632, 4), ("w4096", 4096, 14336, 4)]
     vocab = 32000
     results = {}
 
-    def timed(fn, n):
-        for _ in range(warm):
-            fn()
-        torch.cuda.synchronize()
-        t0 = time.perf_counter()
-        for _ in range(n):
-            fn()
-        torch.cuda.synchronize()
-        return (time.perf_counter() - t0) / n
-
     def layered(cls, cfg, **hints):
-        model, _ = cls.initialize_model(cfg, None, "bf16", local_rank, random_seed=0, std=0.02, **hints)
-        cache = model.new_device_cache(max_batch=batch, max_seq=T + 64, pool_tokens=batch * (T + 64))
-        ids = (np.arange(T, dtype=np.uint64) * 7919 % (vocab - 5) + 3).astype(np.uint32)
-
-        def prefill():
-            cache.slot_reset(0)
-            cache.forward_ragged([0], [ids], None)
-        dt_p = timed(prefill, max(2, steps // 4))
-        models.prof_begin(); prefill(); prof_p = models.prof_end()
-        for s in range(1, batch):
-            cache.forward_ragged([s], [ids], None)
-        slots = list(range(batch))
-
-        def decode():
-            cache.forward_ragged(slots, [[7 + s] for s in slots], None)
-        dt_d = timed(decode, steps)
-        models.prof_begin(); decode(); prof_d = models.prof_end()
-        return {"prefill_tok_s": T / dt_p, "prefill_ms": dt_p * 1e3, "decode_tok_s": batch / dt_d, "decode_ms_per_step": dt_d * 1e3,
-                "weight_bytes": model.dev.streamed_bytes(), "prefill_kernels": _profile_table(prof_p), "decode_kernels": _profile_table(prof_d)}
+        return _layered_record(cls, cfg, local_rank, batch, T, steps, warm, vocab, **hints)
 
     with ClockSampler(local_rank) as clk:
         t_wall0 = time.time()
@@ -1062,7 +1066,7 @@ def run_rofetar_compare(args, local_rank):
             def prefill_m():
                 mc.reset()
                 mc.forward_slots([0], ids2, [0])
-            dt_pm = timed(prefill_m, max(2, steps // 4))
+            dt_pm = _timed(prefill_m, max(2, steps // 4), warm)
             models.prof_begin(); prefill_m(); prof_pm = models.prof_end()
             for s in range(1, batch):
                 mc.forward_slots([s], ids2, [0])
@@ -1072,7 +1076,7 @@ def run_rofetar_compare(args, local_rank):
                 mc.forward_slots(slots, np.asarray([[7 + s] for s in slots], dtype=np.uint32), pos)
                 for i in range(batch):
                     pos[i] += 1
-            dt_dm = timed(decode_m, steps)
+            dt_dm = _timed(decode_m, steps, warm)
             models.prof_begin(); decode_m(); prof_dm = models.prof_end()
             rec["mistral"] = {"prefill_tok_s": T / dt_pm, "prefill_ms": dt_pm * 1e3, "decode_tok_s": batch / dt_dm, "decode_ms_per_step": dt_dm * 1e3,
                               "weight_bytes": mx.dev.streamed_bytes(), "prefill_kernels": _profile_table(prof_pm), "decode_kernels": _profile_table(prof_dm)}
@@ -1125,43 +1129,14 @@ def run_tozarax_compare(args, local_rank):
     weights -- Rofetar for the mixers (the same attention and delta-rule kernels, one per layer instead of both) and Nifunex for the
     experts (8 experts top-2 on the same grouped GEMMs).  One 2048-token prefill and batch-8 decode steps at a 2k context, through
     the public calls (host ids in, logits out), with the per-kernel CUDA-event profile of one call of each kind."""
-    import torch
     from fastllm_b200 import models
     batch, T, steps, warm = 8, 2048, max(4, min(args.steps, 32)), 3
     sizes = [("w1024", 1024, 1408, 4), ("w2048", 2048, 2816, 4), ("w4096", 4096, 7168, 4)]
     vocab = 32000
     results = {}
 
-    def timed(fn, n):
-        for _ in range(warm):
-            fn()
-        torch.cuda.synchronize()
-        t0 = time.perf_counter()
-        for _ in range(n):
-            fn()
-        torch.cuda.synchronize()
-        return (time.perf_counter() - t0) / n
-
     def layered(cls, cfg, **hints):
-        model, _ = cls.initialize_model(cfg, None, "bf16", local_rank, random_seed=0, std=0.02, **hints)
-        cache = model.new_device_cache(max_batch=batch, max_seq=T + 64, pool_tokens=batch * (T + 64))
-        ids = (np.arange(T, dtype=np.uint64) * 7919 % (vocab - 5) + 3).astype(np.uint32)
-
-        def prefill():
-            cache.slot_reset(0)
-            cache.forward_ragged([0], [ids], None)
-        dt_p = timed(prefill, max(2, steps // 4))
-        models.prof_begin(); prefill(); prof_p = models.prof_end()
-        for s in range(1, batch):
-            cache.forward_ragged([s], [ids], None)
-        slots = list(range(batch))
-
-        def decode():
-            cache.forward_ragged(slots, [[7 + s] for s in slots], None)
-        dt_d = timed(decode, steps)
-        models.prof_begin(); decode(); prof_d = models.prof_end()
-        return {"prefill_tok_s": T / dt_p, "prefill_ms": dt_p * 1e3, "decode_tok_s": batch / dt_d, "decode_ms_per_step": dt_d * 1e3,
-                "weight_bytes": model.dev.streamed_bytes(), "prefill_kernels": _profile_table(prof_p), "decode_kernels": _profile_table(prof_d)}
+        return _layered_record(cls, cfg, local_rank, batch, T, steps, warm, vocab, **hints)
 
     with ClockSampler(local_rank) as clk:
         t_wall0 = time.time()
@@ -1209,43 +1184,14 @@ def run_medulorn_compare(args, local_rank):
     random weights -- Tozarax (two mixers side by side on the same attention and scan kernels, experts on the same grouped GEMMs) and
     Rofetar (attention with q/k norm, rotation and sink).  One 2048-token prefill and batch-8 decode steps at a 2k context, through
     the public calls (host ids in, logits out), with the per-kernel CUDA-event profile of one call of each kind."""
-    import torch
     from fastllm_b200 import models
     batch, T, steps, warm = 8, 2048, max(4, min(args.steps, 32)), 3
     sizes = [("w1024", 1024, 1408, 4), ("w2048", 2048, 2816, 4), ("w4096", 4096, 7168, 4)]
     vocab = 32000
     results = {}
 
-    def timed(fn, n):
-        for _ in range(warm):
-            fn()
-        torch.cuda.synchronize()
-        t0 = time.perf_counter()
-        for _ in range(n):
-            fn()
-        torch.cuda.synchronize()
-        return (time.perf_counter() - t0) / n
-
     def layered(cls, cfg, **hints):
-        model, _ = cls.initialize_model(cfg, None, "bf16", local_rank, random_seed=0, std=0.02, **hints)
-        cache = model.new_device_cache(max_batch=batch, max_seq=T + 64, pool_tokens=batch * (T + 64))
-        ids = (np.arange(T, dtype=np.uint64) * 7919 % (vocab - 5) + 3).astype(np.uint32)
-
-        def prefill():
-            cache.slot_reset(0)
-            cache.forward_ragged([0], [ids], None)
-        dt_p = timed(prefill, max(2, steps // 4))
-        models.prof_begin(); prefill(); prof_p = models.prof_end()
-        for s in range(1, batch):
-            cache.forward_ragged([s], [ids], None)
-        slots = list(range(batch))
-
-        def decode():
-            cache.forward_ragged(slots, [[7 + s] for s in slots], None)
-        dt_d = timed(decode, steps)
-        models.prof_begin(); decode(); prof_d = models.prof_end()
-        return {"prefill_tok_s": T / dt_p, "prefill_ms": dt_p * 1e3, "decode_tok_s": batch / dt_d, "decode_ms_per_step": dt_d * 1e3,
-                "weight_bytes": model.dev.streamed_bytes(), "prefill_kernels": _profile_table(prof_p), "decode_kernels": _profile_table(prof_d)}
+        return _layered_record(cls, cfg, local_rank, batch, T, steps, warm, vocab, **hints)
 
     with ClockSampler(local_rank) as clk:
         t_wall0 = time.time()
@@ -1264,6 +1210,61 @@ def run_medulorn_compare(args, local_rank):
                       "config": {"workload": WORKLOADS[args.workload][3], "batch": batch, "context": T, "timing": "wall clock around the public call "
                                  "(host ids in, f32 logits out) with a device synchronise on both sides; per-kernel figures are CUDA events",
                                  "l2": "weights of a step exceed L2 at every size"},
+                      "clocks": clk.summary(t_wall0, t_wall1), "sizes": results}), flush=True)
+
+
+def _latodra_config(width, ff, layers, vocab, times):
+    """A Latodra config at the sizes of a real model's layers: heads with 128 unrotated and 64 rotated channels, values of 128, latents of
+    512, query latents of 3/8 of the width, YaRN; every other layer without positions and with gated heads; the middle layers run
+    `times` times."""
+    H = width // 128
+    ly = []
+    for i in range(layers):
+        m = {"heads": H, "dim": 128, "vdim": 128, "kv_rank": 512, "q_rank": width * 3 // 8, "scale": 128 ** -0.5}
+        if i % 2 == 0:
+            m.update(rot_dim=64, scale=192 ** -0.5, rot={"base": 10000.0, "dims": 64, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}})
+        ly.append({"type": "latent_attention" if i % 2 == 0 else "latent_attention_2", "mixer": m, "mlp": {"kind": "dense", "ff": ff}})
+    return {"architecture": "Latodra", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "loop": {"start": 1, "stop": layers - 1, "times": times}, "layers": ly}
+
+
+def _nifunex_latent_config(width, ff, layers, vocab):
+    """Nifunex with a latent attention of the same head, value and latent sizes in every layer (its own cache each, no window) and a
+    dense feed-forward of the same width: the closest existing design at equal sizes."""
+    m = {"heads": width // 128, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "scale": 192 ** -0.5, "rot": {"base": 10000.0, "dims": 64}}
+    return {"architecture": "Nifunex", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "layers": [{"type": "latent_attention", "mixer": m, "mlp": {"kind": "dense", "ff": ff, "limit": 7.0}} for _ in range(layers)]}
+
+
+def run_latodra_compare(args, local_rank):
+    """--workload latodra_vs_nifunex (one GPU): Latodra (each layer once, and with its middle layers run twice) beside Nifunex with latent
+    attention in every layer at the same width / ff / head / latent sizes, random weights: one 2048-token prefill and batch-8 decode
+    steps at a 2k context."""
+    from fastllm_b200 import models
+    batch, T, steps, warm = 8, 2048, max(4, min(args.steps, 32)), 3
+    sizes = [("w1024", 1024, 2816, 4), ("w2048", 2048, 5632, 4), ("w4096", 4096, 14336, 4)]
+    vocab = 32000
+    results = {}
+
+    def layered(cls, cfg, **hints):
+        return _layered_record(cls, cfg, local_rank, batch, T, steps, warm, vocab, **hints)
+
+    with ClockSampler(local_rank) as clk:
+        t_wall0 = time.time()
+        for name, width, ff, layers in sizes:
+            rec = {"width": width, "ff": ff, "layers": layers}
+            rec["latodra"] = layered(models.LatodraWithConfig, _latodra_config(width, ff, layers, vocab, 1))
+            rec["latodra_twice"] = layered(models.LatodraWithConfig, _latodra_config(width, ff, layers, vocab, 2))
+            rec["nifunex"] = layered(models.NifunexWithConfig, _nifunex_latent_config(width, ff, layers, vocab))
+            results[name] = rec
+        t_wall1 = time.time()
+        time.sleep(0.12)
+    big = results[sizes[-1][0]]
+    print(json.dumps({"metric": "decode_tokens_per_s", "value": big["latodra"]["decode_tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": steps, "warmup": warm,
+                      "ms_per_step": big["latodra"]["decode_ms_per_step"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16",
+                      "data": "synthetic",
+                      "config": {"workload": WORKLOADS[args.workload][3], "batch": batch, "context": T, "timing": "wall clock around the public call "
+                                 "(host ids in, f32 logits out) with a device synchronise on both sides; per-kernel figures are CUDA events",
+                                 "l2": "weights of a step exceed L2 at the two larger sizes"},
                       "clocks": clk.summary(t_wall0, t_wall1), "sizes": results}), flush=True)
 
 
@@ -1306,6 +1307,9 @@ def main():
     elif args.workload == "medulorn_vs_tozarax":
         if rank == 0:
             run_medulorn_compare(args, local_rank)
+    elif args.workload == "latodra_vs_nifunex":
+        if rank == 0:
+            run_latodra_compare(args, local_rank)
     elif args.workload == "rofetar_vs_nifunex":
         if rank == 0:
             run_rofetar_compare(args, local_rank)

@@ -570,6 +570,17 @@ void layered_finalize(LayeredModel& m) {
             const fl_layer_desc& d = lw.d;
             map(lw.w_in, lw.n_in, m.W, lw.tm_in, lw.tc_in);
             map(lw.w_o, m.W, d.heads * d.vdim, lw.tm_o, lw.tc_o);
+            if (d.mixer == FL_MIXER_LATENT_ATTN) {
+                // sizes in multiples of 8 may end inside a k block (the tensor maps fill its rest with zeros)
+                const int H = d.heads, D = d.dim, Dv = d.vdim, C = d.kv_rank, R = d.rot_dim;
+                lw.lat_tc = D % 8 == 0 && Dv % 8 == 0 && C % 8 == 0 && R % 8 == 0 && m.W % 8 == 0 && (lw.off_g < 0 || lw.off_g % 4 == 0) && lw.n_in % 4 == 0;
+                if (lw.lat_tc) {
+                    lw.tm_uk = make_tmap_bf16(lw.uk_t, (uint64_t)H * C, (uint64_t)D, (uint64_t)D, 128);
+                    lw.tm_uv = make_tmap_bf16(lw.uv, (uint64_t)H * Dv, (uint64_t)C, (uint64_t)C, 128);
+                    if (!lw.tc_o) { lw.tc_o = true; lw.tm_o = make_tmap_bf16(lw.w_o, (uint64_t)m.W, (uint64_t)H * Dv, (uint64_t)H * Dv, 128); }
+                    m.max_hp = std::max(m.max_hp, H * D); m.max_hq = std::max(m.max_hq, H * ((C + R + 63) / 64 * 64)); m.max_c = std::max(m.max_c, C);
+                }
+            }
             // (a query latent may end inside a k block: the tensor maps fill its rest with zeros)
             lw.tc_uq = lw.uq != nullptr && d.q_rank % 8 == 0 && d.heads * (d.dim + d.rot_dim) % 8 == 0;
             if (lw.tc_uq) {
@@ -689,7 +700,11 @@ void layered_cache_create(fl_cache& c, int max_slots, int max_seq, int pool_toke
         }
     }
     y.page_table.alloc((size_t)max_slots * c.pages_per_seq, true);
-    if (m.max_av > 0 && !m.f32) y.at_part.alloc((size_t)kGqaSplitRows * kGqaMaxSplits * (m.max_av + 2));
+    {
+        size_t part = m.max_av > 0 && !m.f32 ? (size_t)kGqaSplitRows * kGqaMaxSplits * (m.max_av + 2) : 0;
+        if (m.max_c > 0) part = std::max(part, (size_t)kNumSMs * 32 * (m.max_c + 2));
+        y.at_part.alloc(part);
+    }
     c.slot_len.assign(max_slots, 0);
     FL_CUDA(cudaDeviceSynchronize());
 }
@@ -728,7 +743,13 @@ static void ensure_ws(fl_cache& c, size_t T, size_t n_want) {
         if (m.max_qr > 0) { y.cq.alloc(R * m.max_qr); y.qx.alloc(R * m.max_q); }
         for (const LayeredLayerW& lw : m.layers)
             if (lw.side && y.y2.n < R * W) y.y2.alloc(R * W);
-        y.qa.alloc(R * std::max(m.max_hc, 1)); y.ol.alloc(R * std::max(m.max_hc, 1));
+        bool plain_latent = false;          // a latent attention that is not on the tensor cores keeps f32 query / value rows
+        for (const LayeredLayerW& lw : m.layers) plain_latent |= lw.d.mixer == FL_MIXER_LATENT_ATTN && !lw.lat_tc;
+        if (plain_latent) { y.qa.alloc(R * m.max_hc); y.ol.alloc(R * m.max_hc); }
+        if (m.max_hq > 0) {
+            y.qp_hi.alloc(R * m.max_hp); y.qp_lo.alloc(R * m.max_hp); y.qo_hi.alloc(R * m.max_hq); y.qo_lo.alloc(R * m.max_hq);
+            y.ol_hi.alloc(R * m.max_hc); y.ol_lo.alloc(R * m.max_hc);
+        }
         y.gu.alloc(P * 2 * std::max(m.max_ff, 1)); y.act.alloc(P * std::max(m.max_ff, 1)); y.eo.alloc(P * W);
         y.sh_gu.alloc(R * 2 * std::max(m.max_ff, 1)); y.sh_act.alloc(R * std::max(m.max_ff, 1)); y.sh_o.alloc(R * W);
         y.route_w.alloc(P); y.route_sel.alloc(P); y.sgate.alloc(R);
@@ -818,6 +839,35 @@ static void launch_latent_attn(LaunchCtx& lc, const LatentAttnArgs& a, int T) {
     else launch(lc, "latent_attn", bytes, ly_latent_attn_kernel<CT, 16>, g, b, smem, a);
 }
 
+template <int MT, int NT>
+static void launch_latent_mma_t(LaunchCtx& lc, const LatMmaArgs& a, int T, int splits) {
+    static bool attr_set = false;
+    if (!attr_set) {
+        FL_CUDA(cudaFuncSetAttribute(ly_latent_mma_kernel<MT, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kLatSmemMax));
+        attr_set = true;
+    }
+    launch(lc, "latent_attn", 0, ly_latent_mma_kernel<MT, NT>, dim3(T, (a.H + 16 * MT - 1) / (16 * MT), splits), dim3(256), lat_mma_smem(a.Ep, MT), a);
+}
+// max_keys: the most keys a row of the launch can see.  Few (row, head group) pairs split each row's pages over several blocks.
+static void launch_latent_mma(LaunchCtx& lc, const LatMmaArgs& a, int T, int max_keys) {
+    if (T <= 0) return;
+    const bool wide = a.H > 16 && lat_mma_smem(a.Ep, 2) <= kLatSmemMax;        // two groups of 16 heads share a block's tiles
+    const int groups = wide ? (a.H + 31) / 32 : (a.H + 15) / 16;
+    int splits = std::max(1, std::min(kGqaMaxSplits, kNumSMs / (T * groups)));
+    splits = std::min(splits, (max_keys + kLatTile - 1) / kLatTile);
+    auto go = [&](auto mt) {
+        constexpr int MT = decltype(mt)::value;
+        if (a.C <= 64) launch_latent_mma_t<MT, 1>(lc, a, T, splits);
+        else if (a.C <= 128) launch_latent_mma_t<MT, 2>(lc, a, T, splits);
+        else if (a.C <= 256) launch_latent_mma_t<MT, 4>(lc, a, T, splits);
+        else launch_latent_mma_t<MT, 8>(lc, a, T, splits);
+    };
+    if (wide) go(std::integral_constant<int, 2>{}); else go(std::integral_constant<int, 1>{});
+    if (splits > 1)
+        launch(lc, "latent_merge", 0, ly_gqa_merge_kernel, dim3(T, a.H), dim3(std::min(256, (a.C + 31) / 32 * 32)), 0, (const float*)a.part, splits, a.H, a.C, a.sink,
+               a.sinkv, a.row_base, (float*)nullptr, a.ohi, a.olo);
+}
+
 static void launch_gla_scan(LaunchCtx& lc, const GlaArgs& a, int n) {
     const int rpt = (a.D + kGlaDG - 1) / kGlaDG;
     const size_t smem = ((size_t)6 * a.D + 2 * kGlaVS + 2 * kGlaDG * kGlaVS) * 4;
@@ -878,7 +928,8 @@ static void launch_rec_scan(LaunchCtx& lc, const RecArgs& a, int n) {
 // Latent attention of rows [r0, r0 + Ts) -- one sequence's portion, positions pos0.. -- on the tensor-core GEMM, in blocks of query
 // rows small enough that a block's score matrix stays within a fixed scratch budget.  A block only gathers the keys its rows'
 // windows reach, so long prompts with short windows never touch fully masked regions.
-static void latent_attn_tc(fl_cache& c, LaunchCtx& lc, const LayeredLayerW& lw, const LatentAttnArgs& a, int r0, int Ts, int pos0, int slot) {
+// mma != nullptr: the step's query operand exists already and the result goes to hi | lo halves (the mixer runs on the tensor cores).
+static void latent_attn_tc(fl_cache& c, LaunchCtx& lc, const LatentAttnArgs& a, const LatMmaArgs* mma, int r0, int Ts, int pos0, int slot) {
     LayeredCache& y = *c.ly;
     const int H = a.H, C = a.C, R = a.R, E = C + R, Ep = (E + 63) / 64 * 64;
     const size_t budget = (size_t)48 << 20;                // floats in a score block (192 MB); P halves take the same again
@@ -894,7 +945,7 @@ static void latent_attn_tc(fl_cache& c, LaunchCtx& lc, const LayeredLayerW& lw, 
     for (int f = 0; f < Ts; f += qb) nkp_max = std::max<size_t>(nkp_max, keys_for(qb, f));
     auto need = [&](auto& buf, size_t n) { if (buf.n < n) { FL_CUDA(cudaStreamSynchronize(c.stream)); buf.alloc(n + n / 4); } };
     need(y.at_kc, nkp_max * Ep); need(y.at_kct, (size_t)C * nkp_max);
-    need(y.at_qhi, rows_max * Ep); need(y.at_qlo, rows_max * Ep);
+    if (mma == nullptr) { need(y.at_qhi, rows_max * Ep); need(y.at_qlo, rows_max * Ep); }
     need(y.at_s, rows_max * nkp_max); need(y.at_phi, rows_max * nkp_max); need(y.at_plo, rows_max * nkp_max);
     const int* page_row = y.page_table.p + (size_t)slot * c.pages_per_seq;
     for (int f = 0; f < Ts; f += qb) {
@@ -902,22 +953,33 @@ static void latent_attn_tc(fl_cache& c, LaunchCtx& lc, const LayeredLayerW& lw, 
         const int k_lo = (a.window > 0 && p_lo - a.window + 1 > 0) ? p_lo - a.window + 1 : 0, nk = p_hi - k_lo, nkp = (nk + 63) / 64 * 64;
         const int rows = nq * H;
         if (rows <= 128) {          // a short tail: the per-(row, head) kernel
-            LatentAttnArgs t = a;
-            t.row_base = r0 + f;
-            launch_latent_attn<uint16_t>(lc, t, nq);
+            if (mma != nullptr) {
+                LatMmaArgs t = *mma;
+                t.row_base = r0 + f;
+                launch_latent_mma(lc, t, nq, p_hi);
+            } else {
+                LatentAttnArgs t = a;
+                t.row_base = r0 + f;
+                launch_latent_attn<uint16_t>(lc, t, nq);
+            }
             continue;
         }
         launch(lc, "attn_gather_keys", 0, ly_attn_gather_keys_kernel, dim3(nkp), dim3(128), 0, (const uint16_t*)a.pool, page_row, k_lo, nk, nkp, C, E, Ep,
                y.at_kc.p, y.at_kct.p);
-        launch(lc, "attn_build_q", 0, ly_attn_build_q_kernel, dim3(nq, H), dim3(128), 0, a.qa, a.proj, a.ldp, a.off_q, r0 + f, H, a.D, R, C, Ep, a.scale,
-               y.at_qhi.p, y.at_qlo.p);
+        const size_t q0 = (size_t)(r0 + f) * H;
+        if (mma == nullptr)
+            launch(lc, "attn_build_q", 0, ly_attn_build_q_kernel, dim3(nq, H), dim3(128), 0, a.qa, a.proj, a.ldp, a.off_q, r0 + f, H, a.D, R, C, Ep, a.scale,
+                   y.at_qhi.p, y.at_qlo.p);
         const CUtensorMap tk = make_tmap_bf16(y.at_kc.p, (uint64_t)nkp, (uint64_t)Ep, (uint64_t)Ep, 128);
-        dense_gemm(c, lc, "gemm_tc_attn_scores", rows, nkp, Ep, tk, y.at_s.p, y.at_qhi.p, y.at_qlo.p);
+        dense_gemm(c, lc, "gemm_tc_attn_scores", rows, nkp, Ep, tk, y.at_s.p, mma ? mma->qhi + q0 * Ep : y.at_qhi.p, mma ? mma->qlo + q0 * Ep : y.at_qlo.p);
         const int keep = std::min(nkp, kSoftmaxKeep);
         launch(lc, "attn_softmax", 0, ly_attn_softmax_kernel, dim3(rows), dim3(256), (size_t)keep * 4, (const float*)y.at_s.p, a.row_pos, r0 + f, H, k_lo, 0, nk, nkp,
                a.window, 0, 0, 0.f, a.sink, a.sinkv, keep, y.at_phi.p, y.at_plo.p);
         const CUtensorMap tv = make_tmap_bf16(y.at_kct.p, (uint64_t)C, (uint64_t)nkp, (uint64_t)nkp, 128);
-        dense_gemm(c, lc, "gemm_tc_attn_values", rows, C, nkp, tv, a.ol + (size_t)(r0 + f) * H * C, y.at_phi.p, y.at_plo.p);
+        if (mma != nullptr)
+            dense_gemm_blocks(c, lc, "gemm_tc_attn_values", rows, 1, C, nkp, tv, y.at_phi.p, y.at_plo.p, mma->ohi + q0 * C, mma->olo + q0 * C, C, 0);
+        else
+            dense_gemm(c, lc, "gemm_tc_attn_values", rows, C, nkp, tv, a.ol + q0 * C, y.at_phi.p, y.at_plo.p);
     }
 }
 
@@ -1197,33 +1259,63 @@ static void run_mixer(fl_cache& c, LaunchCtx& lc, const StepTab& st, const Layer
         if (Q > 0) {
             q = y.qx.p; ldq = H * (D + R);
             gemm_tc_or_exact(c, lc, "gemm_q_up", y.cq.p, y.cq_hi.p, y.cq_lo.p, lw.uq, lw.tm_uq, lw.tc_uq, ldq, Q, q, Ti);
-            if (d.rot_dims > 0)
+            if (d.rot_dims > 0 && !lw.lat_tc)
                 launch(lc, "rotate_q", 0, ly_rotate_q_kernel, dim3(Ti), dim3(128), 0, q, ldq, st.row_pos, (const float*)y.rope_cos[lw.rope_index].p,
                        (const float*)y.rope_sin[lw.rope_index].p, H, D, R, d.rot_dims);
+        }
+        static const bool tc_attn_off = env_flag("FL_LAYERED_NO_TC_ATTN");
+        // Rows are taken in order: long portions (serving precision) run scores and weighted sums as tensor-core GEMMs over the
+        // gathered window, everything else goes to `rest`(first row, rows).
+        auto walk = [&](const LatentAttnArgs& at, const LatMmaArgs* mma, bool gemms, auto&& rest) {
+            int done = 0;           // rows [0, done) are finished
+            for (int si = 0; si < n; ++si) {
+                const int r0 = h_row0[si], Ts = counts[si];
+                if (!gemms || Ts < 64 || (long long)Ts * H <= 128) continue;
+                if (r0 > done) rest(done, r0 - done);
+                latent_attn_tc(c, lc, at, mma, r0, Ts, h_pos0[si], slots[si]);
+                done = r0 + Ts;
+            }
+            if (done < Ti) rest(done, Ti - done);
+        };
+        if (lw.lat_tc) {
+            // the whole mixer over hi | lo halves: split queries -> W_uk absorbed (one block per head) -> attention -> W_uv (and the
+            // gate) -> the output projection's operand
+            const int Ep = (C + R + 63) / 64 * 64;
+            const bool turn = Q > 0 && d.rot_dims > 0;
+            launch(lc, "latent_split_q", 0, ly_latent_split_q_kernel, dim3(Ti), dim3(256), 0, (const float*)q, ldq, st.row_pos,
+                   turn ? (const float*)y.rope_cos[lw.rope_index].p : (const float*)nullptr, (const float*)y.rope_sin[lw.rope_index].p, H, D, R, d.rot_dims, C, Ep,
+                   d.scale, y.qp_hi.p, y.qp_lo.p, y.qo_hi.p, y.qo_lo.p);
+            dense_gemm_blocks(c, lc, "gemm_q_absorb", Ti, H, C, D, lw.tm_uk, y.qp_hi.p, y.qp_lo.p, y.qo_hi.p, y.qo_lo.p, H * Ep, Ep);
+            LatentAttnArgs at{nullptr, q, ldq, 0, y.kv_pool[kv_index], y.page_table.p, c.pages_per_seq, st.row_seq, st.row_pos,
+                              st.seq_slot, nullptr, H, D, R, C, d.window, d.scale, 0, d.sink, lw.sinkv};
+            LatMmaArgs ma{y.qo_hi.p, y.qo_lo.p, (const uint16_t*)y.kv_pool[kv_index], y.page_table.p, c.pages_per_seq, st.row_seq, st.row_pos, st.seq_slot,
+                          y.ol_hi.p, y.ol_lo.p, y.at_part.p, H, C, R, Ep, d.window, 0, d.sink, lw.sinkv};
+            // a step of single tokens is replayed from a captured graph whatever the contexts' lengths: its split count must not follow them
+            int max_keys = c.max_seq;
+            if (Ti != n) {
+                max_keys = 1;
+                for (int si = 0; si < n; ++si) max_keys = std::max(max_keys, h_pos0[si] + counts[si]);
+            }
+            if (d.window > 0) max_keys = std::min(max_keys, d.window + kLatTile);
+            walk(at, &ma, !tc_attn_off, [&](int first, int rows) {
+                LatMmaArgs t = ma;
+                t.row_base = first;
+                launch_latent_mma(lc, t, rows, max_keys);
+            });
+            dense_gemm_blocks(c, lc, "gemm_v_expand", Ti, H, Dv, C, lw.tm_uv, y.ol_hi.p, y.ol_lo.p, uhi, ulo, H * Dv, Dv,
+                              d.out_gate ? (const float*)y.proj.p + lw.off_g : (const float*)nullptr, d.out_gate ? lw.n_in : 0);
+            return;
         }
         // q~[row, h, :] = W_uk[h]^T q_plain[row, h, :]: the score against the latent needs no per-head keys
         LyGemm qa{q, D + R, ldq, nullptr, lw.uk_t, (long long)C * D, C, D, y.qa.p, C, H * C, nullptr, Ti};
         gemm_groups(lc, "gemm_q_absorb", qa, H, Ti);
         LatentAttnArgs at{y.qa.p, q, ldq, 0, y.kv_pool[kv_index], y.page_table.p, c.pages_per_seq, st.row_seq, st.row_pos,
                           st.seq_slot, y.ol.p, H, D, R, C, d.window, d.scale, 0, d.sink, lw.sinkv};
-        // long portions (serving precision): scores and weighted sums as tensor-core GEMMs over the gathered window; everything
-        // else (decoded tokens, short portions, the exact mode) on the per-(row, head) kernel.  Rows are taken in order.
-        static const bool tc_attn_off = env_flag("FL_LAYERED_NO_TC_ATTN");
-        int done = 0;           // rows [0, done) are finished
-        for (int si = 0; si < n; ++si) {
-            const int r0 = h_row0[si], Ts = counts[si];
-            if (m.f32 || tc_attn_off || C % 8 != 0 || Ts < 64 || (long long)Ts * H <= 128) continue;
-            if (r0 > done) {
-                at.row_base = done;
-                launch_latent_attn<uint16_t>(lc, at, r0 - done);
-            }
-            latent_attn_tc(c, lc, lw, at, r0, Ts, h_pos0[si], slots[si]);
-            done = r0 + Ts;
-        }
-        if (done < Ti) {
-            at.row_base = done;
-            if (m.f32) launch_latent_attn<float>(lc, at, Ti - done); else launch_latent_attn<uint16_t>(lc, at, Ti - done);
-        }
+        walk(at, nullptr, !m.f32 && !tc_attn_off && C % 8 == 0, [&](int first, int rows) {      // the exact mode: everything on the per-(row, head) kernel
+            LatentAttnArgs t = at;
+            t.row_base = first;
+            if (m.f32) launch_latent_attn<float>(lc, t, rows); else launch_latent_attn<uint16_t>(lc, t, rows);
+        });
         // value expansion after the softmax: out[row, h, :] = W_uv[h] (sum_j p_j c_j)
         LyGemm ov{y.ol.p, C, H * C, nullptr, lw.uv, (long long)Dv * C, Dv, C, y.u.p, Dv, H * Dv, nullptr, Ti};
         gemm_groups(lc, "gemm_v_expand", ov, H, Ti);

@@ -1168,6 +1168,47 @@ int dense_gemm(fl_cache& c, LaunchCtx& lc, const char* tag, int R, int N, int K,
     return ks;
 }
 
+// Block-diagonal GEMM with hi | lo output (see GemmArgs.blocks): tokens are the M dimension above 128 rows, else the weights are
+// (swap-AB, never split over K: the halves are those of the finished sum).
+void dense_gemm_blocks(fl_cache& c, LaunchCtx& lc, const char* tag, int R, int blocks, int N, int K, const CUtensorMap& tmW, const uint16_t* xhi,
+                       const uint16_t* xlo, uint16_t* ohi, uint16_t* olo, int ldo, int o_bs, const float* gate, int ldg) {
+    FL_CHECK(K % 8 == 0 && N % 8 == 0 && ldo % 8 == 0 && o_bs % 8 == 0 && ldg % 4 == 0, FL_ERR_STATE, "internal: block-diagonal GEMM alignment");
+    const bool prof = g_prof.on && !lc.capturing;
+    const bool pdl = lc.pdl && !prof;
+    ProfEntry pe;
+    if (prof) {
+        pe.tag = tag;
+        pe.bytes = (uint64_t)blocks * N * K * 2;
+        FL_CUDA(cudaEventCreate(&pe.e0));
+        FL_CUDA(cudaEventCreate(&pe.e1));
+        FL_CUDA(cudaEventRecord(pe.e0, lc.stream));
+    }
+    const bool swap = R <= 128;
+    GemmArgs g{swap ? N : R, swap ? R : N, K, nullptr, nullptr, 0, ohi, ldo, 1, 0, olo};
+    g.blocks = blocks; g.o_bs = o_bs; g.gate = gate; g.ldg = ldg;
+    const uint64_t KX = (uint64_t)blocks * K;
+    if (swap) {
+        const int bn = R <= 16 ? 16 : (R <= 32 ? 32 : (R <= 64 ? 64 : 128)), tiles = blocks * ((N + 127) / 128);
+        const CUtensorMap hi = make_tmap_bf16(xhi, R, KX, KX, bn), lo = make_tmap_bf16(xlo, R, KX, KX, bn);
+        switch (bn) {
+            case 16: launch_gemm_tc<16, GEPI_HL_T, DUAL_B>(lc.stream, pdl, tiles, tmW, hi, lo, g); break;
+            case 32: launch_gemm_tc<32, GEPI_HL_T, DUAL_B>(lc.stream, pdl, tiles, tmW, hi, lo, g); break;
+            case 64: launch_gemm_tc<64, GEPI_HL_T, DUAL_B>(lc.stream, pdl, tiles, tmW, hi, lo, g); break;
+            default: launch_gemm_tc<128, GEPI_HL_T, DUAL_B>(lc.stream, pdl, tiles, tmW, hi, lo, g); break;
+        }
+    } else {
+        const int mt = (R + kGemmBM - 1) / kGemmBM;
+        const CUtensorMap hi = make_tmap_bf16(xhi, R, KX, KX, kGemmBM), lo = make_tmap_bf16(xlo, R, KX, KX, kGemmBM);
+        if (N % 256 == 0 || N > 512) launch_gemm_tc<256, GEPI_HL, DUAL_A>(lc.stream, pdl, mt * blocks * ((N + 255) / 256), hi, lo, tmW, g);
+        else launch_gemm_tc<128, GEPI_HL, DUAL_A>(lc.stream, pdl, mt * blocks * ((N + 127) / 128), hi, lo, tmW, g);
+    }
+    if (prof) {
+        FL_CUDA(cudaEventRecord(pe.e1, lc.stream));
+        g_prof.entries.push_back(pe);
+    }
+    if (lc.capturing) lc.captured++; else g_launches.fetch_add(1, std::memory_order_relaxed);
+}
+
 // Grouped swap-AB GEMM over this rank's experts (decode batches): group j multiplies ITS gathered rows (block j of xhi / xlo,
 // `cap` rows, cnt[j] valid) with ITS matrix (block j of the stacked weights, Ne rows): out[ks][j * cap + n][Ne].  ONE launch over
 // (expert, weight tile, k slice) work items; an expert without rows costs nothing.  Returns the split-K factor.

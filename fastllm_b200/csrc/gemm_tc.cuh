@@ -18,7 +18,7 @@
 
 namespace fl {
 
-enum : int { GEPI_BIAS_BF16 = 0, GEPI_BIAS_GELU_BF16 = 1, GEPI_BIAS_RESID_F32 = 2, GEPI_F32 = 3, GEPI_ATOMIC_F32 = 4, GEPI_F32_T = 5, GEPI_SILU_HL = 6 };
+enum : int { GEPI_BIAS_BF16 = 0, GEPI_BIAS_GELU_BF16 = 1, GEPI_BIAS_RESID_F32 = 2, GEPI_F32 = 3, GEPI_ATOMIC_F32 = 4, GEPI_F32_T = 5, GEPI_SILU_HL = 6, GEPI_HL = 7, GEPI_HL_T = 8 };
 enum : int { DUAL_NONE = 0, DUAL_A = 1, DUAL_B = 2 };
 
 constexpr int kGemmBM = 128;
@@ -35,7 +35,7 @@ struct GemmArgs {
     int ldo;
     int ksplit;                 // >1: K is cut into ksplit ranges handled by different work items (GEPI_F32 / GEPI_ATOMIC_F32)
     long long split_stride;     // GEPI_F32 with ksplit > 1: split s writes its partial sums to out + s * split_stride (deterministic)
-    void* out2 = nullptr;       // GEPI_SILU_HL: the lo half ([M, ldo] bf16, like `out` = the hi half)
+    void* out2 = nullptr;       // GEPI_SILU_HL / GEPI_HL / GEPI_HL_T: the lo half (bf16, laid out like `out` = the hi half)
     int w_prefetch = 0;         // DUAL_B: request the first ring-full of WEIGHT tiles before griddepcontrol.wait (see the producer)
     // GROUPED swap-AB GEMM (DUAL_B + GEPI_F32_T; the Mixtral experts): A stacks `M / grp_m` weight matrices of grp_m rows each,
     // B stacks one block of grp_cap (<= BN) activation rows per group -- the rows routed to that expert, gathered -- and group j
@@ -45,6 +45,15 @@ struct GemmArgs {
     int grp_m = 0;
     int grp_cap = 0;
     const int* grp_cnt = nullptr;
+    // BLOCK-DIAGONAL GEMM (GEPI_HL with DUAL_A, GEPI_HL_T with DUAL_B): `blocks` stacked weight matrices, block b multiplies columns
+    // [b K, (b + 1) K) of the activations [tokens, blocks K]; the weight rows per block (N with DUAL_A, M with DUAL_B) and K are per
+    // block.  Where a block's K ends inside a k-block the weights are zero-filled (their map is K wide), so the neighbour's
+    // activations there count nothing.  Token t, block b, weight row n of the result goes to out[t * ldo + b * o_bs + n] as bf16 hi and
+    // out2 as lo, times sigmoid(gate[t * ldg + b * rows + n]) when there is a gate.
+    int blocks = 0;
+    int o_bs = 0;
+    const float* gate = nullptr;
+    int ldg = 0;
     int dbg = 0;                // dev knob FL_GEMM_DBG (timing experiments only, results are garbage): bit 0 = DUAL_B without the
                                 // activation loads, bit 1 = no MMAs (the issuer releases a stage as soon as it has landed)
 };
@@ -200,7 +209,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
     const int nk = (g.K + kGemmBK - 1) / kGemmBK;
     const bool grouped = (DUAL == DUAL_B) && g.grp_m > 0;
     const int mt_e = grouped ? (g.grp_m + kGemmBM - 1) / kGemmBM : 0;      // m tiles per group
-    const int mt = grouped ? (g.M / g.grp_m) * mt_e : (g.M + kGemmBM - 1) / kGemmBM, nt = grouped ? 1 : (g.N + BN - 1) / BN;
+    constexpr bool kBlocks = EPI == GEPI_HL || EPI == GEPI_HL_T;           // block-diagonal forms
+    const int nblk = kBlocks && g.blocks > 1 ? g.blocks : 1;
+    const int mt_b = (g.M + kGemmBM - 1) / kGemmBM, nt_b = (g.N + BN - 1) / BN;
+    const int mt = grouped ? (g.M / g.grp_m) * mt_e : (EPI == GEPI_HL_T ? nblk * mt_b : mt_b), nt = grouped ? 1 : (EPI == GEPI_HL ? nblk * nt_b : nt_b);
     const int ksplit = g.ksplit > 1 ? g.ksplit : 1;
     // tile -> (first row of the A box, first row of the B box, group, first row inside the group)
     auto coords = [&](int tile, int& m0, int& n0, int& grp, int& mrow0) {
@@ -209,6 +221,17 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
             mrow0 = (tile % mt_e) * kGemmBM;
             m0 = grp * g.grp_m + mrow0;
             n0 = grp * g.grp_cap;
+        } else if (EPI == GEPI_HL) {
+            const int bn = tile % nt;
+            grp = bn / nt_b;
+            m0 = mrow0 = (tile / nt) * kGemmBM;
+            n0 = grp * g.N + (bn % nt_b) * BN;
+        } else if (EPI == GEPI_HL_T) {
+            const int bm = tile / nt;
+            grp = bm / mt_b;
+            mrow0 = (bm % mt_b) * kGemmBM;
+            m0 = grp * g.M + mrow0;
+            n0 = (tile % nt) * BN;
         } else {
             grp = 0;
             m0 = mrow0 = (tile / nt) * kGemmBM;
@@ -272,6 +295,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
                 coords(tile, m0, n0, grp, mrow0);
                 if (grouped && g.grp_cnt[grp] == 0) continue;      // no row was routed to this expert: its weights are not read
                 const int kb1 = min((ks + 1) * nkps, nk);
+                const int ax = kBlocks ? grp * g.K : 0;            // first activation column of the item's block
                 for (int kb = ks * nkps; kb < kb1; ++kb, ++c) {
                     const int st = c % kStages;
                     uint8_t* sa = gsm + (size_t)st * kStageBytes;
@@ -289,11 +313,11 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
                     mbar_expect_tx(&full[st], kStageBytes);
                     if (DUAL == DUAL_B) {       // tmA = weights, tmA2 / tmB = activation hi / lo
                         tma_load_2d(sa, &tmA, kb * kGemmBK, m0, &full[st]);
-                        tma_load_2d(sa + kBOff, &tmA2, kb * kGemmBK, n0, &full[st]);
-                        tma_load_2d(sa + kBOff + kBBytes, &tmB, kb * kGemmBK, n0, &full[st]);
+                        tma_load_2d(sa + kBOff, &tmA2, ax + kb * kGemmBK, n0, &full[st]);
+                        tma_load_2d(sa + kBOff + kBBytes, &tmB, ax + kb * kGemmBK, n0, &full[st]);
                     } else {
-                        tma_load_2d(sa, &tmA, kb * kGemmBK, m0, &full[st]);
-                        if (DUAL == DUAL_A) tma_load_2d(sa + kABytes, &tmA2, kb * kGemmBK, m0, &full[st]);
+                        tma_load_2d(sa, &tmA, ax + kb * kGemmBK, m0, &full[st]);
+                        if (DUAL == DUAL_A) tma_load_2d(sa + kABytes, &tmA2, ax + kb * kGemmBK, m0, &full[st]);
                         tma_load_2d(sa + kBOff, &tmB, kb * kGemmBK, n0, &full[st]);
                         // DUAL_A with a 256-row weight tile: the weight descriptors carry a 128-row box (the swap-AB decode GEMMs'
                         // A operand), so the tile arrives as two boxes; rows past the matrix are zero-filled by the TMA engine
@@ -358,6 +382,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
             const int row = mrow0 + q * 32 + lane;
             const int row_lim = grouped ? g.grp_m : g.M, col_lim = grouped ? gcnt : g.N;
             if (grouped) n0 = 0;
+            if (EPI == GEPI_HL) n0 -= grp * g.N;       // columns count inside the block
             mbar_wait(&acc_full[as], (ti_now >> 1) & 1);
             tc_fence_after();
 #pragma unroll 1
@@ -502,6 +527,46 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
                                 *reinterpret_cast<uint4*>(ol + (j >> 1)) = make_uint4(pl[0], pl[1], pl[2], pl[3]);
                             }
                         }
+                    } else if (EPI == GEPI_HL) {
+                        const size_t o = (size_t)row * g.ldo + (size_t)grp * g.o_bs + col;
+                        uint16_t *oh = reinterpret_cast<uint16_t*>(g.out) + o, *ol = reinterpret_cast<uint16_t*>(g.out2) + o;
+                        const float* gt = g.gate != nullptr ? g.gate + (size_t)row * g.ldg + (size_t)grp * g.N + col : nullptr;
+#pragma unroll
+                        for (int j = 0; j < 32; j += 8) {
+                            if (col + j < g.N) {
+                                float v[8];
+#pragma unroll
+                                for (int e = 0; e < 8; ++e) v[e] = __uint_as_float(r[j + e]);
+                                if (gt != nullptr) {
+                                    const float4 z0 = *reinterpret_cast<const float4*>(gt + j), z1 = *reinterpret_cast<const float4*>(gt + j + 4);
+                                    const float z[8] = {z0.x, z0.y, z0.z, z0.w, z1.x, z1.y, z1.z, z1.w};
+#pragma unroll
+                                    for (int e = 0; e < 8; ++e) v[e] *= 1.f / (1.f + expf(-z[e]));
+                                }
+                                uint32_t ph[4], pl[4];
+#pragma unroll
+                                for (int e = 0; e < 4; ++e) {
+                                    ph[e] = pack_bf16x2(v[2 * e], v[2 * e + 1]);
+                                    pl[e] = pack_bf16x2(v[2 * e] - bf16lo(ph[e]), v[2 * e + 1] - bf16hi(ph[e]));
+                                }
+                                *reinterpret_cast<uint4*>(oh + j) = make_uint4(ph[0], ph[1], ph[2], ph[3]);
+                                *reinterpret_cast<uint4*>(ol + j) = make_uint4(pl[0], pl[1], pl[2], pl[3]);
+                            }
+                        }
+                    } else if (EPI == GEPI_HL_T) {
+                        // for a fixed token the 32 lanes of the warp write 32 consecutive halves
+                        const size_t o = (size_t)grp * g.o_bs + row;
+                        uint16_t *oh = reinterpret_cast<uint16_t*>(g.out) + o, *ol = reinterpret_cast<uint16_t*>(g.out2) + o;
+                        const float* gt = g.gate != nullptr ? g.gate + (size_t)grp * g.M + row : nullptr;
+#pragma unroll
+                        for (int j = 0; j < 32; ++j)
+                            if (col + j < g.N) {
+                                float v = __uint_as_float(r[j]);
+                                if (gt != nullptr) v *= 1.f / (1.f + expf(-gt[(size_t)(col + j) * g.ldg]));
+                                const uint16_t h = f32_to_bf16_rne(v);
+                                oh[(size_t)(col + j) * g.ldo] = h;
+                                ol[(size_t)(col + j) * g.ldo] = f32_to_bf16_rne(v - __uint_as_float((uint32_t)h << 16));
+                            }
                     } else if (EPI == GEPI_F32_T) {
                         // transposed store: D[row = weight row, col = activation row] -> out[slice][col, row]; for a fixed col the
                         // 32 lanes of the warp write 32 consecutive floats

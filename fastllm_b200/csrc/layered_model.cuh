@@ -51,8 +51,9 @@ struct LayeredLayerW {
     uint16_t* uv = nullptr;             // [heads * vdim, kv_rank]
     float* dq_norm = nullptr;           // query latent: [q_rank]
     uint16_t* uq = nullptr;             // query latent: [heads * (dim + rot_dim), q_rank]
-    CUtensorMap tm_uq{};
+    CUtensorMap tm_uq{}, tm_uk{}, tm_uv{};
     bool tc_uq = false;
+    bool lat_tc = false;                // serving precision: the whole mixer on the tensor cores (block-diagonal W_uk / W_uv GEMMs over hi | lo halves)
     int kv_owner = -1;                  // layer whose cache this layer reads (itself when it projects its own)
     int kv_index = -1;                  // index of that cache among the model's paged caches (a looped layer: of its first pass; pass t adds t)
     int rope_index = -1;                // index into the model's distinct rotary tables
@@ -120,7 +121,8 @@ struct LayeredModel {
     bool finalized = false;
     uint64_t weight_bytes = 0;
     // widest sizes over the layers (workspace planning)
-    int max_in = 0, max_hv = 0, max_hd = 0, max_hc = 0, max_ff = 0, max_top = 0, max_experts = 0, max_cv = 0, max_heads = 0, max_av = 0, max_qr = 0, max_q = 0;    // max_av: widest value head of a grouped-query attention layer; max_qr / max_q: widest query latent / queries expanded from one
+    int max_in = 0, max_hv = 0, max_hd = 0, max_hc = 0, max_ff = 0, max_top = 0, max_experts = 0, max_cv = 0, max_heads = 0, max_av = 0, max_qr = 0, max_q = 0, max_hp = 0, max_hq = 0, max_c = 0;    // max_av: widest value head of a grouped-query attention layer; max_qr / max_q: widest query latent / queries
+                                        // expanded from one; tensor-core latent attention: max_hp / max_hq widest plain query parts / query operand, max_c latent
     std::mutex mu;
 };
 
@@ -150,13 +152,13 @@ struct LayeredCache {
     DevBuf<int> route_sel, pair_row, pair_of, grp_off;
     PinnedBuf<float> h_logits;
     // serving precision: hi/lo halves of the activations that feed tensor-core GEMMs, and the split-K slices of their outputs
-    DevBuf<uint16_t> h_hi, h_lo, cq_hi, cq_lo, u_hi, u_lo, act_hi, act_lo, hf_hi, hf_lo;
+    DevBuf<uint16_t> h_hi, h_lo, cq_hi, cq_lo, qp_hi, qp_lo, qo_hi, qo_lo, ol_hi, ol_lo, u_hi, u_lo, act_hi, act_lo, hf_hi, hf_lo;
     DevBuf<float> gemm_out;
     DevBuf<uint16_t> gx_hi, gx_lo, ga_hi, ga_lo;        // grouped expert GEMMs: gathered inputs / activations, [experts * cap] rows
     DevBuf<int> grp_cnt;
     // tensor-core latent attention of long portions: gathered keys, their transpose, Q / P operand halves, the score block
     DevBuf<uint16_t> at_kc, at_kct, at_qhi, at_qlo, at_phi, at_plo;
-    DevBuf<float> at_part;              // grouped-query attention with key splits: partial (max, sum, values) per (row, head, split)
+    DevBuf<float> at_part;              // attention with key splits: partial (max, sum, values) per (row, head, split)
     DevBuf<float> at_s, at_o;           // at_o: grouped-query attention, the value GEMMs' outputs per key/value head before they are interleaved
 };
 

@@ -710,6 +710,279 @@ static __global__ void __launch_bounds__(kLatWarps * 32) ly_latent_attn_kernel(L
     }
 }
 
+// ---- latent attention on the tensor cores (serving precision) ---------------------------------------------------------------------
+// The query operand of a step: Q [T * H][Ep] as hi | lo halves, row (token, head) = [q~ * scale | rotated query part * scale | 0], q~ = the
+// plain query part with W_uk absorbed.  This kernel writes the scaled plain parts [T][H * D] (what the block-diagonal GEMM turns
+// into columns 0 .. C of Q) and Q's remaining columns.  cosb != nullptr: the rotated parts are turned here (queries expanded
+// from a latent); otherwise they were turned in place before.
+static __global__ void ly_latent_split_q_kernel(const float* __restrict__ q, int ldq, const int* __restrict__ row_pos, const float* __restrict__ cosb,
+                                                const float* __restrict__ sinb, int H, int D, int R, int rdims, int C, int Ep, float scale,
+                                                uint16_t* __restrict__ phi, uint16_t* __restrict__ plo, uint16_t* __restrict__ qhi,
+                                                uint16_t* __restrict__ qlo) {
+    const int row = blockIdx.x;
+    const float* qr = q + (size_t)row * ldq;
+    for (int i = threadIdx.x * 4; i < H * D; i += blockDim.x * 4) {        // D is a multiple of 8: four channels of one head
+        float v[4];
+        const float* s = qr + (size_t)(i / D) * (D + R) + i % D;
+#pragma unroll
+        for (int k = 0; k < 4; ++k) v[k] = s[k] * scale;
+        split_store_vec<4>(phi, plo, (size_t)row * H * D + i, v);
+    }
+    const int tail = Ep - C, half = rdims / 2;
+    const size_t at = (size_t)row_pos[row] * half;
+    for (int i = threadIdx.x; i < H * tail; i += blockDim.x) {
+        const int hd = i / tail, r = i % tail;
+        const float* s = qr + (size_t)hd * (D + R) + D;
+        float v = 0.f;
+        if (r < rdims && cosb != nullptr) {
+            const float cs = cosb[at + (r >> 1)], sn = sinb[at + (r >> 1)], a = s[r & ~1], b = s[r | 1];
+            v = ((r & 1) ? b * cs + a * sn : a * cs - b * sn) * scale;
+        } else if (r < R) {
+            v = s[r] * scale;
+        }
+        split_store(qhi, qlo, ((size_t)row * H + hd) * Ep + C + r, v);
+    }
+}
+
+// Decoded tokens and short portions.  One block per (row, 16 MT heads, key split): the heads are the M rows of mma.sync m16n8k16 and the
+// row's latent pages are walked tile by tile (a tile = the 64 keys of a page, two shared-memory buffers, the next tile arrives by
+// cp.async while this one is folded):
+//   scores    the eight warps share the latent's 16-channel steps (a warp keeps its query fragments in registers, hi and lo) and leave
+//             partial scores of all 64 keys in shared memory;
+//   softmax   the block's threads add the eight partials in warp order, mask (causal, window), fold the tile into the running maximum
+//             and sum of their row and write the probabilities as hi | lo halves;
+//   values    the warps share the latent's columns: O = O * correction + P . K[:, :C] from the same tile.
+// One split: the block applies the sink, normalises and writes hi | lo halves [T * H][C].  More: partial (max, sum, O) per (row,
+// head, split) for ly_gqa_merge_kernel.  NT: 8-column tiles per warp (C <= 64 NT).  C and R are multiples of 8.
+struct LatMmaArgs {
+    const uint16_t *qhi, *qlo;
+    const uint16_t* pool; const int* page_table; int pps;
+    const int *row_seq, *row_pos, *seq_slot;
+    uint16_t *ohi, *olo;
+    float* part;
+    int H, C, R, Ep, window, row_base;
+    int sink; const float* sinkv;
+};
+constexpr size_t kLatSmemMax = 227 * 1024;
+constexpr int kLatTile = kKvPage, kLatPS = kLatTile + 8;        // row stride of the probabilities (conflict-free ldmatrix)
+inline size_t lat_mma_smem(int Ep, int MT) {
+    return (size_t)2 * kLatTile * (Ep + 8) * 2 + (size_t)8 * MT * 16 * kLatTile * 4 + (size_t)2 * MT * 16 * kLatPS * 2 + (size_t)MT * 16 * 4;
+}
+template <int MT, int NT>
+static __global__ void __launch_bounds__(256) ly_latent_mma_kernel(LatMmaArgs a) {
+    constexpr int KPW = NT == 8 ? 5 : (NT == 4 ? 3 : 2);        // 16-channel steps per warp: 8 KPW >= (C + R) / 16, R <= 128
+    constexpr int MR = MT * 16, TPR = 256 / MR, CPT = kLatTile / TPR;
+    extern __shared__ __align__(16) uint8_t lsm[];
+    const int C = a.C, E = a.C + a.R, LD = a.Ep + 8, KS = (E + 15) / 16;
+    uint16_t* sk = reinterpret_cast<uint16_t*>(lsm);                                            // [2][64][LD]
+    float* red = reinterpret_cast<float*>(lsm + (size_t)2 * kLatTile * LD * 2);                 // [8][MR][64]
+    uint16_t* sph = reinterpret_cast<uint16_t*>(red + 8 * MR * kLatTile);                       // [MR][kLatPS] hi, then lo
+    uint16_t* spl = sph + MR * kLatPS;
+    float* scorr = reinterpret_cast<float*>(spl + MR * kLatPS);                                 // [MR]
+    const int tid = threadIdx.x, lane = tid & 31, wid = tid >> 5, g = lane >> 2, tq = lane & 3, mi = lane >> 3, l8 = lane & 7;
+    const int row = a.row_base + blockIdx.x, h0 = blockIdx.y * MR, split = blockIdx.z, S = gridDim.z;
+    const int pos = a.row_pos[row], slot = a.seq_slot[a.row_seq[row]];
+    const int j0 = (a.window > 0 && pos - a.window + 1 > 0) ? pos - a.window + 1 : 0;
+    const int t_lo = j0 / kLatTile, t_hi = pos / kLatTile + 1, per = (t_hi - t_lo + S - 1) / S;
+    const int tb = t_lo + split * per, te = min(t_hi, tb + per);
+    const int sr = tid / TPR, sc = (tid % TPR) * CPT, shd = h0 + sr;      // softmax: this thread's row (head) and first key of a tile
+    float m = -INFINITY, l = 0.f;
+    float o[MT][NT][4];
+#pragma unroll
+    for (int i = 0; i < MT; ++i)
+#pragma unroll
+        for (int n = 0; n < NT; ++n)
+#pragma unroll
+            for (int k = 0; k < 4; ++k) o[i][n][k] = 0.f;
+    if (tb < te) {
+        const int* pt = a.page_table + (size_t)slot * a.pps;
+        const int CH = E / 8;
+        auto load_tile = [&](int t, int buf) {
+            const uint16_t* src = a.pool + (size_t)pt[t] * kLatTile * E;
+            uint16_t* dst = sk + (size_t)buf * kLatTile * LD;
+            for (int i = tid; i < kLatTile * CH; i += 256) {
+                const int key = i / CH, c = i - key * CH;
+                if (t * kLatTile + key <= pos) cp_async16(dst + key * LD + c * 8, src + (size_t)i * 8);
+                else *reinterpret_cast<uint4*>(dst + key * LD + c * 8) = make_uint4(0u, 0u, 0u, 0u);
+            }
+            cp_async_commit();
+        };
+        load_tile(tb, 0);
+        // the columns behind E meet zero query channels and must be finite
+        for (int i = tid; i < 2 * kLatTile; i += 256)
+            for (int c = E; c < LD; ++c) sk[(size_t)i * LD + c] = 0;
+        uint32_t qf[MT][KPW][2][4];
+#pragma unroll
+        for (int i = 0; i < MT; ++i)
+#pragma unroll
+            for (int s = 0; s < KPW; ++s) {
+                const int ks = wid + 8 * s;
+#pragma unroll
+                for (int k = 0; k < 4; ++k) {
+                    const int hd = h0 + i * 16 + g + (k & 1) * 8;
+                    const size_t at = ((size_t)row * a.H + hd) * a.Ep + ks * 16 + (k >> 1) * 8 + 2 * tq;
+                    const bool ok = ks < KS && hd < a.H;
+                    qf[i][s][0][k] = ok ? *reinterpret_cast<const uint32_t*>(a.qhi + at) : 0u;
+                    qf[i][s][1][k] = ok ? *reinterpret_cast<const uint32_t*>(a.qlo + at) : 0u;
+                }
+            }
+        for (int t = tb; t < te; ++t) {
+            const uint16_t* kt = sk + (size_t)((t - tb) & 1) * kLatTile * LD;
+            cp_async_wait<0>();
+            __syncthreads();                    // the tile has landed; nobody reads the other buffer any more
+            if (t + 1 < te) load_tile(t + 1, (t + 1 - tb) & 1);
+#pragma unroll
+            for (int half = 0; half < 2; ++half) {
+                float acc[MT][4][4] = {};
+#pragma unroll
+                for (int s = 0; s < KPW; ++s) {
+                    const int ks = wid + 8 * s;
+                    if (ks < KS) {
+#pragma unroll
+                        for (int jp = 0; jp < 2; ++jp) {
+                            uint32_t b[4];
+                            ldmatrix_x4(b, kt + (size_t)(half * 32 + jp * 16 + (mi >> 1) * 8 + l8) * LD + ks * 16 + (mi & 1) * 8);
+#pragma unroll
+                            for (int i = 0; i < MT; ++i)
+#pragma unroll
+                                for (int p = 0; p < 2; ++p) {
+                                    mma_bf16_16816(acc[i][2 * jp], qf[i][s][p], b[0], b[1]);
+                                    mma_bf16_16816(acc[i][2 * jp + 1], qf[i][s][p], b[2], b[3]);
+                                }
+                        }
+                    }
+                }
+                // 8-key chunks of a row sit at chunk ^ (row & 7): conflict-free stores
+#pragma unroll
+                for (int i = 0; i < MT; ++i)
+#pragma unroll
+                    for (int n = 0; n < 4; ++n) {
+                        const int ch = ((half * 4 + n) ^ g) * 8 + 2 * tq;
+                        float* r0 = red + (size_t)(wid * MR + i * 16 + g) * kLatTile + ch;
+                        *reinterpret_cast<float2*>(r0) = make_float2(acc[i][n][0], acc[i][n][1]);
+                        *reinterpret_cast<float2*>(r0 + 8 * kLatTile) = make_float2(acc[i][n][2], acc[i][n][3]);
+                    }
+            }
+            __syncthreads();
+            {
+                float v[CPT] = {};
+                const float* rp = red + (size_t)sr * kLatTile + (((sc >> 3) ^ (sr & 7)) << 3) + (sc & 7);
+#pragma unroll
+                for (int w = 0; w < 8; ++w)
+#pragma unroll
+                    for (int i = 0; i < CPT; i += 4) {
+                        const float4 x = *reinterpret_cast<const float4*>(rp + (size_t)w * MR * kLatTile + i);
+                        v[i] += x.x; v[i + 1] += x.y; v[i + 2] += x.z; v[i + 3] += x.w;
+                    }
+                float mx = -INFINITY;
+#pragma unroll
+                for (int i = 0; i < CPT; ++i) {
+                    const int j = t * kLatTile + sc + i;
+                    if (j < j0 || j > pos) v[i] = -INFINITY;
+                    mx = fmaxf(mx, v[i]);
+                }
+#pragma unroll
+                for (int d = TPR / 2; d > 0; d >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
+                const float mn = fmaxf(m, mx), corr = expf(m - mn);      // every tile of the walk holds a visible key: mn is finite
+                float ps = 0.f;
+                uint32_t ph[CPT / 2], pl[CPT / 2];
+#pragma unroll
+                for (int i = 0; i < CPT; i += 2) {
+                    const float p0 = expf(v[i] - mn), p1 = expf(v[i + 1] - mn);
+                    ps += p0 + p1;
+                    ph[i / 2] = pack_bf16x2(p0, p1);
+                    pl[i / 2] = pack_bf16x2(p0 - bf16lo(ph[i / 2]), p1 - bf16hi(ph[i / 2]));
+                }
+#pragma unroll
+                for (int d = TPR / 2; d > 0; d >>= 1) ps += __shfl_xor_sync(0xffffffffu, ps, d);
+                l = l * corr + ps;
+                m = mn;
+#pragma unroll
+                for (int i = 0; i < CPT / 2; ++i) {
+                    *reinterpret_cast<uint32_t*>(sph + sr * kLatPS + sc + 2 * i) = ph[i];
+                    *reinterpret_cast<uint32_t*>(spl + sr * kLatPS + sc + 2 * i) = pl[i];
+                }
+                if (sc == 0) scorr[sr] = corr;
+            }
+            __syncthreads();
+#pragma unroll
+            for (int i = 0; i < MT; ++i) {
+                const float c0 = scorr[i * 16 + g], c1 = scorr[i * 16 + g + 8];
+#pragma unroll
+                for (int n = 0; n < NT; ++n) { o[i][n][0] *= c0; o[i][n][1] *= c0; o[i][n][2] *= c1; o[i][n][3] *= c1; }
+            }
+#pragma unroll
+            for (int kk = 0; kk < kLatTile / 16; ++kk) {
+                uint32_t pa[MT][2][4];
+#pragma unroll
+                for (int i = 0; i < MT; ++i) {
+                    ldmatrix_x4(pa[i][0], sph + (size_t)(i * 16 + (mi & 1) * 8 + l8) * kLatPS + kk * 16 + (mi >> 1) * 8);
+                    ldmatrix_x4(pa[i][1], spl + (size_t)(i * 16 + (mi & 1) * 8 + l8) * kLatPS + kk * 16 + (mi >> 1) * 8);
+                }
+                const uint16_t* vrow = kt + (size_t)(kk * 16 + (mi & 1) * 8 + l8) * LD;
+#pragma unroll
+                for (int n = 0; n < NT; n += 2) {
+                    const int col = (wid * NT + n) * 8;
+                    if (col < C) {
+                        uint32_t b[4];
+                        if (NT == 1) {
+                            uint32_t b2[2];
+                            ldmatrix_x2_trans(b2, vrow + col);          // lanes 0 - 15 name the rows
+                            b[0] = b2[0]; b[1] = b2[1]; b[2] = b[3] = 0u;
+                        } else {
+                            ldmatrix_x4_trans(b, vrow + col + (mi >> 1) * 8);
+                        }
+#pragma unroll
+                        for (int i = 0; i < MT; ++i)
+#pragma unroll
+                            for (int p = 0; p < 2; ++p) {
+                                mma_bf16_16816(o[i][n], pa[i][p], b[0], b[1]);
+                                if (NT > 1) mma_bf16_16816(o[i][n + (NT > 1 ? 1 : 0)], pa[i][p], b[2], b[3]);
+                            }
+                    }
+                }
+            }
+        }
+    }
+    float* part = a.part;
+    if (S == 1) {
+        if (sc == 0) {
+            const float sv = (a.sink && a.sinkv && shd < a.H) ? a.sinkv[shd] : 0.f;
+            const float M = a.sink ? fmaxf(m, sv) : m, f = expf(m - M);
+            scorr[sr] = f / (l * f + (a.sink ? expf(sv - M) : 0.f));
+        }
+        __syncthreads();
+    } else {
+        if (sc == 0 && shd < a.H) {
+            float* pp = part + (((size_t)blockIdx.x * a.H + shd) * S + split) * (C + 2);
+            pp[0] = m; pp[1] = l;
+        }
+        if (tb >= te) return;
+    }
+#pragma unroll
+    for (int i = 0; i < MT; ++i)
+#pragma unroll
+        for (int hh = 0; hh < 2; ++hh) {
+            const int r = i * 16 + g + hh * 8, hd = h0 + r;
+            if (hd >= a.H) continue;
+            const float f = S == 1 ? scorr[r] : 1.f;
+#pragma unroll
+            for (int n = 0; n < NT; ++n) {
+                const int col = (wid * NT + n) * 8 + 2 * tq;
+                if (col >= C) continue;
+                const float x = o[i][n][2 * hh] * f, y = o[i][n][2 * hh + 1] * f;
+                if (S == 1) {
+                    const size_t at = ((size_t)row * a.H + hd) * C + col;
+                    const uint32_t h = pack_bf16x2(x, y);
+                    *reinterpret_cast<uint32_t*>(a.ohi + at) = h;
+                    *reinterpret_cast<uint32_t*>(a.olo + at) = pack_bf16x2(x - bf16lo(h), y - bf16hi(h));
+                } else {
+                    *reinterpret_cast<float2*>(part + (((size_t)blockIdx.x * a.H + hd) * S + split) * (C + 2) + 2 + col) = make_float2(x, y);
+                }
+            }
+        }
+}
+
 // ---- latent attention for long portions on the tensor-core GEMM (serving precision) ---------------------------------------------
 // A block of consecutive query rows of ONE sequence and the keys its window can reach [k_lo, k_lo + nk):
 //   S = Q~ . Kc^T (one GEMM: rows = (token, head) pairs -- every head of a token meets the same latent keys),
@@ -1045,7 +1318,8 @@ static __global__ void __launch_bounds__(kGqaWarps * 32) ly_gqa_attn_kernel(GqaA
         }
     }
 }
-// Folds the key splits of ly_gqa_attn_kernel in split order (and the sink): one block per (row, head).
+// Folds the key splits of ly_gqa_attn_kernel (or ly_latent_mma_kernel) in split order (and the sink): one block per (row, head).
+// out == nullptr: only the halves are wanted.
 static __global__ void ly_gqa_merge_kernel(const float* __restrict__ part, int S, int H, int Dv, int sink, const float* __restrict__ sinkv, int row_base,
                                            float* __restrict__ out, uint16_t* __restrict__ ohi, uint16_t* __restrict__ olo) {
     const int row = row_base + blockIdx.x, hd = blockIdx.y;
@@ -1067,7 +1341,7 @@ static __global__ void ly_gqa_merge_kernel(const float* __restrict__ part, int S
             if (ms != -INFINITY) t += pp[(size_t)s * (Dv + 2) + 2 + c] * expf(ms - M);
         }
         t *= inv;
-        out[ob + c] = t;
+        if (out != nullptr) out[ob + c] = t;
         split_store(ohi, olo, ob + c, t);
     }
 }

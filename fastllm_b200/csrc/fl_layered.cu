@@ -606,9 +606,11 @@ void layered_finalize(LayeredModel& m) {
         }
         map(m.head, m.V, m.W, m.tm_head, m.tc_head);
     }
-    // the norm of the sum parks a row in shared memory: above the default 48 KB the kernels are told so once
-    if (m.cfg.post_sum_norm && (size_t)m.W * 4 > 48 * 1024) {
-        FL_CHECK((size_t)m.W * 4 <= 200 * 1024, FL_ERR_UNSUPPORTED, "a norm of the sum is built for widths up to 51200");
+    // the norms behind a sublayer park a row in shared memory: above the default 48 KB the kernels are told so once
+    if (!m.cfg.no_post_norm && (size_t)m.W * 4 > 48 * 1024) {
+        FL_CHECK((size_t)m.W * 4 <= 200 * 1024, FL_ERR_UNSUPPORTED, "norms behind a sublayer are built for widths up to 51200");
+        FL_CUDA(cudaFuncSetAttribute(ly_post_norm_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, m.W * 4));
+        FL_CUDA(cudaFuncSetAttribute(ly_post_norm_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, m.W * 4));
         FL_CUDA(cudaFuncSetAttribute(ly_sum_norm_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, m.W * 4));
         FL_CUDA(cudaFuncSetAttribute(ly_sum_norm_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, m.W * 4));
     }
@@ -801,22 +803,33 @@ static void gemm(LaunchCtx& lc, const char* tag, const float* A, int lda, const 
     else launch(lc, tag, (uint64_t)N * K * 2, ly_gemm_kernel<float>, grid, dim3(256), 0, g);
 }
 // Y[R, N] = A[R, K] . Wt[N, K]^T on the tensor cores when the matrix has a descriptor (serving precision; A as hi | lo halves),
-// else on the exact kernel.  Split-K slices of the tensor-core GEMM are folded in slice order.
-static void gemm_tc_or_exact(fl_cache& c, LaunchCtx& lc, const char* tag, const float* A, const uint16_t* ahi, const uint16_t* alo, const uint16_t* Wt,
-                             const CUtensorMap& tm, bool tc, int N, int K, float* Y, int R) {
-    if (R <= 0) return;
-    if (!tc || ahi == nullptr) { gemm(lc, tag, A, K, Wt, N, K, Y, N, R); return; }
+// else on the exact kernel.  A tensor-core GEMM of few rows may leave split-K slices in the shared scratch: the caller hands them to
+// the kernel that reads the result next (before another split GEMM runs), which folds them in slice order.
+static Slices gemm_slices(fl_cache& c, LaunchCtx& lc, const char* tag, const float* A, const uint16_t* ahi, const uint16_t* alo, const uint16_t* Wt,
+                          const CUtensorMap& tm, bool tc, int N, int K, float* Y, int R) {
+    if (R <= 0) return Slices{Y, 1, 0};
+    if (!tc || ahi == nullptr) { gemm(lc, tag, A, K, Wt, N, K, Y, N, R); return Slices{Y, 1, 0}; }
     LayeredCache& y = *c.ly;
     const int ks_plan = R <= 128 ? pick_ksplit((N + 127) / 128, (K + 63) / 64, R) : 1;
     float* out = ks_plan == 1 ? Y : y.gemm_out.p;
     FL_CHECK(ks_plan == 1 || (size_t)ks_plan * R * N <= y.gemm_out.n, FL_ERR_STATE, "internal: split-K scratch too small");
     const int ks = dense_gemm(c, lc, tag, R, N, K, tm, out, ahi, alo);
     FL_CHECK(ks == ks_plan, FL_ERR_STATE, "internal: split-K plan mismatch");
-    if (ks > 1) {
-        const size_t n = (size_t)R * N;
-        launch(lc, "sum_slices", 0, ly_sum_slices_kernel, dim3((unsigned)std::min<size_t>(4 * kNumSMs, (n + 255) / 256)), dim3(256), 0,
-               (const float*)out, ks, n, n, Y);
-    }
+    return Slices{out, ks, (size_t)R * N};
+}
+// the same with the slices folded into Y
+static void gemm_tc_or_exact(fl_cache& c, LaunchCtx& lc, const char* tag, const float* A, const uint16_t* ahi, const uint16_t* alo, const uint16_t* Wt,
+                             const CUtensorMap& tm, bool tc, int N, int K, float* Y, int R) {
+    const Slices s = gemm_slices(c, lc, tag, A, ahi, alo, Wt, tm, tc, N, K, Y, R);
+    if (s.n > 1)
+        launch(lc, "sum_slices", 0, ly_sum_slices_kernel, dim3((unsigned)std::min<size_t>(4 * kNumSMs, (s.stride + 255) / 256)), dim3(256), 0,
+               s.p, s.n, s.stride, s.stride, Y);
+}
+// feed-forward activation of `rows` rows (see ly_glu_kernel)
+static void launch_glu(LaunchCtx& lc, const Slices& gu, int rows, int F, float limit, int act, const float* bias, float* out, uint16_t* hi, uint16_t* lo) {
+    if (rows <= 0) return;
+    if (F % 4 == 0) launch(lc, "glu", 0, ly_glu_kernel<4>, dim3(rows, (F + 1023) / 1024), dim3(256), 0, gu, F, limit, act, bias, out, hi, lo);
+    else launch(lc, "glu", 0, ly_glu_kernel<1>, dim3(rows, (F + 255) / 256), dim3(256), 0, gu, F, limit, act, bias, out, hi, lo);
 }
 
 static void gemm_groups(LaunchCtx& lc, const char* tag, const LyGemm& g, int groups, int max_rows) {
@@ -1143,10 +1156,11 @@ void layered_forward(fl_cache& c, const int* slots, const int* counts, int n, co
     for (int i = 0; i < n; ++i) c.slot_len[slots[i]] += counts[i];
 }
 
-// One mixer over all rows of the step (`pass`: which pass of a loop, 0 elsewhere -- its own cache and state): reads its columns of the projected buffer y.proj (row stride lw.n_in), its cache pages / state
+// One mixer over all rows of the step (`pass`: which pass of a loop, 0 elsewhere -- its own cache and state): reads its columns of the projected buffer y.proj (row stride lw.n_in; `in`: the same as
+// the GEMM left it, perhaps in slices), its cache pages / state
 // slots, and leaves the mixer's inner output (what its output projection reads) in y.u with the hi | lo halves when that
 // projection runs on the tensor cores.
-static void run_mixer(fl_cache& c, LaunchCtx& lc, const StepTab& st, const LayeredLayerW& lw, int pass, const int* slots, const int* counts, int n,
+static void run_mixer(fl_cache& c, LaunchCtx& lc, const StepTab& st, const LayeredLayerW& lw, const Slices& in, int pass, const int* slots, const int* counts, int n,
                       const int* h_row0, const int* h_pos0) {
     const LayeredModel& m = *c.lm;
     LayeredCache& y = *c.ly;
@@ -1249,16 +1263,22 @@ static void run_mixer(fl_cache& c, LaunchCtx& lc, const StepTab& st, const Layer
     } else {
         const int R = d.rot_dim, C = d.kv_rank, Q = d.q_rank;
         LatentAppendArgs aa{y.proj.p, lw.n_in, lw.off_q, lw.off_dkv, lw.dkv_norm, eps, y.kv_pool[kv_index], y.page_table.p, c.pages_per_seq,
-                            st.row_seq, st.row_pos, st.seq_slot, y.rope_cos[lw.rope_index].p, y.rope_sin[lw.rope_index].p, H, D, R, C, d.rot_dims, lw.off_q, Q, lw.dq_norm, y.cq.p,
-                            lw.tc_uq ? y.cq_hi.p : (uint16_t*)nullptr, y.cq_lo.p};
-        if (m.f32) launch(lc, "latent_append", 0, ly_latent_append_kernel<float>, dim3(Ti), dim3(128), 0, aa);
-        else launch(lc, "latent_append", 0, ly_latent_append_kernel<uint16_t>, dim3(Ti), dim3(128), 0, aa);
+                            st.row_seq, st.row_pos, st.seq_slot, y.rope_cos[lw.rope_index].p, y.rope_sin[lw.rope_index].p, H, D, R, C, d.rot_dims, lw.off_q, Q, lw.dq_norm, lw.tc_uq ? (float*)nullptr : y.cq.p,
+                            lw.tc_uq ? y.cq_hi.p : (uint16_t*)nullptr, y.cq_lo.p, in, lw.off_g, d.out_gate ? H * Dv : 0};
+        const int ath = Ti <= 2 * kNumSMs ? std::min(1024, std::max(128, (Q + C + 31) / 32 * 32)) : 128;
+        if (m.f32) launch(lc, "latent_append", 0, ly_latent_append_kernel<float>, dim3(Ti), dim3(ath), 0, aa);
+        else launch(lc, "latent_append", 0, ly_latent_append_kernel<uint16_t>, dim3(Ti), dim3(ath), 0, aa);
         // queries [T][H][D + R]: columns of the projected buffer, or expanded from the normed query latent
         float* q = y.proj.p + lw.off_q;
         int ldq = lw.n_in;
+        Slices qs{q, 1, 0};
         if (Q > 0) {
             q = y.qx.p; ldq = H * (D + R);
-            gemm_tc_or_exact(c, lc, "gemm_q_up", y.cq.p, y.cq_hi.p, y.cq_lo.p, lw.uq, lw.tm_uq, lw.tc_uq, ldq, Q, q, Ti);
+            qs = gemm_slices(c, lc, "gemm_q_up", y.cq.p, y.cq_hi.p, y.cq_lo.p, lw.uq, lw.tm_uq, lw.tc_uq, ldq, Q, q, Ti);
+            if (qs.n > 1 && !lw.lat_tc) {
+                launch(lc, "sum_slices", 0, ly_sum_slices_kernel, dim3((unsigned)std::min<size_t>(4 * kNumSMs, (qs.stride + 255) / 256)), dim3(256), 0, qs.p, qs.n,
+                       qs.stride, qs.stride, q);
+            }
             if (d.rot_dims > 0 && !lw.lat_tc)
                 launch(lc, "rotate_q", 0, ly_rotate_q_kernel, dim3(Ti), dim3(128), 0, q, ldq, st.row_pos, (const float*)y.rope_cos[lw.rope_index].p,
                        (const float*)y.rope_sin[lw.rope_index].p, H, D, R, d.rot_dims);
@@ -1282,7 +1302,7 @@ static void run_mixer(fl_cache& c, LaunchCtx& lc, const StepTab& st, const Layer
             // gate) -> the output projection's operand
             const int Ep = (C + R + 63) / 64 * 64;
             const bool turn = Q > 0 && d.rot_dims > 0;
-            launch(lc, "latent_split_q", 0, ly_latent_split_q_kernel, dim3(Ti), dim3(256), 0, (const float*)q, ldq, st.row_pos,
+            launch(lc, "latent_split_q", 0, ly_latent_split_q_kernel, dim3(Ti, Ti <= kNumSMs ? 4 : 1), dim3(256), 0, qs, ldq, st.row_pos,
                    turn ? (const float*)y.rope_cos[lw.rope_index].p : (const float*)nullptr, (const float*)y.rope_sin[lw.rope_index].p, H, D, R, d.rot_dims, C, Ep,
                    d.scale, y.qp_hi.p, y.qp_lo.p, y.qo_hi.p, y.qo_lo.p);
             dense_gemm_blocks(c, lc, "gemm_q_absorb", Ti, H, C, D, lw.tm_uk, y.qp_hi.p, y.qp_lo.p, y.qo_hi.p, y.qo_lo.p, H * Ep, Ep);
@@ -1404,6 +1424,24 @@ static void enqueue_step(fl_cache& c, LaunchCtx& lc, const StepTab& st, const in
             launch(lc, "join", 0, ly_join_kernel<1>, dim3(Ti), dim3(nthr), 0, y.x.p, (const float*)y.y.p, y2, wa, wb, gz, gate_bias, y.xs.p, hist_stride,
                    hist_slot, dw, wnext, eps, W, plain, y.h.p, hhi, hlo);
     };
+    // a sublayer's result (still in split-K slices, perhaps) is normed and joins the stream
+    // (hout == nullptr: the next sublayer's first matrix reads the hi | lo halves alone)
+    auto post_norm = [&](const Slices& yv, const float* yb, const float* wb, const float* wnext, const float* ls, const float* x0, const float* step, int split,
+                         float* hout) {
+        if (W % 4 == 0)
+            launch(lc, "post_norm", 0, ly_post_norm_kernel<4>, dim3(Ti), dim3(std::min(Ti <= kNumSMs ? 1024 : 256, std::max(32, (W / 4 + 31) / 32 * 32))), (size_t)W * 4,
+                   y.x.p, yv, yb, wb, wnext, ls, x0, step, eps, W, plain, split, hout, hhi, hlo);
+        else
+            launch(lc, "post_norm", 0, ly_post_norm_kernel<1>, dim3(Ti), dim3(nthr), (size_t)W * 4, y.x.p, yv, yb, wb, wnext, ls, x0, step, eps, W, plain, split, hout,
+                   hhi, hlo);
+    };
+    // the other arrangements read the folded rows
+    auto fold = [&](Slices& s) {
+        if (s.n > 1)
+            launch(lc, "sum_slices", 0, ly_sum_slices_kernel, dim3((unsigned)std::min<size_t>(4 * kNumSMs, (s.stride + 255) / 256)), dim3(256), 0, s.p, s.n, s.stride,
+                   s.stride, y.y.p);
+        s = Slices{y.y.p, 1, 0};
+    };
     const int n_runs = (int)m.runs.size();
     for (int run = 0; run < n_runs; ++run) {
         const int li = m.runs[run].layer, pass = m.runs[run].pass;
@@ -1412,15 +1450,23 @@ static void enqueue_step(fl_cache& c, LaunchCtx& lc, const StepTab& st, const in
         const int H = d.heads, Dv = d.vdim;
         sublayer_front(lw, run, 0);
         if (shifted) shift_front(lw, run);
-        gemm_tc_or_exact(c, lc, "gemm_mix_in", shifted ? (const float*)y.hc.p : sub_in, hhi, hlo, lw.w_in, lw.tm_in, lw.tc_in, lw.n_in, W, y.proj.p, Ti);
-        run_mixer(c, lc, st, lw, pass, slots, counts, n, h_row0, h_pos0);
-        gemm_tc_or_exact(c, lc, "gemm_mix_out", y.u.p, uhi, ulo, lw.w_o, lw.tm_o, lw.tc_o, W, H * Dv, y.y.p, Ti);
+        Slices in = gemm_slices(c, lc, "gemm_mix_in", shifted ? (const float*)y.hc.p : sub_in, hhi, hlo, lw.w_in, lw.tm_in, lw.tc_in, lw.n_in, W, y.proj.p, Ti);
+        if (in.n > 1 && !(d.mixer == FL_MIXER_LATENT_ATTN && d.q_rank > 0)) {        // only that mixer folds the slices itself
+            launch(lc, "sum_slices", 0, ly_sum_slices_kernel, dim3((unsigned)std::min<size_t>(4 * kNumSMs, (in.stride + 255) / 256)), dim3(256), 0, in.p, in.n, in.stride,
+                   in.stride, y.proj.p);
+            in = Slices{y.proj.p, 1, 0};
+        }
+        run_mixer(c, lc, st, lw, in, pass, slots, counts, n, h_row0, h_pos0);
+        Slices mix = gemm_slices(c, lc, "gemm_mix_out", y.u.p, uhi, ulo, lw.w_o, lw.tm_o, lw.tc_o, W, H * Dv, y.y.p, Ti), ff{y.y.p, 1, 0};
+        if (!post || sum_norm || lw.side) fold(mix);
         if (lw.side) {
             const LayeredLayerW& sw = *lw.side;
-            run_mixer(c, lc, st, sw, pass, slots, counts, n, h_row0, h_pos0);
+            run_mixer(c, lc, st, sw, in, pass, slots, counts, n, h_row0, h_pos0);
             gemm_tc_or_exact(c, lc, "gemm_mix_out", y.u.p, uhi, ulo, sw.w_o, sw.tm_o, sw.tc_o, W, sw.d.heads * sw.d.vdim, y.y2.p, Ti);
         }
         const bool last = run + 1 == n_runs, has_ff = d.ffn != FL_FFN_NONE;
+        // whether the next sublayer (the feed-forward; the next run's mixer) takes its input as hi | lo halves only
+        const bool ff_halves = lw.tc_gu && d.ffn == FL_FFN_DENSE && !canon && !gated, mix_halves = !last && m.layers[m.runs[run + 1].layer].tc_in && !canon && !gated;
         const float* next1 = (pre && !last) ? m.layers[m.runs[run + 1].layer].norm1 : nullptr;
         const int more = last ? 0 : split_x;               // whether another sublayer reads x after this layer
         // what joins the stream between this layer and the next run when that one starts a pass of the loop
@@ -1432,9 +1478,8 @@ static void enqueue_step(fl_cache& c, LaunchCtx& lc, const StepTab& st, const in
             sum_norm_join(nullptr, lw.side ? (const float*)y.y2.p : (const float*)nullptr, lw.side ? d.out_scale : 1.f, lw.side ? lw.side->d.out_scale : 0.f,
                           lw.norm1b, (has_ff || !shifted) ? (has_ff ? split_x : more) : 0);
         else if (post)
-            launch(lc, "post_norm", 0, ly_post_norm_kernel, dim3(Ti), dim3(nthr), 0, y.x.p, (const float*)y.y.p, (const float*)nullptr, (const float*)lw.norm1b,
-                   has_ff ? (const float*)lw.norm2 : next1, (const float*)lw.ls1, has_ff ? (const float*)nullptr : again, has_ff ? (const float*)nullptr : pstep, eps, W, plain,
-                   has_ff ? split_x : more, y.h.p, hhi, hlo);
+            post_norm(mix, nullptr, lw.norm1b, has_ff ? (const float*)lw.norm2 : next1, lw.ls1, has_ff ? nullptr : again, has_ff ? nullptr : pstep, has_ff ? split_x : more,
+                      (has_ff ? ff_halves : mix_halves) ? nullptr : y.h.p);
         else
             join(lw.side ? (const float*)y.y2.p : (const float*)nullptr, lw.pair_wa, lw.pair_wb, lw.rg1b, (depth && !has_ff) ? li + 1 : -1, lw.dwa,
                  has_ff ? (const float*)lw.norm2 : next1);
@@ -1442,10 +1487,10 @@ static void enqueue_step(fl_cache& c, LaunchCtx& lc, const StepTab& st, const in
         sublayer_front(lw, run, 1);
         const int F = d.ff, act = d.ffn_act, GF = act == FL_ACT_RELU2 ? F : 2 * F;
         if (d.ffn == FL_FFN_DENSE) {
-            gemm_tc_or_exact(c, lc, "gemm_ff_in", sub_in, hhi, hlo, lw.w_gu, lw.tm_gu, lw.tc_gu, GF, W, y.gu.p, Ti);
-            launch(lc, "glu", 0, ly_glu_kernel, dim3(std::min(4 * kNumSMs, (Ti * F + 255) / 256)), dim3(256), 0, (const float*)y.gu.p, F, d.limit,
-                   act, (const float*)lw.b_gu, (const int*)nullptr, Ti, lw.tc_down ? (float*)nullptr : y.act.p, lw.tc_down ? ahi : (uint16_t*)nullptr, alo);
-            gemm_tc_or_exact(c, lc, "gemm_ff_out", y.act.p, ahi, alo, lw.w_down, lw.tm_down, lw.tc_down, W, F, y.y.p, Ti);
+            const Slices gu = gemm_slices(c, lc, "gemm_ff_in", sub_in, hhi, hlo, lw.w_gu, lw.tm_gu, lw.tc_gu, GF, W, y.gu.p, Ti);
+            launch_glu(lc, gu, Ti, F, d.limit, act, lw.b_gu, lw.tc_down ? (float*)nullptr : y.act.p, lw.tc_down ? ahi : (uint16_t*)nullptr, alo);
+            ff = gemm_slices(c, lc, "gemm_ff_out", y.act.p, ahi, alo, lw.w_down, lw.tm_down, lw.tc_down, W, F, y.y.p, Ti);
+            if (!post || sum_norm) fold(ff);
         } else {
             const int E = d.experts, top = d.top, P = Ti * top;
             if (d.router == FL_ROUTER_SIGMOID_GROUPS)
@@ -1458,9 +1503,8 @@ static void enqueue_step(fl_cache& c, LaunchCtx& lc, const StepTab& st, const in
             const float* sh = nullptr;
             if (d.shared_ff > 0) {          // the always-on expert first: its split-K scratch is free again before the routed experts run
                 const int Fs = d.shared_ff;
-                gemm_tc_or_exact(c, lc, "gemm_shared_in", sub_in, hhi, hlo, lw.s_gu, lw.tm_sgu, lw.tc_sgu, 2 * Fs, W, y.sh_gu.p, Ti);
-                launch(lc, "glu", 0, ly_glu_kernel, dim3(std::min(4 * kNumSMs, (Ti * Fs + 255) / 256)), dim3(256), 0, (const float*)y.sh_gu.p, Fs,
-                       d.shared_limit, 0, (const float*)nullptr, (const int*)nullptr, Ti, lw.tc_sdown ? (float*)nullptr : y.sh_act.p, lw.tc_sdown ? ahi : (uint16_t*)nullptr, alo);
+                const Slices gu = gemm_slices(c, lc, "gemm_shared_in", sub_in, hhi, hlo, lw.s_gu, lw.tm_sgu, lw.tc_sgu, 2 * Fs, W, y.sh_gu.p, Ti);
+                launch_glu(lc, gu, Ti, Fs, d.shared_limit, 0, nullptr, lw.tc_sdown ? (float*)nullptr : y.sh_act.p, lw.tc_sdown ? ahi : (uint16_t*)nullptr, alo);
                 gemm_tc_or_exact(c, lc, "gemm_shared_out", y.sh_act.p, ahi, alo, lw.s_down, lw.tm_sdown, lw.tc_sdown, W, Fs, y.sh_o.p, Ti);
                 sh = y.sh_o.p;
             }
@@ -1469,8 +1513,7 @@ static void enqueue_step(fl_cache& c, LaunchCtx& lc, const StepTab& st, const in
                 // many rows: every expert over all rows on the tensor cores, kept where the row picked it (ascending expert order)
                 for (int e = 0; e < E; ++e) {
                     dense_gemm(c, lc, "gemm_tc_moe_in", Ti, GF, W, lw.tm_egu[e], y.gu.p, hhi, hlo);
-                    launch(lc, "glu", 0, ly_glu_kernel, dim3(std::min(4 * kNumSMs, (Ti * F + 255) / 256)), dim3(256), 0, (const float*)y.gu.p, F, d.limit,
-                           act, (const float*)nullptr, (const int*)nullptr, Ti, (float*)nullptr, ahi, alo);
+                    launch_glu(lc, Slices{y.gu.p, 1, 0}, Ti, F, d.limit, act, nullptr, nullptr, ahi, alo);
                     dense_gemm(c, lc, "gemm_tc_moe_out", Ti, W, F, lw.tm_edown[e], y.eo.p, ahi, alo);
                     launch(lc, "moe_accum", 0, ly_moe_accum_kernel, gw, dim3(256), 0, (const float*)y.eo.p, (const int*)y.route_sel.p,
                            (const float*)y.route_w.p, top, e, (const float*)nullptr, e == 0 ? 1 : 0, W, y.y.p);
@@ -1498,8 +1541,7 @@ static void enqueue_step(fl_cache& c, LaunchCtx& lc, const StepTab& st, const in
                 } else {
                     LyGemm g1{sub_in, 0, W, y.pair_row.p, lw.w_gu, (long long)GF * W, GF, W, y.gu.p, 0, GF, y.grp_off.p, P};
                     gemm_groups(lc, "gemm_moe_in", g1, E, P);
-                    launch(lc, "glu", 0, ly_glu_kernel, dim3(std::min(4 * kNumSMs, (P * F + 255) / 256)), dim3(256), 0, (const float*)y.gu.p, F, d.limit,
-                           act, (const float*)nullptr, (const int*)nullptr, P, y.act.p, (uint16_t*)nullptr, (uint16_t*)nullptr);
+                    launch_glu(lc, Slices{y.gu.p, 1, 0}, P, F, d.limit, act, nullptr, y.act.p, nullptr, nullptr);
                     LyGemm g2{y.act.p, 0, F, nullptr, lw.w_down, (long long)W * F, W, F, y.eo.p, 0, W, y.grp_off.p, P};
                     gemm_groups(lc, "gemm_moe_out", g2, E, P);
                     launch(lc, "moe_combine", 0, ly_moe_combine_kernel, gw, dim3(256), 0, (const float*)y.eo.p, (const int*)y.pair_of.p,
@@ -1510,8 +1552,7 @@ static void enqueue_step(fl_cache& c, LaunchCtx& lc, const StepTab& st, const in
         if (sum_norm)
             sum_norm_join(lw.b_down, nullptr, 1.f, 0.f, lw.norm2b, shifted ? 0 : more);
         else if (post)
-            launch(lc, "post_norm", 0, ly_post_norm_kernel, dim3(Ti), dim3(nthr), 0, y.x.p, (const float*)y.y.p, (const float*)lw.b_down, (const float*)lw.norm2b,
-                   next1, (const float*)lw.ls2, again, pstep, eps, W, plain, more, y.h.p, hhi, hlo);
+            post_norm(ff, lw.b_down, lw.norm2b, next1, lw.ls2, again, pstep, more, mix_halves ? nullptr : y.h.p);
         else
             join(nullptr, nullptr, nullptr, lw.rg2b, depth ? li + 1 : -1, lw.dwa, next1);
     }

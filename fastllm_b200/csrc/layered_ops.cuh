@@ -48,6 +48,21 @@ __device__ __forceinline__ float block_sum(float v, float* red) {      // red: >
     return red[32];
 }
 
+__device__ __forceinline__ float2 block_sum2(float2 v, float2* red) {     // two sums at once; red: >= 33 pairs of shared memory
+    v.x = warp_sum(v.x); v.y = warp_sum(v.y);
+    const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5, nw = (blockDim.x + 31) >> 5;
+    __syncthreads();
+    if (lane == 0) red[wid] = v;
+    __syncthreads();
+    if (wid == 0) {
+        float2 t = lane < nw ? red[lane] : make_float2(0.f, 0.f);
+        t.x = warp_sum(t.x); t.y = warp_sum(t.y);
+        if (lane == 0) red[32] = t;
+    }
+    __syncthreads();
+    return red[32];
+}
+
 __device__ __forceinline__ float sigmoidf_(float z) { return 1.f / (1.f + expf(-z)); }
 
 // The tensor-core GEMMs take an f32 activation as two bf16 halves, v = hi + lo (about 16 mantissa bits): written by the kernel
@@ -93,6 +108,22 @@ __device__ __forceinline__ void split_store_vec(uint16_t* hi, uint16_t* lo, size
     } else {
 #pragma unroll
         for (int k = 0; k < V; ++k) { hi[i + k] = h[k]; lo[i + k] = l[k]; }
+    }
+}
+// A GEMM's output as its split-K slices left it: element i is p[i] + p[i + stride] + ... (n terms, added in slice order)
+struct Slices {
+    const float* p;
+    int n;
+    size_t stride;
+};
+template <int V>
+__device__ __forceinline__ void ld_slices(const Slices& s, size_t i, float (&o)[V]) {
+    ld_vec<V>(s.p + i, o);
+    for (int k = 1; k < s.n; ++k) {
+        float t[V];
+        ld_vec<V>(s.p + (size_t)k * s.stride + i, t);
+#pragma unroll
+        for (int j = 0; j < V; ++j) o[j] += t[j];
     }
 }
 // out[i] = sum over the split-K slices of a tensor-core GEMM, in slice order
@@ -152,37 +183,67 @@ static __global__ void ly_embed_norm_kernel(const uint16_t* __restrict__ embed, 
 // itself (the next sublayer reads the stream un-normed).  yb: optional bias of the projection that produced y.  ls (optional) [W] scales
 // the normed result per channel.  Between two passes of a loop the stream then gains x0[row] (optional: the embedding output once
 // more) and step (optional [W]: the next pass's vector), in this order, before the next norm.
-static __global__ void ly_post_norm_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ yb, const float* __restrict__ wb,
+// One block per row, V consecutive channels per thread (V = 4: 16-byte accesses, W a multiple of 4); the row waits in shared memory
+// ([W] floats) between the passes (a thread reads back what it wrote itself).
+template <int V>
+static __global__ void __launch_bounds__(1024) ly_post_norm_kernel(float* __restrict__ x, Slices y, const float* __restrict__ yb, const float* __restrict__ wb,
                                            const float* __restrict__ wnext, const float* __restrict__ ls, const float* __restrict__ x0, const float* __restrict__ step,
                                            float eps, int W, int plain, int split_x, float* __restrict__ h, uint16_t* __restrict__ hhi, uint16_t* __restrict__ hlo) {
+    extern __shared__ __align__(16) float srow[];
     __shared__ float red[33];
-    const int row = blockIdx.x;
-    const float* yr = y + (size_t)row * W;
-    float* xr = x + (size_t)row * W;
+    const size_t rb = (size_t)blockIdx.x * W;
+    const int stride = blockDim.x * V;
     float ss = 0.f;
-    for (int c = threadIdx.x; c < W; c += blockDim.x) {
-        const float v = yr[c] + (yb ? yb[c] : 0.f);
-        ss += v * v;
+    for (int c = threadIdx.x * V; c < W; c += stride) {
+        float v[V];
+        ld_slices<V>(y, rb + c, v);
+        if (yb != nullptr) {
+            float b[V];
+            ld_vec<V>(yb + c, b);
+#pragma unroll
+            for (int i = 0; i < V; ++i) v[i] += b[i];
+        }
+#pragma unroll
+        for (int i = 0; i < V; ++i) ss += v[i] * v[i];
+        st_vec<V>(srow + c, v);
     }
     const float r = 1.f / sqrtf(block_sum(ss, red) / (float)W + eps);
     float s2 = 0.f;
-    for (int c = threadIdx.x; c < W; c += blockDim.x) {
-        float d = (yr[c] + (yb ? yb[c] : 0.f)) * r * norm_scale(wb, c, plain);
-        if (ls) d *= ls[c];
-        float v = xr[c] + d;
-        if (x0) v += x0[(size_t)row * W + c];
-        if (step) v += step[c];
-        xr[c] = v;
-        s2 += v * v;
-        if (wnext == nullptr && split_x) split_store(hhi, hlo, (size_t)row * W + c, v);
+    auto add = [&](float (&v)[V], const float* p) {
+        float t[V];
+        ld_vec<V>(p, t);
+#pragma unroll
+        for (int i = 0; i < V; ++i) v[i] += t[i];
+    };
+    for (int c = threadIdx.x * V; c < W; c += stride) {
+        float d[V], w[V], v[V];
+        ld_vec<V>(srow + c, d); ld_vec<V>(wb + c, w); ld_vec<V>(x + rb + c, v);
+#pragma unroll
+        for (int i = 0; i < V; ++i) d[i] = d[i] * r * (plain ? w[i] : 1.f + w[i]);
+        if (ls != nullptr) {
+            ld_vec<V>(ls + c, w);
+#pragma unroll
+            for (int i = 0; i < V; ++i) d[i] *= w[i];
+        }
+#pragma unroll
+        for (int i = 0; i < V; ++i) v[i] += d[i];
+        if (x0 != nullptr) add(v, x0 + rb + c);
+        if (step != nullptr) add(v, step + c);
+        st_vec<V>(x + rb + c, v);
+#pragma unroll
+        for (int i = 0; i < V; ++i) s2 += v[i] * v[i];
+        if (wnext != nullptr) st_vec<V>(srow + c, v);
+        else if (split_x) split_store_vec<V>(hhi, hlo, rb + c, v);
     }
     if (wnext == nullptr) return;
     const float r2 = 1.f / sqrtf(block_sum(s2, red) / (float)W + eps);
-    float* hr = h + (size_t)row * W;
-    for (int c = threadIdx.x; c < W; c += blockDim.x) {
-        const float v = xr[c] * r2 * norm_scale(wnext, c, plain);
-        hr[c] = v;
-        split_store(hhi, hlo, (size_t)row * W + c, v);
+    for (int c = threadIdx.x * V; c < W; c += stride) {
+        float v[V], w[V];
+        ld_vec<V>(srow + c, v); ld_vec<V>(wnext + c, w);
+#pragma unroll
+        for (int i = 0; i < V; ++i) v[i] = v[i] * r2 * (plain ? w[i] : 1.f + w[i]);
+        if (h != nullptr) st_vec<V>(h + rb + c, v);
+        split_store_vec<V>(hhi, hlo, rb + c, v);
     }
 }
 
@@ -543,47 +604,55 @@ struct LatentAppendArgs {
     const float *cosb, *sinb;                    // [max_seq][rdims / 2], already multiplied by the YaRN magnitude
     int H, D, R, C, rdims;
     int off_dq, Q; const float* dq_norm;         // Q > 0: columns off_dq .. of proj are a query latent instead of queries
-    float* cq; uint16_t *cqhi, *cqlo;            // [T, Q] the normed query latent and its hi | lo halves
+    float* cq; uint16_t *cqhi, *cqlo;            // [T, Q] the normed query latent (nullptr: not wanted) and its hi | lo halves
+    Slices in;                                   // what the columns are read from (proj itself, or the GEMM's slices)
+    int off_gate, n_gate;                        // gate columns to fold into proj when there are slices
 };
 // Per row: the latent (RMS-normed, plain weight) and the rotated shared key part go into the row's cache page; the rotated part of
 // every head's query is turned in place (with a query latent: the latent is normed instead, the queries do not exist yet).  Pairs (2i, 2i+1) of the first rdims channels turn by pos * f_i; the rest pass through.
+// Both norms' sums of squares are taken in one pass.  With a query latent the projected row may still lie in split-K slices (`in`):
+// they are folded as the columns are read, and the gate's columns are folded into proj for the kernel that reads them later.
 template <typename CT>
-static __global__ void ly_latent_append_kernel(LatentAppendArgs a) {
-    __shared__ float red[33];
-    const int row = blockIdx.x, pos = a.row_pos[row];
-    float* pr = a.proj + (size_t)row * a.ldp;
+static __global__ void __launch_bounds__(1024) ly_latent_append_kernel(LatentAppendArgs a) {
+    __shared__ float2 red[33];
+    const int row = blockIdx.x, pos = a.row_pos[row], tid = threadIdx.x, nt = blockDim.x;
+    const size_t rb = (size_t)row * a.ldp;
+    float* pr = a.proj + rb;
     const float* cs = a.cosb + (size_t)pos * (a.rdims / 2);
     const float* sn = a.sinb + (size_t)pos * (a.rdims / 2);
+    auto in = [&](int c) { float v[1]; ld_slices<1>(a.in, rb + c, v); return v[0]; };
+    const bool own = a.off_dkv >= 0;
+    float2 ss = make_float2(0.f, 0.f);
+    for (int c = tid; c < a.Q; c += nt) { const float v = in(a.off_dq + c); ss.x += v * v; }
+    if (own)
+        for (int c = tid; c < a.C; c += nt) { const float v = in(a.off_dkv + c); ss.y += v * v; }
+    ss = block_sum2(ss, red);
     if (a.Q > 0) {
-        const float* dq = pr + a.off_dq;
-        float sq = 0.f;
-        for (int c = threadIdx.x; c < a.Q; c += blockDim.x) sq += dq[c] * dq[c];
-        const float rq = 1.f / sqrtf(block_sum(sq, red) / (float)a.Q + a.eps);
-        for (int c = threadIdx.x; c < a.Q; c += blockDim.x) {
-            const float v = dq[c] * rq * a.dq_norm[c];
-            a.cq[(size_t)row * a.Q + c] = v;
+        const float rq = 1.f / sqrtf(ss.x / (float)a.Q + a.eps);
+        for (int c = tid; c < a.Q; c += nt) {
+            const float v = in(a.off_dq + c) * rq * a.dq_norm[c];
+            if (a.cq != nullptr) a.cq[(size_t)row * a.Q + c] = v;
             split_store(a.cqhi, a.cqlo, (size_t)row * a.Q + c, v);
         }
+        if (a.in.n > 1)
+            for (int c = tid; c < a.n_gate; c += nt) pr[a.off_gate + c] = in(a.off_gate + c);
     } else {
-        for (int i = threadIdx.x; i < a.H * (a.rdims / 2); i += blockDim.x) turn_pair(pr + a.off_q, a.D, a.R, a.rdims / 2, i, cs, sn);
+        for (int i = tid; i < a.H * (a.rdims / 2); i += nt) turn_pair(pr + a.off_q, a.D, a.R, a.rdims / 2, i, cs, sn);
     }
-    if (a.off_dkv < 0) return;
+    if (!own) return;
     const int slot = a.seq_slot[a.row_seq[row]];
     const int page = a.page_table[(size_t)slot * a.pps + pos / kKvPage];
     CT* dst = (CT*)a.pool + ((size_t)page * kKvPage + pos % kKvPage) * (a.C + a.R);
-    const float* ckv = pr + a.off_dkv;
-    float ss = 0.f;
-    for (int c = threadIdx.x; c < a.C; c += blockDim.x) ss += ckv[c] * ckv[c];
-    const float r = 1.f / sqrtf(block_sum(ss, red) / (float)a.C + a.eps);
-    for (int c = threadIdx.x; c < a.C; c += blockDim.x) st_c(dst + c, ckv[c] * r * a.dkv_norm[c]);
-    for (int i = threadIdx.x; i < a.R; i += blockDim.x) {
+    const float r = 1.f / sqrtf(ss.y / (float)a.C + a.eps);
+    for (int c = tid; c < a.C; c += nt) st_c(dst + c, in(a.off_dkv + c) * r * a.dkv_norm[c]);
+    for (int i = tid; i < a.R; i += nt) {
         float val;
         if (i < a.rdims) {
             const int pi = i >> 1;
-            const float u = ckv[a.C + 2 * pi], v = ckv[a.C + 2 * pi + 1];
+            const float u = in(a.off_dkv + a.C + 2 * pi), v = in(a.off_dkv + a.C + 2 * pi + 1);
             val = (i & 1) ? v * cs[pi] + u * sn[pi] : u * cs[pi] - v * sn[pi];
         } else {
-            val = ckv[a.C + i];
+            val = in(a.off_dkv + a.C + i);
         }
         st_c(dst + a.C + i, val);
     }
@@ -715,32 +784,46 @@ static __global__ void __launch_bounds__(kLatWarps * 32) ly_latent_attn_kernel(L
 // plain query part with W_uk absorbed.  This kernel writes the scaled plain parts [T][H * D] (what the block-diagonal GEMM turns
 // into columns 0 .. C of Q) and Q's remaining columns.  cosb != nullptr: the rotated parts are turned here (queries expanded
 // from a latent); otherwise they were turned in place before.
-static __global__ void ly_latent_split_q_kernel(const float* __restrict__ q, int ldq, const int* __restrict__ row_pos, const float* __restrict__ cosb,
+static __global__ void ly_latent_split_q_kernel(Slices q, int ldq, const int* __restrict__ row_pos, const float* __restrict__ cosb,
                                                 const float* __restrict__ sinb, int H, int D, int R, int rdims, int C, int Ep, float scale,
                                                 uint16_t* __restrict__ phi, uint16_t* __restrict__ plo, uint16_t* __restrict__ qhi,
                                                 uint16_t* __restrict__ qlo) {
-    const int row = blockIdx.x;
-    const float* qr = q + (size_t)row * ldq;
-    for (int i = threadIdx.x * 4; i < H * D; i += blockDim.x * 4) {        // D is a multiple of 8: four channels of one head
+    // grid (rows, chunks): the chunks of a row share its heads' channels
+    const int row = blockIdx.x, t0 = blockIdx.y * blockDim.x + threadIdx.x, nt = gridDim.y * blockDim.x;
+    const size_t rb = (size_t)row * ldq;
+    const bool v4 = (ldq & 3) == 0 && ((D + R) & 3) == 0 && (reinterpret_cast<uintptr_t>(q.p) & 15) == 0 && (q.stride & 3) == 0;
+    for (int i = t0 * 4; i < H * D; i += nt * 4) {        // D is a multiple of 8: four channels of one head
         float v[4];
-        const float* s = qr + (size_t)(i / D) * (D + R) + i % D;
+        const size_t s = rb + (size_t)(i / D) * (D + R) + i % D;
+        if (v4) {
+            ld_slices<4>(q, s, v);
+        } else {
 #pragma unroll
-        for (int k = 0; k < 4; ++k) v[k] = s[k] * scale;
+            for (int k = 0; k < 4; ++k) { float t[1]; ld_slices<1>(q, s + k, t); v[k] = t[0]; }
+        }
+#pragma unroll
+        for (int k = 0; k < 4; ++k) v[k] *= scale;
         split_store_vec<4>(phi, plo, (size_t)row * H * D + i, v);
     }
-    const int tail = Ep - C, half = rdims / 2;
+    const int pairs = (Ep - C) / 2, half = rdims / 2;       // C and R are multiples of 8: whole pairs
     const size_t at = (size_t)row_pos[row] * half;
-    for (int i = threadIdx.x; i < H * tail; i += blockDim.x) {
-        const int hd = i / tail, r = i % tail;
-        const float* s = qr + (size_t)hd * (D + R) + D;
-        float v = 0.f;
-        if (r < rdims && cosb != nullptr) {
-            const float cs = cosb[at + (r >> 1)], sn = sinb[at + (r >> 1)], a = s[r & ~1], b = s[r | 1];
-            v = ((r & 1) ? b * cs + a * sn : a * cs - b * sn) * scale;
-        } else if (r < R) {
-            v = s[r] * scale;
+    for (int i = t0; i < H * pairs; i += nt) {
+        const int hd = i / pairs, r = 2 * (i % pairs);
+        float a[1] = {0.f}, b[1] = {0.f};
+        if (r < R) {
+            const size_t s = rb + (size_t)hd * (D + R) + D + r;
+            ld_slices<1>(q, s, a); ld_slices<1>(q, s + 1, b);
+            if (r < rdims && cosb != nullptr) {
+                const float cs = cosb[at + (r >> 1)], sn = sinb[at + (r >> 1)], u = a[0], w = b[0];
+                a[0] = u * cs - w * sn;
+                b[0] = w * cs + u * sn;
+            }
         }
-        split_store(qhi, qlo, ((size_t)row * H + hd) * Ep + C + r, v);
+        const float x = a[0] * scale, y = b[0] * scale;
+        const size_t o = ((size_t)row * H + hd) * Ep + C + r;
+        const uint32_t h = pack_bf16x2(x, y);
+        *reinterpret_cast<uint32_t*>(qhi + o) = h;
+        *reinterpret_cast<uint32_t*>(qlo + o) = pack_bf16x2(x - bf16lo(h), y - bf16hi(h));
     }
 }
 
@@ -1048,6 +1131,48 @@ static __global__ void ly_attn_softmax_kernel(const float* __restrict__ S, const
     const int b_lo = n_first + max(first_main - k_lo, 0), c_hi = n_first + min(nk, pos - k_lo + 1);
     auto vis = [&](int c) { const int j = k_lo + c - n_first; return j >= ks.j0 || (j >= ks.s_lo && j < ks.s_hi); };
     const float* sr = S + r * nkp;
+    if (na == 0 && first_main == ks.j0 && ((c_hi + 3) & ~3) - (b_lo & ~3) <= keep) {
+        // the visible columns are one range [b_lo, c_hi) and fit: four columns per thread (nkp is a multiple of 64), the row's scores and
+        // then its exponentials stay in shared memory
+        const float sv = sink ? (sinkv ? sinkv[r % H] : 0.f) : 0.f;
+        const int lo4 = b_lo & ~3, step = blockDim.x * 4;
+        float m = sink ? sv : -INFINITY;
+        for (int c = lo4 + threadIdx.x * 4; c < c_hi; c += step) {
+            float v[4];
+            ld_vec<4>(sr + c, v);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                if (softcap > 0.f) v[i] = softcap * tanhf(v[i] * (1.f / softcap));
+                if (c + i < b_lo || c + i >= c_hi) v[i] = -INFINITY;
+                m = fmaxf(m, v[i]);
+            }
+            st_vec<4>(srow + (c - lo4), v);
+        }
+        m = warp_max(m);
+        const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5, nw = blockDim.x >> 5;
+        if (lane == 0) red[wid] = m;
+        __syncthreads();
+        m = warp_max(lane < nw ? red[lane] : -INFINITY);
+        float sum = 0.f;
+        for (int c = lo4 + threadIdx.x * 4; c < c_hi; c += step) {
+            float v[4];
+            ld_vec<4>(srow + (c - lo4), v);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) { v[i] = expf(v[i] - m); sum += v[i]; }
+            st_vec<4>(srow + (c - lo4), v);
+        }
+        const float inv = 1.f / (block_sum(sum, red) + (sink ? expf(sv - m) : 0.f));
+        for (int c = threadIdx.x * 4; c < nkp; c += step) {
+            float v[4] = {};
+            if (c >= lo4 && c < c_hi) {             // the same four columns lie with another thread: block_sum's barriers are behind
+                ld_vec<4>(srow + (c - lo4), v);
+#pragma unroll
+                for (int i = 0; i < 4; ++i) v[i] *= inv;
+            }
+            split_store_vec<4>(phi, plo, r * nkp + c, v);
+        }
+        return;
+    }
     const float inv_cap = softcap > 0.f ? 1.f / softcap : 0.f;
     const int nvis = na + max(c_hi - b_lo, 0);
     const bool kept = nvis <= keep;
@@ -1724,7 +1849,7 @@ static __global__ void ly_gated_group_norm_kernel(const float* __restrict__ y, c
 // ---- feed-forward ----------------------------------------------------------------------------------------------------------
 // act 0: act[p, f] = g * sigmoid(1.702 g) * (u + 1),  g = min(gu[p, f], limit),  u = clamp(gu[p, F + f], -limit, limit);
 // act 1: act[p, f] = gelu_tanh(g) * u,  gelu_tanh(z) = z/2 (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))).  bias [2F] (optional) is added
-// to gate | up first.  act 2: act[p, f] = relu(gu[p, f])^2 -- no gate matrix, gu has F columns.  act 3: act[p, f] = relu(g) * u.  p < *count
+// to gate | up first.  act 2: act[p, f] = relu(gu[p, f])^2 -- no gate matrix, gu has F columns.  act 3: act[p, f] = relu(g) * u.
 __device__ __forceinline__ float glu_value(float g, float u, int act, float limit) {
     if (act == 2) { g = fmaxf(g, 0.f); return g * g; }
     if (act == 3) return fmaxf(g, 0.f) * u;
@@ -1733,20 +1858,30 @@ __device__ __forceinline__ float glu_value(float g, float u, int act, float limi
     u = fminf(fmaxf(u, -limit), limit);
     return g * sigmoidf_(1.702f * g) * (u + 1.f);
 }
-static __global__ void ly_glu_kernel(const float* __restrict__ gu, int F, float limit, int act_kind, const float* __restrict__ bias,
-                                     const int* __restrict__ count, int rows, float* __restrict__ act, uint16_t* __restrict__ ahi,
-                                     uint16_t* __restrict__ alo) {
-    const int n = count ? *count : rows;
-    const size_t total = (size_t)n * F;
-    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
-        const size_t p = i / F, f = i - p * F;
-        const size_t gs = act_kind == 2 ? (size_t)F : (size_t)2 * F;
-        const float g = gu[p * gs + f] + (bias ? bias[f] : 0.f);
-        const float u = act_kind == 2 ? 0.f : gu[p * gs + F + f] + (bias ? bias[F + f] : 0.f);
-        const float v = glu_value(g, u, act_kind, limit);
-        if (act != nullptr) act[i] = v;         // nullptr: only the hi | lo halves are consumed (a tensor-core GEMM follows)
-        split_store(ahi, alo, i, v);
+// One block per (row p, chunk of 256 V channels); V consecutive channels per thread (V = 4: F a multiple of 4).
+template <int V>
+static __global__ void __launch_bounds__(256) ly_glu_kernel(Slices gu, int F, float limit, int act_kind, const float* __restrict__ bias, float* __restrict__ act,
+                                                            uint16_t* __restrict__ ahi, uint16_t* __restrict__ alo) {
+    const int f = (blockIdx.y * 256 + threadIdx.x) * V;
+    if (f >= F) return;
+    const size_t p = blockIdx.x, base = p * (act_kind == 2 ? (size_t)F : (size_t)2 * F) + f;
+    float g[V], u[V] = {}, b[V];
+    ld_slices<V>(gu, base, g);
+    if (act_kind != 2) ld_slices<V>(gu, base + F, u);
+    if (bias != nullptr) {
+        ld_vec<V>(bias + f, b);
+#pragma unroll
+        for (int i = 0; i < V; ++i) g[i] += b[i];
+        if (act_kind != 2) {
+            ld_vec<V>(bias + F + f, b);
+#pragma unroll
+            for (int i = 0; i < V; ++i) u[i] += b[i];
+        }
     }
+#pragma unroll
+    for (int i = 0; i < V; ++i) g[i] = glu_value(g[i], u[i], act_kind, limit);
+    if (act != nullptr) st_vec<V>(act + p * F + f, g);          // nullptr: only the hi | lo halves are consumed (a tensor-core GEMM follows)
+    split_store_vec<V>(ahi, alo, p * F + f, g);
 }
 
 // Router: z = Wr h (f32), s = softmax(z) over all experts, the `top` largest (lower index first among equals), weights s / (sum + 1e-20).

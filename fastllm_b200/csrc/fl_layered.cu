@@ -938,6 +938,24 @@ static void launch_rec_scan(LaunchCtx& lc, const RecArgs& a, int n) {
     else go(ly_rec_scan_kernel<64, DELTA>, 64);
 }
 
+// P = softmax of the score block's rows (see ly_attn_softmax_kernel)
+static void launch_attn_softmax(LayeredCache& y, LaunchCtx& lc, const int* row_pos, int row0, int H, int rows, int k_lo, int n_first, int nk, int nkp, int window,
+                                int keep_first, int chunk, float softcap, int sink, const float* sinkv) {
+    if (n_first == 0 && (keep_first == 0 || window == 0) && nkp <= 2048) {
+        auto go = [&](auto kern) {
+            launch(lc, "attn_softmax", 0, kern, dim3((rows + 7) / 8), dim3(256), 0, (const float*)y.at_s.p, row_pos, row0, H, rows, k_lo, nk, nkp, window, chunk, softcap,
+                   sink, sinkv, y.at_phi.p, y.at_plo.p);
+        };
+        if (nkp <= 512) go(ly_attn_softmax_warp_kernel<4>);
+        else if (nkp <= 1024) go(ly_attn_softmax_warp_kernel<8>);
+        else go(ly_attn_softmax_warp_kernel<16>);
+        return;
+    }
+    const int keep = std::min(nkp, kSoftmaxKeep);
+    launch(lc, "attn_softmax", 0, ly_attn_softmax_kernel, dim3(rows), dim3(256), (size_t)keep * 4, (const float*)y.at_s.p, row_pos, row0, H, k_lo, n_first, nk, nkp,
+           window, keep_first, chunk, softcap, sink, sinkv, keep, y.at_phi.p, y.at_plo.p);
+}
+
 // Latent attention of rows [r0, r0 + Ts) -- one sequence's portion, positions pos0.. -- on the tensor-core GEMM, in blocks of query
 // rows small enough that a block's score matrix stays within a fixed scratch budget.  A block only gathers the keys its rows'
 // windows reach, so long prompts with short windows never touch fully masked regions.
@@ -977,18 +995,23 @@ static void latent_attn_tc(fl_cache& c, LaunchCtx& lc, const LatentAttnArgs& a, 
             }
             continue;
         }
-        launch(lc, "attn_gather_keys", 0, ly_attn_gather_keys_kernel, dim3(nkp), dim3(128), 0, (const uint16_t*)a.pool, page_row, k_lo, nk, nkp, C, E, Ep,
-               y.at_kc.p, y.at_kct.p);
+        // without a window every block's keys are a prefix of the last block's: they are gathered once (a later key meets a zero
+        // probability)
+        const int ldt = a.window > 0 ? nkp : (int)nkp_max;
+        if (a.window > 0)
+            launch(lc, "attn_gather_keys", 0, ly_attn_gather_keys_kernel, dim3(nkp / 64, Ep / 64), dim3(256), 0, (const uint16_t*)a.pool, page_row, k_lo, nk, nkp, C, E,
+                   Ep, y.at_kc.p, y.at_kct.p);
+        else if (f == 0)
+            launch(lc, "attn_gather_keys", 0, ly_attn_gather_keys_kernel, dim3(ldt / 64, Ep / 64), dim3(256), 0, (const uint16_t*)a.pool, page_row, 0, pos0 + Ts, ldt, C,
+                   E, Ep, y.at_kc.p, y.at_kct.p);
         const size_t q0 = (size_t)(r0 + f) * H;
         if (mma == nullptr)
             launch(lc, "attn_build_q", 0, ly_attn_build_q_kernel, dim3(nq, H), dim3(128), 0, a.qa, a.proj, a.ldp, a.off_q, r0 + f, H, a.D, R, C, Ep, a.scale,
                    y.at_qhi.p, y.at_qlo.p);
         const CUtensorMap tk = make_tmap_bf16(y.at_kc.p, (uint64_t)nkp, (uint64_t)Ep, (uint64_t)Ep, 128);
         dense_gemm(c, lc, "gemm_tc_attn_scores", rows, nkp, Ep, tk, y.at_s.p, mma ? mma->qhi + q0 * Ep : y.at_qhi.p, mma ? mma->qlo + q0 * Ep : y.at_qlo.p);
-        const int keep = std::min(nkp, kSoftmaxKeep);
-        launch(lc, "attn_softmax", 0, ly_attn_softmax_kernel, dim3(rows), dim3(256), (size_t)keep * 4, (const float*)y.at_s.p, a.row_pos, r0 + f, H, k_lo, 0, nk, nkp,
-               a.window, 0, 0, 0.f, a.sink, a.sinkv, keep, y.at_phi.p, y.at_plo.p);
-        const CUtensorMap tv = make_tmap_bf16(y.at_kct.p, (uint64_t)C, (uint64_t)nkp, (uint64_t)nkp, 128);
+        launch_attn_softmax(y, lc, a.row_pos, r0 + f, H, rows, k_lo, 0, nk, nkp, a.window, 0, 0, 0.f, a.sink, a.sinkv);
+        const CUtensorMap tv = make_tmap_bf16(y.at_kct.p, (uint64_t)C, (uint64_t)nkp, (uint64_t)ldt, 128);
         if (mma != nullptr)
             dense_gemm_blocks(c, lc, "gemm_tc_attn_values", rows, 1, C, nkp, tv, y.at_phi.p, y.at_plo.p, mma->ohi + q0 * C, mma->olo + q0 * C, C, 0);
         else
@@ -1043,9 +1066,8 @@ static void gqa_attn_tc(fl_cache& c, LaunchCtx& lc, const GqaAttnArgs& a, int r0
                    y.at_qlo.p);
             const CUtensorMap tk = make_tmap_bf16(y.at_kc.p, (uint64_t)nkp, (uint64_t)Dp, (uint64_t)Dp, 128);
             dense_gemm(c, lc, "gemm_tc_attn_scores", rows, nkp, Dp, tk, y.at_s.p, y.at_qhi.p, y.at_qlo.p);
-            const int keep = std::min(nkp, kSoftmaxKeep);
-            launch(lc, "attn_softmax", 0, ly_attn_softmax_kernel, dim3(rows), dim3(256), (size_t)keep * 4, (const float*)y.at_s.p, a.row_pos, r0 + f, rep, k_lo, n_first,
-                   nk, nkp, a.window, a.keep_first, a.chunk, a.softcap, a.sink, a.sinkv ? a.sinkv + g * rep : (const float*)nullptr, keep, y.at_phi.p, y.at_plo.p);
+            launch_attn_softmax(y, lc, a.row_pos, r0 + f, rep, rows, k_lo, n_first, nk, nkp, a.window, a.keep_first, a.chunk, a.softcap, a.sink,
+                                a.sinkv ? a.sinkv + g * rep : (const float*)nullptr);
             const CUtensorMap tv = make_tmap_bf16(y.at_kct.p, (uint64_t)Dv, (uint64_t)nkp, (uint64_t)nkp, 128);
             dense_gemm(c, lc, "gemm_tc_attn_values", rows, Dv, nkp, tv, y.at_o.p + (size_t)g * rows * Dv, y.at_phi.p, y.at_plo.p);
         }

@@ -131,6 +131,14 @@ __device__ __forceinline__ void tmem_ld16(uint32_t taddr, uint32_t (&r)[16]) {
     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 }
 
+// 32 bytes per lane in one store (sm_100; the address is 32-byte aligned).  thread == accumulator row scatters a warp's store over 32
+// lines, so the widest store halves the line accesses of an epilogue and writes whole sectors.
+__device__ __forceinline__ void st_global_32b(void* p, const uint32_t (&v)[8]) {
+    asm volatile("st.global.v8.b32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8};" ::"l"(p), "r"(v[0]), "r"(v[1]), "r"(v[2]), "r"(v[3]), "r"(v[4]), "r"(v[5]), "r"(v[6]),
+                 "r"(v[7])
+                 : "memory");
+}
+
 // Shared-memory matrix descriptor for a K-major bf16 tile stored as rows of 128 bytes with the 128-byte swizzle
 // (exactly what TMA SWIZZLE_128B writes): start address >> 4, LBO = 1 (ignored for swizzled K-major), SBO = 1024 B >> 4
 // (stride between 8-row groups), version = 1 (Blackwell), layout type 2 = SWIZZLE_128B.
@@ -531,26 +539,41 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
                         const size_t o = (size_t)row * g.ldo + (size_t)grp * g.o_bs + col;
                         uint16_t *oh = reinterpret_cast<uint16_t*>(g.out) + o, *ol = reinterpret_cast<uint16_t*>(g.out2) + o;
                         const float* gt = g.gate != nullptr ? g.gate + (size_t)row * g.ldg + (size_t)grp * g.N + col : nullptr;
+                        const bool wide = ((g.ldo | g.o_bs | g.N) & 15) == 0 && ((reinterpret_cast<uintptr_t>(g.out) | reinterpret_cast<uintptr_t>(g.out2)) & 31) == 0;
 #pragma unroll
-                        for (int j = 0; j < 32; j += 8) {
+                        for (int j = 0; j < 32; j += 16) {
                             if (col + j < g.N) {
-                                float v[8];
+                                uint32_t ph[8], pl[8];
+                                const bool second = col + j + 8 < g.N;         // N is a multiple of 8
 #pragma unroll
-                                for (int e = 0; e < 8; ++e) v[e] = __uint_as_float(r[j + e]);
-                                if (gt != nullptr) {
-                                    const float4 z0 = *reinterpret_cast<const float4*>(gt + j), z1 = *reinterpret_cast<const float4*>(gt + j + 4);
-                                    const float z[8] = {z0.x, z0.y, z0.z, z0.w, z1.x, z1.y, z1.z, z1.w};
+                                for (int q8 = 0; q8 < 2; ++q8) {
+                                    float v[8];
 #pragma unroll
-                                    for (int e = 0; e < 8; ++e) v[e] *= 1.f / (1.f + expf(-z[e]));
+                                    for (int e = 0; e < 8; ++e) v[e] = __uint_as_float(r[j + 8 * q8 + e]);
+                                    if (gt != nullptr && (q8 == 0 || second)) {
+                                        const float4 z0 = *reinterpret_cast<const float4*>(gt + j + 8 * q8), z1 = *reinterpret_cast<const float4*>(gt + j + 8 * q8 + 4);
+                                        const float z[8] = {z0.x, z0.y, z0.z, z0.w, z1.x, z1.y, z1.z, z1.w};
+#pragma unroll
+                                        for (int e = 0; e < 8; ++e) v[e] *= 1.f / (1.f + expf(-z[e]));
+                                    }
+#pragma unroll
+                                    for (int e = 0; e < 4; ++e) {
+                                        const uint32_t h = pack_bf16x2(v[2 * e], v[2 * e + 1]);
+                                        ph[4 * q8 + e] = h;
+                                        pl[4 * q8 + e] = pack_bf16x2(v[2 * e] - bf16lo(h), v[2 * e + 1] - bf16hi(h));
+                                    }
                                 }
-                                uint32_t ph[4], pl[4];
-#pragma unroll
-                                for (int e = 0; e < 4; ++e) {
-                                    ph[e] = pack_bf16x2(v[2 * e], v[2 * e + 1]);
-                                    pl[e] = pack_bf16x2(v[2 * e] - bf16lo(ph[e]), v[2 * e + 1] - bf16hi(ph[e]));
+                                if (wide) {
+                                    st_global_32b(oh + j, ph);
+                                    st_global_32b(ol + j, pl);
+                                } else {
+                                    *reinterpret_cast<uint4*>(oh + j) = make_uint4(ph[0], ph[1], ph[2], ph[3]);
+                                    *reinterpret_cast<uint4*>(ol + j) = make_uint4(pl[0], pl[1], pl[2], pl[3]);
+                                    if (second) {
+                                        *reinterpret_cast<uint4*>(oh + j + 8) = make_uint4(ph[4], ph[5], ph[6], ph[7]);
+                                        *reinterpret_cast<uint4*>(ol + j + 8) = make_uint4(pl[4], pl[5], pl[6], pl[7]);
+                                    }
                                 }
-                                *reinterpret_cast<uint4*>(oh + j) = make_uint4(ph[0], ph[1], ph[2], ph[3]);
-                                *reinterpret_cast<uint4*>(ol + j) = make_uint4(pl[0], pl[1], pl[2], pl[3]);
                             }
                         }
                     } else if (EPI == GEPI_HL_T) {
@@ -585,6 +608,15 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
                     } else {
                         float* o = reinterpret_cast<float*>(g.out) + (EPI == GEPI_F32 ? (size_t)ksi * (size_t)g.split_stride : 0) + (size_t)row * g.ldo + col;
                         const uint16_t* rs = (EPI == GEPI_BIAS_RESID_F32 && g.resid) ? g.resid + (size_t)row * g.ldr + col : nullptr;
+                        if (EPI == GEPI_F32 && ((g.ldo | g.N) & 7) == 0 && (g.split_stride & 7) == 0 && (reinterpret_cast<uintptr_t>(g.out) & 31) == 0) {
+#pragma unroll
+                            for (int j = 0; j < 32; j += 8)
+                                if (col + j < g.N) {
+                                    const uint32_t v[8] = {r[j], r[j + 1], r[j + 2], r[j + 3], r[j + 4], r[j + 5], r[j + 6], r[j + 7]};
+                                    st_global_32b(o + j, v);
+                                }
+                            continue;
+                        }
 #pragma unroll
                         for (int j = 0; j < 32; j += 4) {
                             if (col + j < g.N) {

@@ -1072,18 +1072,25 @@ static __global__ void __launch_bounds__(256) ly_latent_mma_kernel(LatMmaArgs a)
 //   P = masked softmax(S) in f32,   O = P . Kc[:, :C] (a second GEMM against the transposed latents).
 // Kc [nkp, Ep]: the keys' cache rows (latent | rotated part | zero padding), KcT [C, nkp]: the latents transposed; padding is
 // zero so that masked probabilities (exact zeros) meet finite values.
-static __global__ void ly_attn_gather_keys_kernel(const uint16_t* __restrict__ pool, const int* __restrict__ page_row, int k_lo, int nk, int nkp, int C,
-                                                  int E, int Ep, uint16_t* __restrict__ kc, uint16_t* __restrict__ kct) {
-    const int r = blockIdx.x;
-    const uint16_t* src = nullptr;
-    if (r < nk) {
-        const int j = k_lo + r;
-        src = pool + ((size_t)page_row[j / kKvPage] * kKvPage + j % kKvPage) * E;
+// One block per 64 keys x 64 columns: the tile passes through shared memory so that both copies are written in runs.
+static __global__ void __launch_bounds__(256) ly_attn_gather_keys_kernel(const uint16_t* __restrict__ pool, const int* __restrict__ page_row, int k_lo, int nk, int nkp,
+                                                                         int C, int E, int Ep, uint16_t* __restrict__ kc, uint16_t* __restrict__ kct) {
+    __shared__ uint16_t tile[64][66];
+    const int r0 = blockIdx.x * 64, c0 = blockIdx.y * 64;
+    for (int i = threadIdx.x; i < 64 * 64; i += 256) {
+        const int r = i >> 6, c = i & 63, key = r0 + r;
+        uint16_t v = 0;
+        if (key < nk && c0 + c < E) {
+            const int j = k_lo + key;
+            v = pool[((size_t)page_row[j / kKvPage] * kKvPage + j % kKvPage) * E + c0 + c];
+        }
+        kc[(size_t)key * Ep + c0 + c] = v;
+        tile[r][c] = v;
     }
-    for (int c = threadIdx.x; c < Ep; c += blockDim.x) {
-        const uint16_t v = (src != nullptr && c < E) ? src[c] : (uint16_t)0;
-        kc[(size_t)r * Ep + c] = v;
-        if (c < C) kct[(size_t)c * nkp + r] = v;
+    __syncthreads();
+    for (int i = threadIdx.x; i < 64 * 64; i += 256) {
+        const int c = i >> 6, r = i & 63;
+        if (c0 + c < C) kct[(size_t)(c0 + c) * nkp + r0 + r] = tile[r][c];
     }
 }
 // Q operand rows (token, head): [q~ * scale | rotated query part * scale | 0] as hi | lo halves
@@ -1222,6 +1229,53 @@ static __global__ void ly_out_gate_kernel(float* __restrict__ u, const float* __
         const float v = u[i] * sigmoidf_(proj[row * ldp + off_g + (i - row * n)]);
         u[i] = v;
         split_store(uhi, ulo, i, v);
+    }
+}
+
+// The same for masks whose visible keys form one range (no kept first keys) and rows of at most 128 NG columns: one warp per row, the
+// row's scores stay in registers (lane l owns columns 128 k + 4 l ..).
+template <int NG>
+static __global__ void __launch_bounds__(256) ly_attn_softmax_warp_kernel(const float* __restrict__ S, const int* __restrict__ row_pos, int row0, int H, int rows,
+                                                                          int k_lo, int nk, int nkp, int window, int chunk, float softcap, int sink,
+                                                                          const float* __restrict__ sinkv, uint16_t* __restrict__ phi, uint16_t* __restrict__ plo) {
+    const int r = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (r >= rows) return;
+    const int pos = row_pos[row0 + r / H];
+    const int b_lo = max(key_span(pos, window, 0, chunk).j0 - k_lo, 0), c_hi = min(nk, pos - k_lo + 1);
+    const float sv = sink ? (sinkv ? sinkv[r % H] : 0.f) : 0.f, inv_cap = softcap > 0.f ? 1.f / softcap : 0.f;
+    const size_t rb = (size_t)r * nkp;
+    float v[NG][4], m = sink ? sv : -INFINITY;
+#pragma unroll
+    for (int k = 0; k < NG; ++k) {
+        const int c = k * 128 + lane * 4;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) v[k][i] = -INFINITY;
+        if (c < c_hi && c + 4 > b_lo) {
+            ld_vec<4>(S + rb + c, v[k]);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                if (softcap > 0.f) v[k][i] = softcap * tanhf(v[k][i] * inv_cap);
+                if (c + i < b_lo || c + i >= c_hi) v[k][i] = -INFINITY;
+                m = fmaxf(m, v[k][i]);
+            }
+        }
+    }
+    m = warp_max(m);
+    float sum = 0.f;
+#pragma unroll
+    for (int k = 0; k < NG; ++k)
+        if (k * 128 < c_hi) {
+#pragma unroll
+            for (int i = 0; i < 4; ++i) { v[k][i] = expf(v[k][i] - m); sum += v[k][i]; }
+        }
+    const float inv = 1.f / (warp_sum(sum) + (sink ? expf(sv - m) : 0.f));
+#pragma unroll
+    for (int k = 0; k < NG; ++k) {
+        const int c = k * 128 + lane * 4;
+        if (c >= nkp) continue;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) v[k][i] = k * 128 < c_hi ? v[k][i] * inv : 0.f;
+        split_store_vec<4>(phi, plo, rb + c, v[k]);
     }
 }
 

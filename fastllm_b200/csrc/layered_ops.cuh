@@ -1,5 +1,6 @@
 // Kernels of the layered decoders (sm_100a): residual / norm glue, the exact-f32 GEMM, gated linear attention (decay, scan, head
-// norm + gate), latent attention over the paged latent cache (append + rotary, absorbed-query attention), grouped-query attention
+// norm + gate), latent attention over the paged latent cache (append + rotary, absorbed-query attention on the tensor cores or per
+// (row, head), query latents, output gate), grouped-query attention
 // with per-head q/k norm, score cap and softmax sink, the short-convolution recurrent mixers (Mamba-2, gated delta rule: prep, scan,
 // gated norms), the feed-forward (clamped swish or tanh-gelu GLU with optional biases, ungated squared relu), the mixture-of-experts
 // routers (softmax top-k; sigmoid scores with a choice correction and group-limited choice) / row lists / combine, and the pieces of

@@ -102,8 +102,7 @@ struct PkArgs {
     float* peer_logits[8];           // rank r's full-vocabulary logits [Vfull]
     unsigned int ar_epoch0;          // exchanges completed on this communicator before this launch
     int* comm_err;                   // set to 1 when a peer did not show up within the spin budget
-    int flags;            // dev knob (FL_PK_FLAGS) bit 0: prefetch this CTA's KV pages into L2 at the top of P1; bits 1-3: timing
-                          // experiments with garbage results (2: no arithmetic, 4: no attention, 8: no weight traffic)
+    int flags;            // dev knob (FL_PK_FLAGS) bit 0: prefetch this CTA's KV pages into L2 at the top of P1
     long long* dbg;       // optional: CTA 0 writes %globaltimer at the phase boundaries of layer L/2 (FL_PK_DEBUG=1)
 };
 
@@ -274,10 +273,6 @@ __global__ void __launch_bounds__(kPkThreads, 1) decode_persistent_kernel(const 
                             a.dbg[660 + (g & 3) * 10 + 8] = t;
                             a.dbg[660 + (g & 3) * 10 + 9] = ++pn;
                         }
-                        if (a.flags & 8) {      // timing experiment: no weight traffic at all (results are garbage)
-                            mbar_arrive(&full[st]);
-                            continue;
-                        }
                         mbar_expect_tx(&full[st], kPkStageBytes);      // the whole box always arrives (out-of-range columns as zeros)
                         // weights are dead once staged: evict_first keeps the L2 for the KV cache and the activations
                         asm volatile(
@@ -360,7 +355,6 @@ __global__ void __launch_bounds__(kPkThreads, 1) decode_persistent_kernel(const 
             // c % NS: faster with the weight traffic switched off, 0.8-3.6 % SLOWER in the real run on all three models: dropped.)
             constexpr int KPW = kPkChunkCols / 16 / kPkConsumerWarps;      // k-steps per warp per full chunk (8)
             const uint16_t* xcol = xrow + (col0 + bk + warp * 16);
-            if (!(a.flags & 2))      // (timing experiment: bit 1 skips the arithmetic)
 #pragma unroll
             for (int h = 0; h < KPW; h += 4) {
                 uint32_t af[4][4], bf[4][2];
@@ -624,7 +618,7 @@ __global__ void __launch_bounds__(kPkThreads, 1) decode_persistent_kernel(const 
                 const int per = (npages + a.nsplit - 1) / a.nsplit;
                 float* gacc = xs;                            // [NG][HG][D]
                 float* gml = xs + NG * HG * D;               // [NG][HG][2]
-                for (int item = (a.flags & 4) ? a.nkv * a.nsplit : cta; item < a.nkv * a.nsplit; item += ncta) {      // (bit 2: timing experiment without attention)
+                for (int item = cta; item < a.nkv * a.nsplit; item += ncta) {
                     const int kvh = item / a.nsplit, split = item % a.nsplit;
                     const int tok0 = split * per * kKvPage, tok1 = min(min((split + 1) * per, npages) * kKvPage, len);
                     const int gidx = warp * TPW + grp;

@@ -54,8 +54,6 @@ struct GemmArgs {
     int o_bs = 0;
     const float* gate = nullptr;
     int ldg = 0;
-    int dbg = 0;                // dev knob FL_GEMM_DBG (timing experiments only, results are garbage): bit 0 = DUAL_B without the
-                                // activation loads, bit 1 = no MMAs (the issuer releases a stage as soon as it has landed)
 };
 
 // ---- PTX wrappers ------------------------------------------------------------------------------------------------------
@@ -200,7 +198,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
     constexpr uint32_t kBOff = (DUAL == DUAL_A ? 2 : 1) * kABytes;
     // DUAL_B: the hi and lo activation tiles sit back to back in a stage ([BN rows x 128 B] each, same swizzle), so ONE MMA of
     // N = 2 BN multiplies the weight tile with both -- half the tcgen05.mma instructions per staged byte (at N = 16 the issue rate
-    // of these tiny MMAs, not the weight stream, was the limit: FL_GEMM_DBG=2 measured it) -- into two accumulator column blocks
+    // of these tiny MMAs, not the weight stream, was the limit) -- into two accumulator column blocks
     // [W.hi | W.lo] that the epilogue adds.
     constexpr int kMmaN = (DUAL == DUAL_B) ? 2 * BN : BN;
     static_assert(kMmaN <= 256, "UMMA N <= 256");
@@ -313,11 +311,6 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
                         continue;
                     }
                     mbar_wait(&empty[st], ((c / kStages) & 1) ^ 1);
-                    if (DUAL == DUAL_B && (g.dbg & 1)) {        // timing experiment: the weight stream alone
-                        mbar_expect_tx(&full[st], kABytes);
-                        tma_load_2d(sa, &tmA, kb * kGemmBK, m0, &full[st]);
-                        continue;
-                    }
                     mbar_expect_tx(&full[st], kStageBytes);
                     if (DUAL == DUAL_B) {       // tmA = weights, tmA2 / tmB = activation hi / lo
                         tma_load_2d(sa, &tmA, kb * kGemmBK, m0, &full[st]);
@@ -353,10 +346,6 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
                     const int st = c % kStages;
                     mbar_wait(&full[st], (c / kStages) & 1);
                     tc_fence_after();
-                    if (g.dbg & 2) {            // timing experiment: no tensor-core work, the stage goes straight back
-                        mbar_arrive(&empty[st]);
-                        continue;
-                    }
                     const uint8_t* sa = gsm + (size_t)st * kStageBytes;
                     const uint64_t adesc = umma_smem_desc_sw128(sa), bdesc = umma_smem_desc_sw128(sa + kBOff);
 #pragma unroll

@@ -12,11 +12,11 @@ HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(HERE, "libfastllm_b200.so")
 
 FL_ARCH = {"llama": 0, "mistral": 1, "qwen2": 2, "mixtral": 3, "bert": 4, "nifunex": 5, "rofetar": 6, "tozarax": 7, "medulorn": 8,
-           "latodra": 9}
+           "latodra": 9, "tufazen": 10}
 FL_MIXER = {"gla": 0, "latent_attention": 1, "attention": 2, "mamba2": 3, "delta": 4, "lightning": 5}
-FL_ACT = {"swish_clamp": 0, "gelu_tanh": 1, "relu2": 2, "relu": 3}
+FL_ACT = {"swish_clamp": 0, "gelu_tanh": 1, "relu2": 2, "relu": 3, "silu": 4}
 FL_ROT_SCALE = {"yarn": 0, "bands": 1}
-FL_ROUTER = {"softmax": 0, "sigmoid_groups": 1}
+FL_ROUTER = {"softmax": 0, "sigmoid_groups": 1, "softmax_groups": 2}
 FL_FFN = {"none": 0, "dense": 1, "moe": 2}
 FL_DTYPE_F32, FL_DTYPE_BF16, FL_DTYPE_F16 = 0, 1, 2
 
@@ -43,7 +43,7 @@ class FlLayerDesc(C.Structure):
                 ("route_keep", C.c_int32), ("qkv_bias", C.c_int32), ("qk_norm_whole", C.c_int32), ("mask_chunk", C.c_int32),
                 ("keep_first", C.c_int32), ("rot_scaling", C.c_int32), ("out_scale", C.c_float), ("pair_sum", C.c_int32),
                 ("router_bias", C.c_int32), ("shared_plain", C.c_int32), ("q_rank", C.c_int32), ("out_gate", C.c_int32),
-                ("reserved", C.c_int32 * 2)]
+                ("v_from_k", C.c_int32), ("route_best", C.c_int32), ("route_renorm", C.c_int32), ("reserved", C.c_int32 * 1)]
 
 
 class FlStackConfig(C.Structure):
@@ -53,7 +53,9 @@ class FlStackConfig(C.Structure):
                 ("post_sum_norm", C.c_int32), ("residual_alpha", C.c_float), ("norm_scalar", C.c_int32), ("embed_scale", C.c_float),
                 ("logit_softcap", C.c_float), ("token_shift", C.c_int32), ("embed_norm", C.c_int32), ("layer_scale", C.c_int32),
                 ("tied_head", C.c_int32), ("loop_start", C.c_int32), ("loop_stop", C.c_int32), ("loop_times", C.c_int32),
-                ("loop_reinject", C.c_int32), ("loop_step", C.c_int32), ("reserved", C.c_int32 * 3)]
+                ("loop_reinject", C.c_int32), ("loop_step", C.c_int32), ("norm_tanh", C.c_int32), ("parallel_sub", C.c_int32),
+                ("token_side", C.c_int32), ("bigram_buckets", C.c_int32), ("logit_scale", C.c_float), ("bigram_mul_prev", C.c_int64),
+                ("bigram_mul_cur", C.c_int64), ("reserved", C.c_int32 * 2)]
 
 
 class FastllmError(RuntimeError):

@@ -1,4 +1,4 @@
-// Layered decoders (FL_ARCH_NIFUNEX, FL_ARCH_ROFETAR, FL_ARCH_TOZARAX, FL_ARCH_MEDULORN, FL_ARCH_LATODRA): weight layout + ingest, pooled cache (pages of latents or keys | values +
+// Layered decoders (FL_ARCH_NIFUNEX, FL_ARCH_ROFETAR, FL_ARCH_TOZARAX, FL_ARCH_MEDULORN, FL_ARCH_LATODRA, FL_ARCH_TUFAZEN): weight layout + ingest, pooled cache (pages of latents or keys | values +
 // recurrent-state slots), and the step function for mixed batches (portions of prompts beside single decoded tokens).
 #include <cmath>
 #include <map>
@@ -41,6 +41,11 @@ struct LyRoute {
     void* dst;
     int64_t rows, cols;     // shape handed over
     int heads;              // UK_T: source rows = heads * (rows / heads)
+    int64_t ld = 0;         // MAT16: row stride of the destination (0: cols)
+    // MAT16 with turn_dims > 0: the rows form blocks of turn_per; inside each, the turn_dims rows from turn_at on hold rotary pairs as two
+    // halves (i, i + turn_dims / 2) and are laid out as neighbours (2i, 2i + 1) -- what the latent attention's kernels turn.  A score does
+    // not change when query and key channels are reordered alike.
+    int turn_per = 0, turn_at = 0, turn_dims = 0;
 };
 struct LayeredRoutes {
     std::map<std::string, LyRoute> r;
@@ -63,11 +68,12 @@ static void check_mixer(const LayeredModel& m, int i, const fl_layer_desc& d, bo
         FL_CHECK(d.rot_dims >= 0 && d.rot_dims <= d.rot_dim && d.rot_dims % 2 == 0, FL_ERR_INVALID, at + "rotated channels must be even and <= rot_dim");
         FL_CHECK(d.window >= 0, FL_ERR_INVALID, at + "negative window");
         FL_CHECK(d.q_rank >= 0 && d.sink >= 0 && d.sink <= 2, FL_ERR_INVALID, at + "bad query latent size / sink kind");
+        FL_CHECK(d.out_gate >= 0 && d.out_gate <= 2, FL_ERR_INVALID, at + "unknown gate kind");
         if (d.kv_from >= 0) {
             FL_CHECK(d.kv_from < i, FL_ERR_INVALID, at + "kv_from must name an earlier layer");
             const fl_layer_desc& s = m.layers[d.kv_from].d;
             FL_CHECK(s.mixer == FL_MIXER_LATENT_ATTN && s.kv_from < 0 && s.kv_rank == d.kv_rank && s.rot_dim == d.rot_dim &&
-                         s.rot_dims == d.rot_dims && s.rot_base == d.rot_base && s.yarn_factor == d.yarn_factor &&
+                         s.rot_dims == d.rot_dims && s.rot_halves == d.rot_halves && s.rot_base == d.rot_base && s.yarn_factor == d.yarn_factor &&
                          s.yarn_original == d.yarn_original && s.yarn_fast == d.yarn_fast && s.yarn_slow == d.yarn_slow,
                      FL_ERR_INVALID, at + "kv_from must name a latent-attention layer with its own cache and the same latent / rotary sizes");
         }
@@ -79,6 +85,9 @@ static void check_mixer(const LayeredModel& m, int i, const fl_layer_desc& d, bo
         FL_CHECK(d.window >= 0 && d.softcap >= 0.f, FL_ERR_INVALID, at + "negative window / score cap");
         FL_CHECK(d.keep_first >= 0 && d.mask_chunk >= 0 && d.sink >= 0 && d.sink <= 2, FL_ERR_INVALID, at + "bad mask sizes / sink kind");
         FL_CHECK(d.rot_scaling == FL_ROT_SCALE_YARN || d.rot_scaling == FL_ROT_SCALE_BANDS, FL_ERR_INVALID, at + "unknown rotary scaling");
+        FL_CHECK(d.out_gate >= 0 && d.out_gate <= 2, FL_ERR_INVALID, at + "unknown gate kind");
+        FL_CHECK(!d.v_from_k || (d.no_qk_norm && d.vdim == d.dim && d.kv_from < 0), FL_ERR_UNSUPPORTED,
+                 at + "values that are the keys: built without q/k norms, with vdim = dim and a cache of its own");
         FL_CHECK(!(d.qk_norm_whole && d.no_qk_norm), FL_ERR_INVALID, at + "a q/k norm over the whole projection needs the q/k norm");
         FL_CHECK(!(d.qkv_bias && d.kv_from >= 0), FL_ERR_UNSUPPORTED, at + "biased projections are built for layers with their own cache");
         if (d.kv_from >= 0) {
@@ -108,24 +117,27 @@ static void check_mixer(const LayeredModel& m, int i, const fl_layer_desc& d, bo
 static void check_layer(const LayeredModel& m, int i, const fl_layer_desc& d) {
     const std::string at = "layer " + std::to_string(i) + ": ";
     check_mixer(m, i, d, false);
-    FL_CHECK(d.ffn_act == FL_ACT_SWISH_CLAMP || d.ffn_act == FL_ACT_GELU_TANH || d.ffn_act == FL_ACT_RELU2 || d.ffn_act == FL_ACT_RELU, FL_ERR_INVALID,
+    FL_CHECK(d.ffn_act == FL_ACT_SWISH_CLAMP || d.ffn_act == FL_ACT_GELU_TANH || d.ffn_act == FL_ACT_RELU2 || d.ffn_act == FL_ACT_RELU ||
+                 d.ffn_act == FL_ACT_SILU, FL_ERR_INVALID,
              at + "unknown feed-forward activation");
     FL_CHECK(!(d.ffn_act == FL_ACT_RELU && d.ffn_bias), FL_ERR_UNSUPPORTED, at + "the relu-gated feed-forward has no biases");
-    FL_CHECK(d.ffn != FL_FFN_MOE || ((d.ffn_act == FL_ACT_SWISH_CLAMP || d.ffn_act == FL_ACT_RELU2) && !d.ffn_bias), FL_ERR_UNSUPPORTED,
-             at + "experts use the clamped or the squared-relu activation, without biases");
+    FL_CHECK(d.ffn != FL_FFN_MOE || ((d.ffn_act == FL_ACT_SWISH_CLAMP || d.ffn_act == FL_ACT_RELU2 || d.ffn_act == FL_ACT_SILU) && !d.ffn_bias),
+             FL_ERR_UNSUPPORTED, at + "experts use the clamped swish, the silu or the squared-relu activation, without biases");
     FL_CHECK(!(d.ffn_act == FL_ACT_RELU2 && d.ffn_bias), FL_ERR_UNSUPPORTED, at + "the squared-relu feed-forward has no biases");
     if (d.ffn == FL_FFN_DENSE) {
         FL_CHECK(d.ff >= 1, FL_ERR_INVALID, at + "ff must be positive");
     } else if (d.ffn == FL_FFN_MOE) {
         FL_CHECK(d.ff >= 1 && d.experts >= 1 && d.experts <= 1024 && d.top >= 1 && d.top <= d.experts && d.shared_ff >= 0, FL_ERR_INVALID,
                  at + "bad expert counts");
-        FL_CHECK(d.router == FL_ROUTER_SOFTMAX || d.router == FL_ROUTER_SIGMOID_GROUPS, FL_ERR_INVALID, at + "unknown router");
-        if (d.router == FL_ROUTER_SIGMOID_GROUPS) {
+        FL_CHECK(d.router == FL_ROUTER_SOFTMAX || d.router == FL_ROUTER_SIGMOID_GROUPS || d.router == FL_ROUTER_SOFTMAX_GROUPS, FL_ERR_INVALID,
+                 at + "unknown router");
+        if (d.router != FL_ROUTER_SOFTMAX) {
             FL_CHECK(d.route_groups >= 1 && d.experts % d.route_groups == 0 && d.route_keep >= 1 && d.route_keep <= d.route_groups, FL_ERR_INVALID,
                      at + "experts must divide into route_groups groups of which 1..route_groups are kept");
             FL_CHECK(d.top <= d.route_keep * (d.experts / d.route_groups), FL_ERR_INVALID, at + "the kept groups hold fewer than `top` experts");
-            FL_CHECK(d.shared_ff == 0, FL_ERR_UNSUPPORTED, at + "the sigmoid router has no shared expert");
-            FL_CHECK(!d.router_bias, FL_ERR_UNSUPPORTED, at + "the sigmoid router has a choice correction, not a bias");
+            FL_CHECK(d.shared_ff == 0 || (d.router == FL_ROUTER_SOFTMAX_GROUPS && d.shared_plain), FL_ERR_UNSUPPORTED,
+                     at + "beside a router with groups a shared expert is built for softmax scores, ungated");
+            FL_CHECK(!d.router_bias, FL_ERR_UNSUPPORTED, at + "a router with groups has no bias");
         }
     } else {
         FL_CHECK(d.ffn == FL_FFN_NONE, FL_ERR_INVALID, at + "unknown feed-forward kind");
@@ -135,7 +147,7 @@ static void check_layer(const LayeredModel& m, int i, const fl_layer_desc& d) {
 void layered_build(LayeredModel& m, const fl_layer_desc* descs) {
     const fl_stack_config& c = m.cfg;
     FL_CHECK(c.arch == FL_ARCH_NIFUNEX || c.arch == FL_ARCH_ROFETAR || c.arch == FL_ARCH_TOZARAX || c.arch == FL_ARCH_MEDULORN ||
-                 c.arch == FL_ARCH_LATODRA, FL_ERR_INVALID,
+                 c.arch == FL_ARCH_LATODRA || c.arch == FL_ARCH_TUFAZEN, FL_ERR_INVALID,
              "layered models: unknown arch");
     FL_CHECK(c.vocab >= 1 && c.width >= 1 && c.n_layers >= 1 && c.n_layers <= 4096, FL_ERR_INVALID, "layered models: sizes must be positive");
     FL_CHECK(c.compute_dtype == FL_DTYPE_BF16 || c.compute_dtype == FL_DTYPE_F32, FL_ERR_INVALID, "compute_dtype must be bf16 or f32");
@@ -151,10 +163,20 @@ void layered_build(LayeredModel& m, const fl_layer_desc* descs) {
     const bool both_norms = !c.no_pre_norm && !c.no_post_norm && !c.post_sum_norm;
     FL_CHECK(!c.layer_scale || both_norms, FL_ERR_UNSUPPORTED, "layer scales are built for stacks with a norm before and after every sublayer");
     FL_CHECK(!(c.tied_head && c.max_positions > 0), FL_ERR_UNSUPPORTED, "a tied output projection with a position table is not built");
+    FL_CHECK(c.no_post_norm || !(c.parallel_sub || c.norm_tanh || c.token_side > 0), FL_ERR_UNSUPPORTED,
+             "parallel sublayers, tanh norms and token vectors are built for stacks whose sublayer results join the stream un-normed");
+    FL_CHECK(!c.parallel_sub || (c.canon_taps == 0 && !c.gated_residual && !c.depth_avg && !c.token_shift), FL_ERR_UNSUPPORTED,
+             "parallel sublayers are built without input convolutions, gated contributions, depth average and token shift");
+    FL_CHECK(c.token_side >= 0 && c.bigram_buckets >= 0 && c.bigram_mul_prev >= 0 && c.bigram_mul_cur >= 0, FL_ERR_INVALID, "bad token vector / bigram sizes");
+    // the hash is taken in 64-bit
+    FL_CHECK(c.bigram_buckets == 0 || (c.bigram_mul_prev <= INT64_MAX / 2 / c.vocab && c.bigram_mul_cur <= INT64_MAX / 2 / c.vocab), FL_ERR_UNSUPPORTED,
+             "bigram multipliers too large");
+    FL_CHECK(c.token_side == 0 || !c.depth_avg, FL_ERR_UNSUPPORTED, "token vectors and a depth average do not go together");
+    FL_CHECK(c.bigram_buckets == 0 || !(c.embed_norm || c.tied_head), FL_ERR_UNSUPPORTED, "a bigram table is built for plain, untied embeddings");
     if (c.loop_times > 0) {
         FL_CHECK(c.loop_start >= 0 && c.loop_stop > c.loop_start && c.loop_stop <= c.n_layers && c.loop_times <= 4096, FL_ERR_INVALID, "bad loop span");
-        FL_CHECK(both_norms || !(c.loop_reinject || c.loop_step), FL_ERR_UNSUPPORTED,
-                 "what a loop adds between its passes is built for stacks with a norm before and after every sublayer");
+        FL_CHECK(both_norms || c.no_post_norm || !(c.loop_reinject || c.loop_step), FL_ERR_UNSUPPORTED,
+                 "what a loop adds between its passes is built for stacks with a norm before every sublayer");
         FL_CHECK(!c.depth_avg, FL_ERR_UNSUPPORTED, "a loop and a depth average do not go together");
     } else {
         FL_CHECK(c.loop_times == 0 && !c.loop_reinject && !c.loop_step, FL_ERR_INVALID, "loop options without a loop");
@@ -168,6 +190,9 @@ void layered_build(LayeredModel& m, const fl_layer_desc* descs) {
     reg(&m.embed, (size_t)m.V * W * 2); reg(&m.final_norm, W * 4);
     if (!c.tied_head) reg(&m.head, (size_t)m.V * W * 2);
     if (c.embed_norm) reg(&m.embed_norm, W * 4);
+    if (c.norm_tanh) { reg(&m.final_bias, W * 4); reg(&m.final_alpha, 4); }
+    if (c.bigram_buckets > 0) reg(&m.bigram, ((size_t)c.bigram_buckets + 1) * W * 2);
+    if (c.token_side > 0) reg(&m.side_embed, (size_t)m.V * m.L * c.token_side * 2);
     if (c.loop_step) reg(&m.loop_step, (size_t)c.loop_times * W * 4);
     // the order of computation: the layers before the loop, its passes, the layers behind it
     const bool loop = c.loop_times > 0;
@@ -200,13 +225,14 @@ void layered_build(LayeredModel& m, const fl_layer_desc* descs) {
         if (d.mixer == FL_MIXER_ATTN) {
             if (lw.d.kv_heads <= 0) lw.d.kv_heads = lw.d.heads;
             const size_t G = lw.d.kv_heads;
-            lw.off_q = 0; lw.n_in = (int)(H * D); lw.off_k = lw.off_v = -1;
+            lw.off_q = 0; lw.n_in = (int)(H * D); lw.off_k = lw.off_v = lw.off_g = -1;
             if (!d.no_qk_norm) reg(&lw.qnorm, (d.qk_norm_whole ? H * D : D) * 4);
             if (d.qkv_bias) { reg(&lw.bq, H * D * 4); reg(&lw.bk, G * D * 4); reg(&lw.bv, G * Dv * 4); }
             if (d.sink == 2) reg(&lw.sinkv, H * 4);
             m.max_av = std::max<int>(m.max_av, (int)Dv);
             if (d.kv_from < 0) {
-                lw.off_k = lw.n_in; lw.off_v = lw.off_k + (int)(G * D); lw.n_in = lw.off_v + (int)(G * Dv);
+                lw.off_k = lw.n_in; lw.n_in += (int)(G * D);
+                if (!d.v_from_k) { lw.off_v = lw.n_in; lw.n_in += (int)(G * Dv); }
                 if (!d.no_qk_norm) reg(&lw.knorm, (d.qk_norm_whole ? G * D : D) * 4);
                 lw.kv_owner = i;
                 lw.kv_index = (int)m.kv_layers.size();
@@ -216,6 +242,7 @@ void layered_build(LayeredModel& m, const fl_layer_desc* descs) {
                 lw.kv_owner = d.kv_from;
                 lw.kv_index = m.layers[d.kv_from].kv_index;
             }
+            if (d.out_gate) { lw.off_g = lw.n_in; lw.n_in += (int)(d.out_gate == 2 ? H : H * Dv); }
             lw.n_in = pad8(lw.n_in);
             rope();
         } else if (d.mixer == FL_MIXER_MAMBA2) {
@@ -271,7 +298,7 @@ void layered_build(LayeredModel& m, const fl_layer_desc* descs) {
                 lw.kv_owner = d.kv_from;
                 lw.kv_index = m.layers[d.kv_from].kv_index;
             }
-            if (d.out_gate) { lw.off_g = lw.n_in; lw.n_in += (int)(H * Dv); }
+            if (d.out_gate) { lw.off_g = lw.n_in; lw.n_in += (int)(d.out_gate == 2 ? H : H * Dv); }
             if (Q > 0 || d.out_gate) lw.n_in = pad8(lw.n_in);
             if (d.sink == 2) reg(&lw.sinkv, H * 4);
             reg(&lw.uk_t, H * C * D * 2); reg(&lw.uv, H * Dv * C * 2);
@@ -283,7 +310,15 @@ void layered_build(LayeredModel& m, const fl_layer_desc* descs) {
                 if (*o >= 0) *o += base;
             lw.conv_off += base;
         }
-        reg(&lw.w_o, W * H * Dv * 2);
+        lw.fx = 0;
+        if (c.parallel_sub && d.ffn != FL_FFN_NONE) lw.fx = d.ffn == FL_FFN_DENSE ? d.ff : d.shared_ff;
+        lw.u_ld = (int)(H * Dv) + lw.fx;
+        if (lw.fx > 0) {
+            lw.off_ff = pad8(lw.n_in);
+            lw.n_in = pad8(lw.off_ff + (d.ffn_act == FL_ACT_RELU2 ? 1 : 2) * lw.fx);
+        }
+        reg(&lw.w_o, W * lw.u_ld * 2);
+        m.max_u = std::max(m.max_u, lw.u_ld);
         m.max_hv = std::max<int>(m.max_hv, (int)(H * Dv));
         m.max_cv = std::max(m.max_cv, lw.conv_ch);
     };
@@ -295,7 +330,14 @@ void layered_build(LayeredModel& m, const fl_layer_desc* descs) {
         check_layer(m, i, d);
         const bool pre = !c.no_pre_norm, post = !c.no_post_norm;
         if (pre) reg(&lw.norm1, W * 4);
+        if (c.norm_tanh) { reg(&lw.norm1_bias, W * 4); reg(&lw.norm1_alpha, 4); }
         if (post) reg(&lw.norm1b, W * 4);
+        FL_CHECK(!(c.parallel_sub && (d.beside || d.ffn_bias || (d.ffn == FL_FFN_MOE && d.shared_ff > 0 && !d.shared_plain))), FL_ERR_UNSUPPORTED,
+                 "parallel sublayers are built for one mixer, a feed-forward without biases and an ungated shared expert");
+        if (c.token_side > 0) {
+            const size_t S = c.token_side;
+            reg(&lw.side_gate, S * W * 2); reg(&lw.side_proj, W * S * 2); reg(&lw.side_norm, W * 4);
+        }
         if (c.layer_scale) reg(&lw.ls1, W * 4);
         if (c.token_shift) reg(&lw.shift, W * 4);
         build_mixer(lw, i, 0);
@@ -317,14 +359,16 @@ void layered_build(LayeredModel& m, const fl_layer_desc* descs) {
         if (c.gated_residual) { reg(&lw.rg1, W * W * 2); reg(&lw.rg1b, W * 4); }
         if (c.depth_avg) reg(&lw.dwa, (size_t)(i + 2) * 4);
         if (d.ffn != FL_FFN_NONE) {
-            if (pre) reg(&lw.norm2, W * 4);
+            const bool par = c.parallel_sub != 0;       // one norm per layer; the always-on part lives in w_in and w_o
+            if (pre && !par) reg(&lw.norm2, W * 4);
+            if (c.norm_tanh && !par) { reg(&lw.norm2_bias, W * 4); reg(&lw.norm2_alpha, 4); }
             if (post) reg(&lw.norm2b, W * 4);
             if (c.layer_scale) reg(&lw.ls2, W * 4);
             if (c.canon_taps > 0) reg(&lw.canon2, W * c.canon_taps * 4);
             if (c.gated_residual) { reg(&lw.rg2, W * W * 2); reg(&lw.rg2b, W * 4); }
             if (d.ffn == FL_FFN_DENSE && d.ffn_bias) { reg(&lw.b_gu, (size_t)2 * d.ff * 4); reg(&lw.b_down, W * 4); }
             const size_t G = d.ffn == FL_FFN_MOE ? d.experts : 1, F = d.ff, GF = d.ffn_act == FL_ACT_RELU2 ? F : 2 * F;
-            reg(&lw.w_gu, G * GF * W * 2); reg(&lw.w_down, G * W * F * 2);
+            if (!par || d.ffn == FL_FFN_MOE) { reg(&lw.w_gu, G * GF * W * 2); reg(&lw.w_down, G * W * F * 2); }
             m.max_ff = std::max<int>(m.max_ff, (int)F);
             m.max_top = std::max(m.max_top, d.ffn == FL_FFN_MOE ? d.top : 1);
             if (d.ffn == FL_FFN_MOE) {
@@ -332,7 +376,7 @@ void layered_build(LayeredModel& m, const fl_layer_desc* descs) {
                 if (d.router_bias) reg(&lw.router_b, (size_t)d.experts * 4);
                 if (d.router == FL_ROUTER_SIGMOID_GROUPS) reg(&lw.route_corr, (size_t)d.experts * 4);
                 m.max_experts = std::max(m.max_experts, d.experts);
-                if (d.shared_ff > 0) {
+                if (d.shared_ff > 0 && !par) {
                     reg(&lw.s_gu, (size_t)2 * d.shared_ff * W * 2); reg(&lw.s_down, W * (size_t)d.shared_ff * 2);
                     if (!d.shared_plain) reg(&lw.shared_gate, W * 4);
                     m.max_ff = std::max(m.max_ff, d.shared_ff);
@@ -346,17 +390,33 @@ void layered_build(LayeredModel& m, const fl_layer_desc* descs) {
     size_t off = 0;
     for (const Reg& r : regs) { *r.pp = m.slab.p + off; off += up256(r.bytes); }
     if (c.tied_head) m.head = m.embed;
-    m.weight_bytes = total - (c.tied_head ? 0 : up256((size_t)m.V * W * 2)) - (c.max_positions > 0 ? up256((size_t)c.max_positions * W * 2) : 0);
+    m.weight_bytes = total - (c.tied_head ? 0 : up256((size_t)m.V * W * 2)) - (c.max_positions > 0 ? up256((size_t)c.max_positions * W * 2) : 0) -
+                     (m.bigram ? up256(((size_t)c.bigram_buckets + 1) * W * 2) : 0) - (m.side_embed ? up256((size_t)m.V * m.L * c.token_side * 2) : 0);
 
     // names -> destinations
     LayeredRoutes R;
     auto mat = [&](const std::string& n, uint16_t* base, int64_t row0, int64_t rows, int64_t cols) {
         R.r[n] = LyRoute{LyRoute::MAT16, base + row0 * cols, rows, cols, 0};
     };
+    auto mat_cols = [&](const std::string& n, uint16_t* base, int64_t ld, int64_t col0, int64_t rows, int64_t cols) {     // columns of a wider matrix
+        R.r[n] = LyRoute{LyRoute::MAT16, base + col0, rows, cols, 0, ld};
+    };
+    // rows whose rotary pairs arrive as halves (see LyRoute)
+    auto turned = [&](const std::string& n, const fl_layer_desc& d, int per, int at) {
+        if (!d.rot_halves) return;
+        LyRoute& r = R.r[n];
+        r.turn_per = per; r.turn_at = at; r.turn_dims = d.rot_dims;
+    };
     auto vec = [&](const std::string& n, float* base, int64_t rows, int64_t cols) { R.r[n] = LyRoute{LyRoute::F32, base, rows, cols, 0}; };
     // a layer norm's weight: [W], or one number for all channels (norm_scalar), kept as W equal floats so that the kernels index it alike
     auto normw = [&](const std::string& n, float* base) { R.r[n] = LyRoute{c.norm_scalar ? LyRoute::F32_FILL : LyRoute::F32, base, (int64_t)W, 1, 0}; };
+    auto tanh_parts = [&](const std::string& n, float* b, float* alpha) {
+        if (b != nullptr) { vec(n + ".b", b, W, 1); vec(n + ".alpha", alpha, 1, 1); }
+    };
     mat("embed", m.embed, 0, m.V, W); normw("final.norm", m.final_norm);
+    tanh_parts("final.norm", m.final_bias, m.final_alpha);
+    if (m.bigram != nullptr) mat("bigram", m.bigram, 0, (int64_t)c.bigram_buckets + 1, W);
+    if (m.side_embed != nullptr) mat("side.embed", m.side_embed, 0, m.V, (int64_t)m.L * c.token_side);
     if (!c.tied_head) mat("head", m.head, 0, m.V, W);
     if (m.embed_norm != nullptr) normw("embed.norm", m.embed_norm);
     if (m.loop_step != nullptr) vec("loop.step", m.loop_step, c.loop_times, W);
@@ -370,10 +430,13 @@ void layered_build(LayeredModel& m, const fl_layer_desc* descs) {
             mat(p + "q", lw.w_in, lw.off_q, H * D, W);
             if (!d.no_qk_norm) vec(p + "q.norm", lw.qnorm, d.qk_norm_whole ? H * D : D, 1);
             if (d.kv_from < 0) {
-                mat(p + "k", lw.w_in, lw.off_k, G * D, W); mat(p + "v", lw.w_in, lw.off_v, G * Dv, W);
+                mat(p + "k", lw.w_in, lw.off_k, G * D, W);
+                if (lw.off_v >= 0) mat(p + "v", lw.w_in, lw.off_v, G * Dv, W);
                 if (!d.no_qk_norm) vec(p + "k.norm", lw.knorm, d.qk_norm_whole ? G * D : D, 1);
             }
-            if (d.qkv_bias) { vec(p + "q.b", lw.bq, H * D, 1); vec(p + "k.b", lw.bk, G * D, 1); vec(p + "v.b", lw.bv, G * Dv, 1); }
+            if (d.qkv_bias) { vec(p + "q.b", lw.bq, H * D, 1); vec(p + "k.b", lw.bk, G * D, 1); }
+            if (d.qkv_bias && lw.off_v >= 0) vec(p + "v.b", lw.bv, G * Dv, 1);
+            if (d.out_gate) mat(p + "g", lw.w_in, lw.off_g, d.out_gate == 2 ? H : H * Dv, W);
             if (d.sink == 2) vec(p + "sink", lw.sinkv, H, 1);
         } else if (d.mixer == FL_MIXER_MAMBA2) {
             mat(p + "in", lw.w_in, lw.off_g, lw.off_dt - lw.off_g + H, W);
@@ -403,16 +466,18 @@ void layered_build(LayeredModel& m, const fl_layer_desc* descs) {
             const int64_t Rr = d.rot_dim, C = d.kv_rank, Q = d.q_rank;
             if (Q > 0) {
                 mat(p + "dq", lw.w_in, lw.off_q, Q, W); vec(p + "dq.norm", lw.dq_norm, Q, 1); mat(p + "uq", lw.uq, 0, H * (D + Rr), Q);
+                turned(p + "uq", d, (int)(D + Rr), (int)D);
             } else {
                 mat(p + "q", lw.w_in, lw.off_q, H * (D + Rr), W);
+                turned(p + "q", d, (int)(D + Rr), (int)D);
             }
-            if (d.out_gate) mat(p + "g", lw.w_in, lw.off_g, H * Dv, W);
+            if (d.out_gate) mat(p + "g", lw.w_in, lw.off_g, d.out_gate == 2 ? H : H * Dv, W);
             if (d.sink == 2) vec(p + "sink", lw.sinkv, H, 1);
-            if (d.kv_from < 0) { mat(p + "dkv", lw.w_in, lw.off_dkv, C + Rr, W); vec(p + "dkv.norm", lw.dkv_norm, C, 1); }
+            if (d.kv_from < 0) { mat(p + "dkv", lw.w_in, lw.off_dkv, C + Rr, W); turned(p + "dkv", d, (int)(C + Rr), (int)C); vec(p + "dkv.norm", lw.dkv_norm, C, 1); }
             R.r[p + "uk"] = LyRoute{LyRoute::UK_T, lw.uk_t, H * D, C, (int)H};
             mat(p + "uv", lw.uv, 0, H * Dv, C);
         }
-        mat(p + "o", lw.w_o, 0, W, H * Dv);
+        mat_cols(p + "o", lw.w_o, lw.u_ld, 0, W, H * Dv);
     };
     for (int i = 0; i < m.L; ++i) {
         LayeredLayerW& lw = m.layers[i];
@@ -421,6 +486,11 @@ void layered_build(LayeredModel& m, const fl_layer_desc* descs) {
         const bool pre = !c.no_pre_norm, post = !c.no_post_norm;
         if (pre && post) { normw(p + "norm1", lw.norm1); normw(p + "norm1b", lw.norm1b); }
         else normw(p + "norm1", pre ? lw.norm1 : lw.norm1b);
+        tanh_parts(p + "norm1", lw.norm1_bias, lw.norm1_alpha);
+        if (lw.side_gate) {
+            mat(p + "side.gate", lw.side_gate, 0, c.token_side, W); mat(p + "side.proj", lw.side_proj, 0, W, c.token_side);
+            vec(p + "side.norm", lw.side_norm, W, 1);
+        }
         if (lw.shift) vec(p + "shift", lw.shift, W, 1);
         if (lw.ls1) vec(p + "ls1", lw.ls1, W, 1);
         if (lw.ls2) vec(p + "ls2", lw.ls2, W, 1);
@@ -436,13 +506,23 @@ void layered_build(LayeredModel& m, const fl_layer_desc* descs) {
         if (lw.dwa) vec(p + "dwa", lw.dwa, i + 2, 1);
         if (d.ffn == FL_FFN_NONE) continue;
         if (pre && post) { normw(p + "norm2", lw.norm2); normw(p + "norm2b", lw.norm2b); }
-        else normw(p + "norm2", pre ? lw.norm2 : lw.norm2b);
+        else if (!c.parallel_sub) normw(p + "norm2", pre ? lw.norm2 : lw.norm2b);
+        tanh_parts(p + "norm2", lw.norm2_bias, lw.norm2_alpha);
+        // the always-on feed-forward of parallel sublayers: rows of w_in, columns of w_o
+        auto always_on = [&](const std::string& q) {
+            const bool has_gate = d.ffn_act != FL_ACT_RELU2;
+            if (has_gate) mat(q + "gate", lw.w_in, lw.off_ff, lw.fx, W);
+            mat(q + "up", lw.w_in, lw.off_ff + (has_gate ? lw.fx : 0), lw.fx, W);
+            mat_cols(q + "down", lw.w_o, lw.u_ld, lw.u_ld - lw.fx, W, lw.fx);
+        };
         if (lw.canon2) vec(p + "canon2", lw.canon2, W, c.canon_taps);
         if (lw.rg2) { mat(p + "rg2", lw.rg2, 0, W, W); vec(p + "rg2.b", lw.rg2b, W, 1); }
         const int64_t F = d.ff;
         const bool gated = d.ffn_act != FL_ACT_RELU2;
         const int64_t GF = gated ? 2 * F : F;
-        if (d.ffn == FL_FFN_DENSE) {
+        if (d.ffn == FL_FFN_DENSE && c.parallel_sub) {
+            always_on(p + "mlp.");
+        } else if (d.ffn == FL_FFN_DENSE) {
             if (gated) mat(p + "mlp.gate", lw.w_gu, 0, F, W);
             mat(p + "mlp.up", lw.w_gu, gated ? F : 0, F, W); mat(p + "mlp.down", lw.w_down, 0, W, F);
             if (d.ffn_bias) {
@@ -458,7 +538,9 @@ void layered_build(LayeredModel& m, const fl_layer_desc* descs) {
                 mat(q + "up", lw.w_gu, (int64_t)e * GF + (gated ? F : 0), F, W);
                 mat(q + "down", lw.w_down, (int64_t)e * W, W, F);
             }
-            if (d.shared_ff > 0) {
+            if (d.shared_ff > 0 && c.parallel_sub) {
+                always_on(p + "mlp.shared.");
+            } else if (d.shared_ff > 0) {
                 const int64_t Fs = d.shared_ff;
                 mat(p + "mlp.shared.gate", lw.s_gu, 0, Fs, W); mat(p + "mlp.shared.up", lw.s_gu, Fs, Fs, W);
                 mat(p + "mlp.shared.down", lw.s_down, 0, W, Fs);
@@ -487,7 +569,7 @@ void layered_put_tensor(LayeredModel& m, const char* name, int dtype, const int6
     for (int i = 0; i < rank; ++i) numel *= shape[i];
     const bool shape_ok = r->kind == LyRoute::F32_FILL
                               ? numel == 1
-                              : numel == r->rows * r->cols && (rank == 1 || (rank == 2 && (shape[0] == r->rows || r->cols == 1 || r->rows == 1)));
+                              : numel == r->rows * r->cols && (rank == 0 || rank == 1 || (rank == 2 && (shape[0] == r->rows || r->cols == 1 || r->rows == 1)));
     FL_CHECK(shape_ok, FL_ERR_INVALID, std::string("shape mismatch for ") + name);
     FL_CHECK(dtype == FL_DTYPE_F32 || dtype == FL_DTYPE_BF16 || dtype == FL_DTYPE_F16, FL_ERR_INVALID, "bad dtype");
     if (r->kind == LyRoute::F32_RAW && dtype == FL_DTYPE_F32) {
@@ -500,7 +582,17 @@ void layered_put_tensor(LayeredModel& m, const char* name, int dtype, const int6
     else if (dtype == FL_DTYPE_F32) for (int64_t i = 0; i < numel; ++i) bits[i] = f32_to_bits(((const float*)host)[i]);
     else for (int64_t i = 0; i < numel; ++i) bits[i] = f32_to_bits(half_to_f32(((const uint16_t*)host)[i]));
     if (r->kind == LyRoute::MAT16) {
-        FL_CUDA(cudaMemcpy(r->dst, bits.data(), (size_t)numel * 2, cudaMemcpyHostToDevice));
+        if (r->turn_dims > 0) {
+            std::vector<uint16_t> t(bits);
+            const int half = r->turn_dims / 2;
+            for (int64_t b = 0; b < r->rows; b += r->turn_per)
+                for (int i = 0; i < r->turn_dims; ++i)
+                    std::memcpy(t.data() + (size_t)(b + r->turn_at + i) * r->cols, bits.data() + (size_t)(b + r->turn_at + (i & 1) * half + i / 2) * r->cols,
+                                (size_t)r->cols * 2);
+            bits.swap(t);
+        }
+        const int64_t ld = r->ld > 0 ? r->ld : r->cols;
+        FL_CUDA(cudaMemcpy2D(r->dst, (size_t)ld * 2, bits.data(), (size_t)r->cols * 2, (size_t)r->cols * 2, (size_t)r->rows, cudaMemcpyHostToDevice));
     } else if (r->kind == LyRoute::F32 || r->kind == LyRoute::F32_RAW) {
         std::vector<float> v((size_t)numel);
         for (int64_t i = 0; i < numel; ++i) v[i] = bits_to_f32(bits[i]);
@@ -529,20 +621,23 @@ void layered_random_init(LayeredModel& m, uint64_t seed, float stdv) {
         if (r->kind == LyRoute::F32 || r->kind == LyRoute::F32_RAW || r->kind == LyRoute::F32_FILL) {
             auto ends = [&](const char* t) { const size_t k = std::strlen(t); return n.size() >= k && n.compare(n.size() - k, k, t) == 0; };
             // a plain norm weight sits around one, a zero-centred one around zero
-            const bool around_one = ends("mix.norm") || ends("left.norm") || ends("right.norm") || ends("dkv.norm") || ends("dq.norm") || n == "embed.norm" || ends(".ls1") || ends(".ls2") || ends("q.norm") || ends("k.norm") || ends("mix.D") || ends("left.out") || ends("right.out") ||
+            const bool around_one = ends("mix.norm") || ends("left.norm") || ends("right.norm") || ends("dkv.norm") || ends("dq.norm") || n == "embed.norm" || ends(".ls1") || ends(".ls2") || ends("side.norm") || ends("q.norm") || ends("k.norm") || ends("mix.D") || ends("left.out") || ends("right.out") ||
                                     (m.cfg.norm_plain && (ends("norm1") || ends("norm2") || ends("norm1b") || ends("norm2b") || n == "final.norm"));
             const bool is_mat = n.find("router") != std::string::npos || n.find("mix.a2") != std::string::npos || n.find("shared.sg") != std::string::npos ||
                                 ends(".conv") || ends(".canon1") || ends(".canon2") || n == "loop.step";
             const bool is_bias = n.size() >= 4 && n.compare(n.size() - 4, 4, "a2.b") == 0;
             if (around_one) fill_f32_kernel<<<8, 256>>>((float*)r->dst, numel, 1.0f);
             else if (ends(".decay")) fill_f32_kernel<<<8, 256>>>((float*)r->dst, numel, 0.96875f);
+            else if (ends(".alpha")) fill_f32_kernel<<<8, 256>>>((float*)r->dst, numel, 0.5f);
             else if (ends(".shift")) fill_f32_kernel<<<8, 256>>>((float*)r->dst, numel, 0.25f);
             else if (ends(".dwa")) fill_f32_kernel<<<8, 256>>>((float*)r->dst, numel, 1.0f / (float)numel);     // a plain mean over the outputs so far
             else if (is_bias) fill_f32_kernel<<<8, 256>>>((float*)r->dst, numel, 3.0f);
             else if (is_mat) synth_fill_f32_kernel<<<kNumSMs, 256>>>((float*)r->dst, numel, ts, stdv, ident);
             else fill_f32_kernel<<<8, 256>>>((float*)r->dst, numel, 0.0f);
         } else {
-            synth_fill_bf16_kernel<<<kNumSMs * 8, 256>>>((uint16_t*)r->dst, 1, numel, numel, ts, n == "embed" && !m.cfg.tied_head ? 1.0f : stdv, ident);
+            const bool unit = (n == "embed" && !m.cfg.tied_head) || n == "bigram" || n == "side.embed";
+            if (r->ld > 0) synth_fill_bf16_kernel<<<kNumSMs * 8, 256>>>((uint16_t*)r->dst, r->rows, r->cols, r->ld, ts, stdv, ident);
+            else synth_fill_bf16_kernel<<<kNumSMs * 8, 256>>>((uint16_t*)r->dst, 1, numel, numel, ts, unit ? 1.0f : stdv, ident);
         }
         g_launches.fetch_add(1);
         m.have.insert(n);
@@ -558,10 +653,10 @@ void layered_finalize(LayeredModel& m) {
         std::lock_guard<std::mutex> g(g_routes_mu);
         g_routes.erase(&m);
     }
-    // serving precision: the projections whose shapes fit the tcgen05 GEMM's tiles (whole 64-column k blocks, 16-byte rows) run
-    // there; everything else, and every product of the exact mode, stays on the f32 FMA kernel
+    // serving precision: the projections whose rows are whole 16-byte pieces run on the tcgen05 GEMM (a K that ends inside a 64-column
+    // k block is filled up with zeros by the tensor maps of both operands); everything else, and every product of the exact mode, stays on the f32 FMA kernel
     if (!m.f32 && !env_flag("FL_LAYERED_NO_TC")) {
-        auto fits = [](int N, int K) { return K % 64 == 0 && N % 8 == 0; };
+        auto fits = [](int N, int K) { return K % 8 == 0 && N % 8 == 0; };
         auto map = [&](const uint16_t* p, int N, int K, CUtensorMap& tm, bool& ok) {
             ok = p != nullptr && fits(N, K);
             if (ok) tm = make_tmap_bf16(p, (uint64_t)N, (uint64_t)K, (uint64_t)K, 128);
@@ -569,15 +664,15 @@ void layered_finalize(LayeredModel& m) {
         for (LayeredLayerW& lw : m.layers) {
             const fl_layer_desc& d = lw.d;
             map(lw.w_in, lw.n_in, m.W, lw.tm_in, lw.tc_in);
-            map(lw.w_o, m.W, d.heads * d.vdim, lw.tm_o, lw.tc_o);
+            map(lw.w_o, m.W, lw.u_ld, lw.tm_o, lw.tc_o);
             if (d.mixer == FL_MIXER_LATENT_ATTN) {
                 // sizes in multiples of 8 may end inside a k block (the tensor maps fill its rest with zeros)
                 const int H = d.heads, D = d.dim, Dv = d.vdim, C = d.kv_rank, R = d.rot_dim;
-                lw.lat_tc = D % 8 == 0 && Dv % 8 == 0 && C % 8 == 0 && R % 8 == 0 && m.W % 8 == 0 && (lw.off_g < 0 || lw.off_g % 4 == 0) && lw.n_in % 4 == 0;
+                lw.lat_tc = D % 8 == 0 && Dv % 8 == 0 && C % 8 == 0 && R % 8 == 0 && m.W % 8 == 0 && lw.u_ld % 8 == 0 &&
+                            (d.out_gate != 1 || lw.off_g % 4 == 0) && lw.n_in % 4 == 0;
                 if (lw.lat_tc) {
                     lw.tm_uk = make_tmap_bf16(lw.uk_t, (uint64_t)H * C, (uint64_t)D, (uint64_t)D, 128);
                     lw.tm_uv = make_tmap_bf16(lw.uv, (uint64_t)H * Dv, (uint64_t)C, (uint64_t)C, 128);
-                    if (!lw.tc_o) { lw.tc_o = true; lw.tm_o = make_tmap_bf16(lw.w_o, (uint64_t)m.W, (uint64_t)H * Dv, (uint64_t)H * Dv, 128); }
                     m.max_hp = std::max(m.max_hp, H * D); m.max_hq = std::max(m.max_hq, H * ((C + R + 63) / 64 * 64)); m.max_c = std::max(m.max_c, C);
                 }
             }
@@ -590,6 +685,7 @@ void layered_finalize(LayeredModel& m) {
             if (lw.side) map(lw.side->w_o, m.W, lw.side->d.heads * lw.side->d.vdim, lw.side->tm_o, lw.side->tc_o);
             map(lw.rg1, m.W, m.W, lw.tm_rg1, lw.tc_rg1); map(lw.rg2, m.W, m.W, lw.tm_rg2, lw.tc_rg2);
             const int GF = d.ffn_act == FL_ACT_RELU2 ? d.ff : 2 * d.ff;       // rows of the first feed-forward matrix: up, or gate | up
+            map(lw.side_gate, m.cfg.token_side, m.W, lw.tm_tgate, lw.tc_tgate); map(lw.side_proj, m.W, m.cfg.token_side, lw.tm_tproj, lw.tc_tproj);
             if (d.ffn == FL_FFN_DENSE) { map(lw.w_gu, GF, m.W, lw.tm_gu, lw.tc_gu); map(lw.w_down, m.W, d.ff, lw.tm_down, lw.tc_down); }
             if (d.ffn == FL_FFN_MOE && d.shared_ff > 0) {
                 map(lw.s_gu, 2 * d.shared_ff, m.W, lw.tm_sgu, lw.tc_sgu); map(lw.s_down, m.W, d.shared_ff, lw.tm_sdown, lw.tc_sdown);
@@ -607,7 +703,7 @@ void layered_finalize(LayeredModel& m) {
         map(m.head, m.V, m.W, m.tm_head, m.tc_head);
     }
     // the norms behind a sublayer park a row in shared memory: above the default 48 KB the kernels are told so once
-    if (!m.cfg.no_post_norm && (size_t)m.W * 4 > 48 * 1024) {
+    if ((!m.cfg.no_post_norm || m.cfg.token_side > 0) && (size_t)m.W * 4 > 48 * 1024) {
         FL_CHECK((size_t)m.W * 4 <= 200 * 1024, FL_ERR_UNSUPPORTED, "norms behind a sublayer are built for widths up to 51200");
         FL_CUDA(cudaFuncSetAttribute(ly_post_norm_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, m.W * 4));
         FL_CUDA(cudaFuncSetAttribute(ly_post_norm_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, m.W * 4));
@@ -654,6 +750,12 @@ static void rope_tables(const RopeSpec& rs, int max_seq, std::vector<float>& cs,
         }
 }
 
+static KvLayout kv_layout(const fl_layer_desc& d) {
+    const int G = d.kv_heads, D = d.dim, Dv = d.vdim, r = d.rot_dims;
+    if (d.v_from_k) return KvLayout{G * (D + r), D + r, r, D + r, r == D ? 0 : r};
+    return KvLayout{G * (D + Dv), D, G * D, Dv, 0};
+}
+
 void layered_cache_create(fl_cache& c, int max_slots, int max_seq, int pool_tokens) {
     const LayeredModel& m = *c.lm;
     FL_CHECK(m.finalized, FL_ERR_STATE, "model not finalized");
@@ -670,7 +772,7 @@ void layered_cache_create(fl_cache& c, int max_slots, int max_seq, int pool_toke
     y.kv_store.resize(m.kv_layers.size());
     for (size_t k = 0; k < m.kv_layers.size(); ++k) {
         const fl_layer_desc& d = m.kv_layers[k]->d;
-        const size_t width = d.mixer == FL_MIXER_ATTN ? (size_t)d.kv_heads * (d.dim + d.vdim) : (size_t)(d.kv_rank + d.rot_dim);
+        const size_t width = d.mixer == FL_MIXER_ATTN ? (size_t)kv_layout(d).E : (size_t)(d.kv_rank + d.rot_dim);
         y.kv_store[k].alloc((size_t)pages * kKvPage * width * esz, true);
         y.kv_pool.push_back(y.kv_store[k].p);
     }
@@ -708,12 +810,14 @@ void layered_cache_create(fl_cache& c, int max_slots, int max_seq, int pool_toke
         y.at_part.alloc(part);
     }
     c.slot_len.assign(max_slots, 0);
+    y.slot_last.assign(max_slots, -1);
     FL_CUDA(cudaDeviceSynchronize());
 }
 
 void layered_slot_reset(fl_cache& c, int slot) {
     c.ly->pool.release(slot);       // the recurrent state needs no clearing: a sequence that starts at position 0 starts from zero
     c.slot_len[slot] = 0;
+    c.ly->slot_last[slot] = -1;
 }
 
 void layered_cache_reset(fl_cache& c) {
@@ -735,7 +839,7 @@ static void ensure_ws(fl_cache& c, size_t T, size_t n_want) {
         drop_graphs(c);
         const size_t R = std::max<size_t>(T, 2 * y.rows), W = m.W, P = R * std::max(m.max_top, 1);
         y.x.alloc(R * W); y.h.alloc(R * W); y.y.alloc(R * W);
-        y.proj.alloc(R * m.max_in); y.u.alloc(R * std::max(m.max_hv, 1)); y.go.alloc(R * std::max(m.max_hv, 1));
+        y.proj.alloc(R * m.max_in); y.u.alloc(R * std::max(m.max_u, 1)); y.go.alloc(R * std::max(m.max_hv, 1));
         y.la.alloc(R * std::max(m.max_hd, 1));
         y.cv.alloc(R * std::max(m.max_cv, 1)); y.rs.alloc(R * 2 * std::max(m.max_heads, 1));
         if (m.cfg.canon_taps > 0 || m.cfg.token_shift) y.hc.alloc(R * W);
@@ -743,8 +847,9 @@ static void ensure_ws(fl_cache& c, size_t T, size_t n_want) {
         if (m.cfg.depth_avg) y.xs.alloc((size_t)(m.L + 1) * R * W);
         else if (m.cfg.loop_reinject) y.xs.alloc(R * W);
         if (m.max_qr > 0) { y.cq.alloc(R * m.max_qr); y.qx.alloc(R * m.max_q); }
+        if (m.cfg.token_side > 0) { y.tz.alloc(R * m.cfg.token_side); y.ta.alloc(R * m.cfg.token_side); }
         for (const LayeredLayerW& lw : m.layers)
-            if (lw.side && y.y2.n < R * W) y.y2.alloc(R * W);
+            if ((lw.side || (m.cfg.parallel_sub && lw.d.ffn == FL_FFN_MOE)) && y.y2.n < R * W) y.y2.alloc(R * W);
         bool plain_latent = false;          // a latent attention that is not on the tensor cores keeps f32 query / value rows
         for (const LayeredLayerW& lw : m.layers) plain_latent |= lw.d.mixer == FL_MIXER_LATENT_ATTN && !lw.lat_tc;
         if (plain_latent) { y.qa.alloc(R * m.max_hc); y.ol.alloc(R * m.max_hc); }
@@ -759,10 +864,11 @@ static void ensure_ws(fl_cache& c, size_t T, size_t n_want) {
         if (!m.f32) {
             y.h_hi.alloc(R * W); y.h_lo.alloc(R * W);
             if (m.max_qr > 0) { y.cq_hi.alloc(R * m.max_qr); y.cq_lo.alloc(R * m.max_qr); }
-            y.u_hi.alloc(R * std::max(m.max_hv, 1)); y.u_lo.alloc(R * std::max(m.max_hv, 1));
+            y.u_hi.alloc(R * std::max(m.max_u, 1)); y.u_lo.alloc(R * std::max(m.max_u, 1));
+            if (m.cfg.token_side > 0) { y.ta_hi.alloc(R * m.cfg.token_side); y.ta_lo.alloc(R * m.cfg.token_side); }
             y.act_hi.alloc(R * std::max(m.max_ff, 1)); y.act_lo.alloc(R * std::max(m.max_ff, 1));
             // split-K slices of a tensor-core GEMM with <= 128 rows: ks * rows <= 256 (see pick_ksplit)
-            const size_t nmax = std::max<size_t>(std::max<size_t>(std::max(m.max_in, m.max_q), W), std::max<size_t>(2 * (size_t)m.max_ff, m.V));
+            const size_t nmax = std::max<size_t>(std::max<size_t>(std::max(m.max_in, m.max_q), W), std::max<size_t>(std::max<size_t>(2 * (size_t)m.max_ff, m.cfg.token_side), m.V));
             size_t need = 256 * nmax;
             size_t gx_rows = 0;
             for (const LayeredLayerW& lw : m.layers) {          // grouped expert GEMMs: [slices][experts * cap rows][2 ff | W]
@@ -826,10 +932,17 @@ static void gemm_tc_or_exact(fl_cache& c, LaunchCtx& lc, const char* tag, const 
                s.p, s.n, s.stride, s.stride, Y);
 }
 // feed-forward activation of `rows` rows (see ly_glu_kernel)
-static void launch_glu(LaunchCtx& lc, const Slices& gu, int rows, int F, float limit, int act, const float* bias, float* out, uint16_t* hi, uint16_t* lo) {
+// (ldg, ldo: row strides of gu and of the output; 0 = dense rows.  gu.p, out, hi, lo may start inside a row.)
+static void launch_glu(LaunchCtx& lc, const Slices& gu, int rows, int F, float limit, int act, const float* bias, float* out, uint16_t* hi, uint16_t* lo, int ldg = 0,
+                       int ldo = 0) {
     if (rows <= 0) return;
-    if (F % 4 == 0) launch(lc, "glu", 0, ly_glu_kernel<4>, dim3(rows, (F + 1023) / 1024), dim3(256), 0, gu, F, limit, act, bias, out, hi, lo);
-    else launch(lc, "glu", 0, ly_glu_kernel<1>, dim3(rows, (F + 255) / 256), dim3(256), 0, gu, F, limit, act, bias, out, hi, lo);
+    if (ldg == 0) ldg = act == FL_ACT_RELU2 ? F : 2 * F;
+    if (ldo == 0) ldo = F;
+    auto al = [](const void* p, size_t n) { return (reinterpret_cast<uintptr_t>(p) & (n - 1)) == 0; };
+    if (((F | ldg | ldo) & 3) == 0 && (gu.stride & 3) == 0 && al(gu.p, 16) && al(out, 16) && al(hi, 8) && al(lo, 8))
+        launch(lc, "glu", 0, ly_glu_kernel<4>, dim3(rows, (F + 1023) / 1024), dim3(256), 0, gu, ldg, ldo, F, limit, act, bias, out, hi, lo);
+    else
+        launch(lc, "glu", 0, ly_glu_kernel<1>, dim3(rows, (F + 255) / 256), dim3(256), 0, gu, ldg, ldo, F, limit, act, bias, out, hi, lo);
 }
 
 static void gemm_groups(LaunchCtx& lc, const char* tag, const LyGemm& g, int groups, int max_rows) {
@@ -878,7 +991,7 @@ static void launch_latent_mma(LaunchCtx& lc, const LatMmaArgs& a, int T, int max
     if (wide) go(std::integral_constant<int, 2>{}); else go(std::integral_constant<int, 1>{});
     if (splits > 1)
         launch(lc, "latent_merge", 0, ly_gqa_merge_kernel, dim3(T, a.H), dim3(std::min(256, (a.C + 31) / 32 * 32)), 0, (const float*)a.part, splits, a.H, a.C, a.sink,
-               a.sinkv, a.row_base, (float*)nullptr, a.ohi, a.olo);
+               a.sinkv, a.row_base, a.H * a.C, 0, OutGate{}, (float*)nullptr, a.ohi, a.olo);
 }
 
 static void launch_gla_scan(LaunchCtx& lc, const GlaArgs& a, int n) {
@@ -920,7 +1033,7 @@ static void launch_gqa_attn(LaunchCtx& lc, const GqaAttnArgs& a, int T, int max_
     else launch_gqa_attn_rb<CT, 1>(lc, a, T, splits);
     if (splits > 1)
         launch(lc, "gqa_merge", 0, ly_gqa_merge_kernel, dim3(T, a.H), dim3(std::min(256, std::max(32, (a.Dv + 31) / 32 * 32))), 0, (const float*)a.part, splits,
-               a.H, a.Dv, a.sink, a.sinkv, a.row_base, a.out, a.ohi, a.olo);
+               a.H, a.Dv, a.sink, a.sinkv, a.row_base, a.ldo, a.kv.roll, a.gate, a.out, a.ohi, a.olo);
 }
 
 template <bool DELTA>
@@ -1024,7 +1137,7 @@ static void latent_attn_tc(fl_cache& c, LaunchCtx& lc, const LatentAttnArgs& a, 
 // sink, causal mask) and a value GEMM; the block size keeps a score block within a fixed scratch budget.
 static void gqa_attn_tc(fl_cache& c, LaunchCtx& lc, const GqaAttnArgs& a, int r0, int Ts, int pos0, int slot) {
     LayeredCache& y = *c.ly;
-    const int H = a.H, G = a.G, rep = H / G, D = a.D, Dv = a.Dv, Dp = (D + 63) / 64 * 64, E = G * (D + Dv);
+    const int H = a.H, G = a.G, rep = H / G, D = a.D, Dv = a.Dv, Dp = (D + 63) / 64 * 64;
     const size_t budget = (size_t)48 << 20;                // floats in a score block (192 MB); P halves take the same again
     // first key of the contiguous range a position reads (window and chunk starts only grow with the position, so a block of
     // rows needs the keys from its first row's start on), and the kept first keys that lie before it
@@ -1060,8 +1173,8 @@ static void gqa_attn_tc(fl_cache& c, LaunchCtx& lc, const GqaAttnArgs& a, int r0
             continue;
         }
         for (int g = 0; g < G; ++g) {
-            launch(lc, "gqa_gather_kv", 0, ly_gqa_gather_kv_kernel, dim3(nkp), dim3(128), 0, (const uint16_t*)a.pool, page_row, k_lo, n_first, nk, nkp, E, g * D, D,
-                   Dp, G * D + g * Dv, Dv, y.at_kc.p, y.at_kct.p);
+            launch(lc, "gqa_gather_kv", 0, ly_gqa_gather_kv_kernel, dim3(nkp), dim3(128), 0, (const uint16_t*)a.pool, page_row, k_lo, n_first, nk, nkp, a.kv.E,
+                   g * a.kv.ks, D, Dp, a.kv.vo + g * a.kv.vs, Dv, a.kv.roll, y.at_kc.p, y.at_kct.p);
             launch(lc, "gqa_build_q", 0, ly_gqa_build_q_kernel, dim3(nq, rep), dim3(128), 0, a.proj, a.ldp, a.off_q, r0 + f, rep, g, D, Dp, a.scale, y.at_qhi.p,
                    y.at_qlo.p);
             const CUtensorMap tk = make_tmap_bf16(y.at_kc.p, (uint64_t)nkp, (uint64_t)Dp, (uint64_t)Dp, 128);
@@ -1073,7 +1186,7 @@ static void gqa_attn_tc(fl_cache& c, LaunchCtx& lc, const GqaAttnArgs& a, int r0
         }
         const size_t no = (size_t)nq * H * Dv;
         launch(lc, "gqa_scatter", 0, ly_gqa_scatter_kernel, dim3((unsigned)std::min<size_t>(4 * kNumSMs, (no + 255) / 256)), dim3(256), 0, (const float*)y.at_o.p, nq,
-               G, rep, Dv, r0 + f, a.out, a.ohi, a.olo);
+               G, rep, Dv, r0 + f, a.ldo, a.gate, a.out, a.ohi, a.olo);
     }
 }
 
@@ -1105,7 +1218,7 @@ void layered_forward(fl_cache& c, const int* slots, const int* counts, int n, co
     for (long long i = 0; i < T; ++i) FL_CHECK(ids[i] < (uint32_t)m.V, FL_ERR_INVALID, "token id out of range");
     for (int k = 0; k < n_want; ++k) FL_CHECK(want[k] >= 0 && want[k] < T, FL_ERR_INVALID, "wanted row out of range");
     ensure_ws(c, (size_t)T, (size_t)n_want);
-    const size_t tab_ints = (size_t)3 * T + 3 * (size_t)n + 1 + (size_t)n_want;
+    const size_t tab_ints = (size_t)4 * T + 3 * (size_t)n + 1 + (size_t)n_want;
     if (tab_ints > y.tab_cap) {
         FL_CUDA(cudaStreamSynchronize(c.stream));
         drop_graphs(c);
@@ -1115,12 +1228,15 @@ void layered_forward(fl_cache& c, const int* slots, const int* counts, int n, co
     FL_CUDA(cudaStreamSynchronize(c.stream));      // the pinned staging buffers of the previous step are free again
     int* ht = y.h_step_tab.p;
     int *h_tok = ht, *h_rseq = ht + T, *h_rpos = ht + 2 * T, *h_row0 = ht + 3 * T, *h_slot = h_row0 + n + 1, *h_pos0 = h_slot + n,
-        *h_want = h_pos0 + n;
+        *h_want = h_pos0 + n, *h_prev = h_want + n_want;
     int row = 0;
     for (int i = 0; i < n; ++i) {
         const int sl = slots[i];
         h_row0[i] = row; h_slot[i] = sl; h_pos0[i] = c.slot_len[sl];
-        for (int k = 0; k < counts[i]; ++k, ++row) { h_tok[row] = (int)ids[row]; h_rseq[row] = i; h_rpos[row] = c.slot_len[sl] + k; }
+        int before_tok = y.slot_last[sl];           // -1 for a slot that holds nothing
+        for (int k = 0; k < counts[i]; ++k, ++row) {
+            h_prev[row] = before_tok;
+            before_tok = (int)ids[row]; h_tok[row] = (int)ids[row]; h_rseq[row] = i; h_rpos[row] = c.slot_len[sl] + k; }
         const int before = y.pool.held(sl);
         y.pool.grow(sl, c.slot_len[sl] + counts[i]);
         if (y.pool.held(sl) != before)
@@ -1131,7 +1247,7 @@ void layered_forward(fl_cache& c, const int* slots, const int* counts, int n, co
     for (int k = 0; k < n_want; ++k) h_want[k] = want[k];
     FL_CUDA(cudaMemcpyAsync(y.step_tab.p, ht, tab_ints * 4, cudaMemcpyHostToDevice, c.stream));
     const int* dt = y.step_tab.p;
-    StepTab st{dt, dt + T, dt + 2 * T, dt + 3 * T, dt + 3 * T + n + 1, dt + 3 * T + 2 * n + 1, dt + 3 * T + 3 * n + 1, (int)T, n, n_want};
+    StepTab st{dt, dt + T, dt + 2 * T, dt + 3 * T, dt + 3 * T + n + 1, dt + 3 * T + 2 * n + 1, dt + 3 * T + 3 * n + 1, dt + 3 * T + 3 * n + 1 + n_want, (int)T, n, n_want};
 
     // ---- device: layer by layer over all rows of the step ----
     LaunchCtx lc;
@@ -1175,7 +1291,11 @@ void layered_forward(fl_cache& c, const int* slots, const int* counts, int n, co
     }
     if (n_want > 0)
         FL_CUDA(cudaMemcpyAsync(y.h_logits.p, y.logits.p, (size_t)n_want * m.V * 4, cudaMemcpyDeviceToHost, c.stream));
-    for (int i = 0; i < n; ++i) c.slot_len[slots[i]] += counts[i];
+    for (int i = 0, r = 0; i < n; ++i) {
+        c.slot_len[slots[i]] += counts[i];
+        r += counts[i];
+        y.slot_last[slots[i]] = (int)ids[r - 1];
+    }
 }
 
 // One mixer over all rows of the step (`pass`: which pass of a loop, 0 elsewhere -- its own cache and state): reads its columns of the projected buffer y.proj (row stride lw.n_in; `in`: the same as
@@ -1191,11 +1311,15 @@ static void run_mixer(fl_cache& c, LaunchCtx& lc, const StepTab& st, const Layer
     const float eps = m.cfg.norm_eps;
     const int kv_index = lw.kv_index + pass, gla_index = lw.gla_index + pass;
     uint16_t *uhi = m.f32 ? nullptr : y.u_hi.p, *ulo = m.f32 ? nullptr : y.u_lo.p;
+    const int ldu = lw.u_ld;
+    const OutGate gate = d.out_gate ? OutGate{y.proj.p + lw.off_g, lw.n_in, d.out_gate == 2 ? 1 : Dv, d.out_gate == 2 ? 0 : 1} : OutGate{};
+    const int n_gate = d.out_gate == 0 ? 0 : (d.out_gate == 2 ? H : H * Dv);
     if (d.mixer == FL_MIXER_ATTN) {
         const int G = d.kv_heads;
+        const KvLayout kv = kv_layout(d);
         AttnPrepArgs pa{y.proj.p, lw.n_in, lw.off_q, lw.off_k, lw.off_v, lw.qnorm, lw.knorm, eps, y.kv_pool[kv_index], y.page_table.p,
                         c.pages_per_seq, st.row_seq, st.row_pos, st.seq_slot, y.rope_cos[lw.rope_index].p, y.rope_sin[lw.rope_index].p,
-                        H, G, D, Dv, d.rot_dims, d.rot_halves, lw.bq, lw.bk, lw.bv, d.qk_norm_whole};
+                        H, G, D, Dv, d.rot_dims, d.rot_halves, lw.bq, lw.bk, lw.bv, d.qk_norm_whole, kv, in, lw.off_g, n_gate};
         // eight warps per block take the heads in turn; steps of few rows spread a row's heads over up to four blocks (not with a
         // norm over the whole projection: its sums read every head before any is rewritten in place, which one block orders)
         const size_t psm = (size_t)8 * D * 4;
@@ -1204,7 +1328,7 @@ static void run_mixer(fl_cache& c, LaunchCtx& lc, const StepTab& st, const Layer
         else launch(lc, "attn_prep", 0, ly_attn_prep_kernel<uint16_t>, dim3(Ti, py), dim3(256), psm, pa);
         GqaAttnArgs at{y.proj.p, lw.n_in, lw.off_q, y.kv_pool[kv_index], y.page_table.p, c.pages_per_seq, st.row_seq, st.row_pos, st.seq_slot,
                        y.u.p, lw.tc_o ? uhi : (uint16_t*)nullptr, ulo, H, G, D, Dv, d.window, d.scale, d.softcap, d.sink, 0, y.at_part.p,
-                       d.keep_first, d.mask_chunk, lw.sinkv};
+                       d.keep_first, d.mask_chunk, lw.sinkv, kv, ldu, gate};
         // a step of single tokens is replayed from a captured graph whatever the contexts' lengths: its split count must not follow them
         int max_keys = c.max_seq;
         if (Ti != n) {
@@ -1255,12 +1379,12 @@ static void run_mixer(fl_cache& c, LaunchCtx& lc, const StepTab& st, const Layer
         if (delta) {
             launch_rec_scan<true>(lc, ra, n);
             launch(lc, "gla_out", 0, ly_gla_out_kernel, dim3((Ti * H + 7) / 8), dim3(256), 0, (const float*)y.go.p, (const float*)y.proj.p, lw.n_in, lw.off_g,
-                   (const float*)lw.hnorm, eps, Ti, H, Dv, y.u.p, lw.tc_o ? uhi : (uint16_t*)nullptr, ulo);
+                   (const float*)lw.hnorm, eps, Ti, H, Dv, ldu, y.u.p, lw.tc_o ? uhi : (uint16_t*)nullptr, ulo);
         } else {
             launch_rec_scan<false>(lc, ra, n);
             const int inner = H * Dv, part = inner / d.norm_groups;
             launch(lc, "gated_group_norm", 0, ly_gated_group_norm_kernel, dim3(Ti, d.norm_groups), dim3(std::min(1024, std::max(64, (part + 31) / 32 * 32))), 0,
-                   (const float*)y.go.p, (const float*)y.proj.p, lw.n_in, lw.off_g, (const float*)lw.hnorm, eps, inner, d.norm_groups, 0, y.u.p,
+                   (const float*)y.go.p, (const float*)y.proj.p, lw.n_in, lw.off_g, (const float*)lw.hnorm, eps, inner, d.norm_groups, 0, ldu, y.u.p,
                    lw.tc_o ? uhi : (uint16_t*)nullptr, ulo);
         }
     } else if (d.mixer == FL_MIXER_LIGHTNING) {
@@ -1270,9 +1394,9 @@ static void run_mixer(fl_cache& c, LaunchCtx& lc, const StepTab& st, const Layer
         RecArgs ra{y.cv.p, lw.conv_ch, lw.off_q - lw.conv_off, lw.off_k - lw.conv_off, lw.off_v - lw.conv_off, y.rs.p, (const float*)nullptr, y.go.p,
                    y.gla_state[gla_index].p, st.seq_row0, st.seq_slot, st.seq_pos0, H, H, D, Dv};
         launch_rec_scan<false>(lc, ra, n);
-        const bool v4 = ((inner | lw.n_in | lw.off_g) & 3) == 0;       // four channels per thread
+        const bool v4 = ((inner | lw.n_in | lw.off_g | ldu) & 3) == 0;       // four channels per thread
         launch(lc, "gated_group_norm", 0, ly_gated_group_norm_kernel, dim3(Ti, 1), dim3(std::min(v4 ? 256 : 1024, std::max(64, ((v4 ? inner / 4 : inner) + 31) / 32 * 32))), 0,
-               (const float*)y.go.p, (const float*)y.proj.p, lw.n_in, lw.off_g, (const float*)lw.hnorm, eps, inner, 1, 1, y.u.p,
+               (const float*)y.go.p, (const float*)y.proj.p, lw.n_in, lw.off_g, (const float*)lw.hnorm, eps, inner, 1, 1, ldu, y.u.p,
                lw.tc_o ? uhi : (uint16_t*)nullptr, ulo);
     } else if (d.mixer == FL_MIXER_GLA) {
         // decay pre-activation through the rank-r bottleneck: z = W_a2 a (the bias and the sigmoid^(1/tau) are applied by the scan)
@@ -1281,12 +1405,12 @@ static void run_mixer(fl_cache& c, LaunchCtx& lc, const StepTab& st, const Layer
                    st.seq_slot, st.seq_pos0, H, D, Dv, (float)(1.0 / std::sqrt((double)D))};
         launch_gla_scan(lc, ga, n);
         launch(lc, "gla_out", 0, ly_gla_out_kernel, dim3((Ti * H + 7) / 8), dim3(256), 0, (const float*)ga.o, (const float*)y.proj.p, lw.n_in, lw.off_g,
-               (const float*)lw.hnorm, eps, Ti, H, Dv, y.u.p, lw.tc_o ? uhi : (uint16_t*)nullptr, ulo);
+               (const float*)lw.hnorm, eps, Ti, H, Dv, ldu, y.u.p, lw.tc_o ? uhi : (uint16_t*)nullptr, ulo);
     } else {
         const int R = d.rot_dim, C = d.kv_rank, Q = d.q_rank;
         LatentAppendArgs aa{y.proj.p, lw.n_in, lw.off_q, lw.off_dkv, lw.dkv_norm, eps, y.kv_pool[kv_index], y.page_table.p, c.pages_per_seq,
                             st.row_seq, st.row_pos, st.seq_slot, y.rope_cos[lw.rope_index].p, y.rope_sin[lw.rope_index].p, H, D, R, C, d.rot_dims, lw.off_q, Q, lw.dq_norm, lw.tc_uq ? (float*)nullptr : y.cq.p,
-                            lw.tc_uq ? y.cq_hi.p : (uint16_t*)nullptr, y.cq_lo.p, in, lw.off_g, d.out_gate ? H * Dv : 0};
+                            lw.tc_uq ? y.cq_hi.p : (uint16_t*)nullptr, y.cq_lo.p, in, lw.off_g, n_gate};
         const int ath = Ti <= 2 * kNumSMs ? std::min(1024, std::max(128, (Q + C + 31) / 32 * 32)) : 128;
         if (m.f32) launch(lc, "latent_append", 0, ly_latent_append_kernel<float>, dim3(Ti), dim3(ath), 0, aa);
         else launch(lc, "latent_append", 0, ly_latent_append_kernel<uint16_t>, dim3(Ti), dim3(ath), 0, aa);
@@ -1344,8 +1468,8 @@ static void run_mixer(fl_cache& c, LaunchCtx& lc, const StepTab& st, const Layer
                 t.row_base = first;
                 launch_latent_mma(lc, t, rows, max_keys);
             });
-            dense_gemm_blocks(c, lc, "gemm_v_expand", Ti, H, Dv, C, lw.tm_uv, y.ol_hi.p, y.ol_lo.p, uhi, ulo, H * Dv, Dv,
-                              d.out_gate ? (const float*)y.proj.p + lw.off_g : (const float*)nullptr, d.out_gate ? lw.n_in : 0);
+            dense_gemm_blocks(c, lc, "gemm_v_expand", Ti, H, Dv, C, lw.tm_uv, y.ol_hi.p, y.ol_lo.p, uhi, ulo, ldu, Dv, gate.g,
+                              gate.ld, d.out_gate == 2);
             return;
         }
         // q~[row, h, :] = W_uk[h]^T q_plain[row, h, :]: the score against the latent needs no per-head keys
@@ -1359,16 +1483,11 @@ static void run_mixer(fl_cache& c, LaunchCtx& lc, const StepTab& st, const Layer
             if (m.f32) launch_latent_attn<float>(lc, t, rows); else launch_latent_attn<uint16_t>(lc, t, rows);
         });
         // value expansion after the softmax: out[row, h, :] = W_uv[h] (sum_j p_j c_j)
-        LyGemm ov{y.ol.p, C, H * C, nullptr, lw.uv, (long long)Dv * C, Dv, C, y.u.p, Dv, H * Dv, nullptr, Ti};
+        LyGemm ov{y.ol.p, C, H * C, nullptr, lw.uv, (long long)Dv * C, Dv, C, y.u.p, Dv, ldu, nullptr, Ti};
         gemm_groups(lc, "gemm_v_expand", ov, H, Ti);
-        const size_t nu = (size_t)Ti * H * Dv;
-        if (d.out_gate) {
-            launch(lc, "out_gate", 0, ly_out_gate_kernel, dim3((unsigned)std::min<size_t>(4 * kNumSMs, (nu + 255) / 256)), dim3(256), 0, y.u.p, (const float*)y.proj.p,
-                   lw.n_in, lw.off_g, H * Dv, Ti, lw.tc_o ? uhi : (uint16_t*)nullptr, ulo);
-        } else if (lw.tc_o) {
-            launch(lc, "split_hi_lo", 0, ly_split_kernel, dim3((unsigned)std::min<size_t>(4 * kNumSMs, (nu + 255) / 256)), dim3(256), 0,
-                   (const float*)y.u.p, nu, uhi, ulo);
-        }
+        if (d.out_gate || lw.tc_o)
+            launch(lc, d.out_gate ? "out_gate" : "split_hi_lo", 0, ly_out_gate_kernel, dim3((unsigned)std::min<size_t>(4 * kNumSMs, ((size_t)Ti * H * Dv + 255) / 256)),
+                   dim3(256), 0, y.u.p, ldu, gate, H, Dv, Ti, lw.tc_o ? uhi : (uint16_t*)nullptr, ulo);
     }
 }
 
@@ -1389,11 +1508,20 @@ static void enqueue_step(fl_cache& c, LaunchCtx& lc, const StepTab& st, const in
     const bool pre = !m.cfg.no_pre_norm, post = !m.cfg.no_post_norm, canon = m.cfg.canon_taps > 0, gated = m.cfg.gated_residual != 0,
                depth = m.cfg.depth_avg != 0;
     const int plain = m.cfg.norm_plain ? 1 : 0, split_x = pre ? 0 : 1;
+    const bool par = m.cfg.parallel_sub != 0, tside = m.cfg.token_side > 0;
+    auto norm_of = [&](const float* w, const float* b, const float* alpha) { return NormW{w, b, alpha, plain}; };
+    auto norm1_of = [&](int r) { const LayeredLayerW& l = m.layers[m.runs[r].layer]; return norm_of(l.norm1, l.norm1_bias, l.norm1_alpha); };
+    // whether a run's mixer input is read as hi | lo halves only (routed experts' routers and the FMA kernels read f32 rows)
+    auto halves_only = [&](int r) {
+        const LayeredLayerW& l = m.layers[m.runs[r].layer];
+        return l.tc_in && !canon && !gated && !(par && l.d.ffn == FL_FFN_MOE);
+    };
     const float* norm_out = pre ? y.h.p : y.x.p;                // what the arrangement hands to a sublayer
     const float* sub_in = canon ? y.hc.p : norm_out;            // what the sublayer's own matrices read
     const size_t hist_stride = y.rows * (size_t)W;
     launch(lc, "embed_norm", 0, ly_embed_norm_kernel, dim3(Ti), dim3(nthr), 0, (const uint16_t*)m.embed, st.tok, W,
-           pre ? (const float*)m.layers[0].norm1 : (const float*)nullptr, eps, plain, (const uint16_t*)m.pos, st.row_pos, m.cfg.embed_scale, (const float*)m.embed_norm,
+           pre ? norm1_of(0) : NormW{}, eps, plain, (const uint16_t*)m.pos, st.row_pos, m.cfg.embed_scale, (const float*)m.embed_norm,
+           BigramTab{m.bigram, st.prev, m.cfg.bigram_buckets, (long long)m.cfg.bigram_mul_prev, (long long)m.cfg.bigram_mul_cur},
            m.runs[0].pass_start ? (const float*)m.loop_step : (const float*)nullptr, y.x.p, depth || m.cfg.loop_reinject ? y.xs.p : (float*)nullptr, y.h.p, hhi, hlo);
     // in front of a sublayer: the gate's pre-activation from the normed input, then the input convolution (and its carried inputs)
     auto sublayer_front = [&](const LayeredLayerW& lw, int run, int sub) {
@@ -1436,25 +1564,27 @@ static void enqueue_step(fl_cache& c, LaunchCtx& lc, const StepTab& st, const in
             launch(lc, "sum_norm", 0, ly_sum_norm_kernel<1>, dim3(Ti), dim3(nthr), (size_t)W * 4, y.x.p, (const float*)y.y.p, yb, y2, m.cfg.residual_alpha, sa, sb,
                    w, eps, W, plain, split, hhi, hlo);
     };
-    // a sublayer's result (y.y, and y2 beside it) joins the stream; four channels per thread when the rows are 16-byte multiples
-    auto join = [&](const float* y2, const float* wa, const float* wb, const float* gate_bias, int hist_slot, const float* dw, const float* wnext) {
+    // a sublayer's result (and y2 beside it) joins the stream; four channels per thread when the rows are 16-byte multiples
+    // (hout == nullptr: what comes next reads the hi | lo halves alone; split: without a next norm, the halves of the stream itself)
+    auto join = [&](const Slices& yv, const float* y2, const float* wa, const float* wb, const float* gate_bias, int hist_slot, const float* dw, const float* x0,
+                    const float* step, NormW next, int split, float* hout) {
         const float* gz = gated ? (const float*)y.gz.p : (const float*)nullptr;
         if (W % 4 == 0)
-            launch(lc, "join", 0, ly_join_kernel<4>, dim3(Ti), dim3(std::min(256, std::max(32, (W / 4 + 31) / 32 * 32))), 0, y.x.p, (const float*)y.y.p, y2, wa, wb,
-                   gz, gate_bias, y.xs.p, hist_stride, hist_slot, dw, wnext, eps, W, plain, y.h.p, hhi, hlo);
+            launch(lc, "join", 0, ly_join_kernel<4>, dim3(Ti), dim3(std::min(Ti <= kNumSMs ? 1024 : 256, std::max(32, (W / 4 + 31) / 32 * 32))), 0, y.x.p, yv, y2, wa, wb,
+                   gz, gate_bias, y.xs.p, hist_stride, hist_slot, dw, x0, step, next, eps, W, split, hout, hhi, hlo);
         else
-            launch(lc, "join", 0, ly_join_kernel<1>, dim3(Ti), dim3(nthr), 0, y.x.p, (const float*)y.y.p, y2, wa, wb, gz, gate_bias, y.xs.p, hist_stride,
-                   hist_slot, dw, wnext, eps, W, plain, y.h.p, hhi, hlo);
+            launch(lc, "join", 0, ly_join_kernel<1>, dim3(Ti), dim3(nthr), 0, y.x.p, yv, y2, wa, wb, gz, gate_bias, y.xs.p, hist_stride, hist_slot, dw, x0, step, next,
+                   eps, W, split, hout, hhi, hlo);
     };
-    // a sublayer's result (still in split-K slices, perhaps) is normed and joins the stream
-    // (hout == nullptr: the next sublayer's first matrix reads the hi | lo halves alone)
-    auto post_norm = [&](const Slices& yv, const float* yb, const float* wb, const float* wnext, const float* ls, const float* x0, const float* step, int split,
+    // a sublayer's result (still in split-K slices, perhaps) is normed (weight wb, wplain) and joins the stream
+    // (hout as above)
+    auto post_norm = [&](const Slices& yv, const float* yb, const float* wb, int wplain, NormW next, const float* ls, const float* x0, const float* step, int split,
                          float* hout) {
         if (W % 4 == 0)
             launch(lc, "post_norm", 0, ly_post_norm_kernel<4>, dim3(Ti), dim3(std::min(Ti <= kNumSMs ? 1024 : 256, std::max(32, (W / 4 + 31) / 32 * 32))), (size_t)W * 4,
-                   y.x.p, yv, yb, wb, wnext, ls, x0, step, eps, W, plain, split, hout, hhi, hlo);
+                   y.x.p, yv, yb, wb, next, ls, x0, step, eps, W, wplain, split, hout, hhi, hlo);
         else
-            launch(lc, "post_norm", 0, ly_post_norm_kernel<1>, dim3(Ti), dim3(nthr), (size_t)W * 4, y.x.p, yv, yb, wb, wnext, ls, x0, step, eps, W, plain, split, hout,
+            launch(lc, "post_norm", 0, ly_post_norm_kernel<1>, dim3(Ti), dim3(nthr), (size_t)W * 4, y.x.p, yv, yb, wb, next, ls, x0, step, eps, W, wplain, split, hout,
                    hhi, hlo);
     };
     // the other arrangements read the folded rows
@@ -1463,6 +1593,68 @@ static void enqueue_step(fl_cache& c, LaunchCtx& lc, const StepTab& st, const in
             launch(lc, "sum_slices", 0, ly_sum_slices_kernel, dim3((unsigned)std::min<size_t>(4 * kNumSMs, (s.stride + 255) / 256)), dim3(256), 0, s.p, s.n, s.stride,
                    s.stride, y.y.p);
         s = Slices{y.y.p, 1, 0};
+    };
+    // the experts of a layer over all rows: out[row] = sum of the chosen ones' weighted outputs (+ the shared one)
+    auto experts = [&](const LayeredLayerW& lw, float* out) {
+        const fl_layer_desc& d = lw.d;
+        const int F = d.ff, act = d.ffn_act, GF = act == FL_ACT_RELU2 ? F : 2 * F;
+        const int E = d.experts, top = d.top, P = Ti * top;
+        if (d.router != FL_ROUTER_SOFTMAX)
+            launch(lc, "moe_router", 0, ly_router_groups_kernel, dim3(Ti), dim3(256), ((size_t)2 * E + d.route_groups) * 4, sub_in, W, (const float*)lw.router,
+                   E, top, d.router == FL_ROUTER_SOFTMAX_GROUPS ? 1 : 0, (const float*)lw.route_corr, d.route_groups, d.route_keep, d.route_best ? 0 : 1,
+                   d.route_renorm, y.route_sel.p, y.route_w.p);
+        else
+            launch(lc, "moe_router", 0, ly_router_kernel, dim3(Ti), dim3(256), (size_t)E * 4, sub_in, W, (const float*)lw.router, (const float*)lw.router_b, E, top,
+                   (const float*)lw.shared_gate, y.route_sel.p, y.route_w.p, y.sgate.p);
+        const float* sg = lw.shared_gate ? (const float*)y.sgate.p : (const float*)nullptr;    // nullptr: the shared expert counts fully
+        const float* sh = nullptr;
+        if (d.shared_ff > 0 && !par) {  // the always-on expert first (parallel sublayers hold it in the mixer's matrices): its split-K scratch is free again before the routed experts run
+            const int Fs = d.shared_ff;
+            const Slices gu = gemm_slices(c, lc, "gemm_shared_in", sub_in, hhi, hlo, lw.s_gu, lw.tm_sgu, lw.tc_sgu, 2 * Fs, W, y.sh_gu.p, Ti);
+            launch_glu(lc, gu, Ti, Fs, d.shared_limit, act, nullptr, lw.tc_sdown ? (float*)nullptr : y.sh_act.p, lw.tc_sdown ? ahi : (uint16_t*)nullptr, alo);
+            gemm_tc_or_exact(c, lc, "gemm_shared_out", y.sh_act.p, ahi, alo, lw.s_down, lw.tm_sdown, lw.tc_sdown, W, Fs, y.sh_o.p, Ti);
+            sh = y.sh_o.p;
+        }
+        const dim3 gw((W + 255) / 256, Ti);
+        if (lw.tc_moe && Ti > 128) {
+            // many rows: every expert over all rows on the tensor cores, kept where the row picked it (ascending expert order)
+            for (int e = 0; e < E; ++e) {
+                dense_gemm(c, lc, "gemm_tc_moe_in", Ti, GF, W, lw.tm_egu[e], y.gu.p, hhi, hlo);
+                launch_glu(lc, Slices{y.gu.p, 1, 0}, Ti, F, d.limit, act, nullptr, nullptr, ahi, alo);
+                dense_gemm(c, lc, "gemm_tc_moe_out", Ti, W, F, lw.tm_edown[e], y.eo.p, ahi, alo);
+                launch(lc, "moe_accum", 0, ly_moe_accum_kernel, gw, dim3(256), 0, (const float*)y.eo.p, (const int*)y.route_sel.p,
+                       (const float*)y.route_w.p, top, e, (const float*)nullptr, e == 0 ? 1 : 0, W, out);
+            }
+            if (sh != nullptr)
+                launch(lc, "moe_accum", 0, ly_moe_accum_kernel, gw, dim3(256), 0, sh, (const int*)nullptr, (const float*)nullptr, 0, -1,
+                       sg, 0, W, out);
+        } else {
+            launch(lc, "moe_lists", 0, ly_moe_lists_kernel, dim3(E), dim3(32), 0, (const int*)y.route_sel.p, Ti, top, E, y.grp_off.p, y.pair_row.p,
+                   y.pair_of.p);
+            if (lw.tc_moe) {
+                // few rows: ONE grouped GEMM pair over (expert, weight tile, k slice) items; an expert without rows costs nothing
+                const int cap = Ti <= 16 ? 16 : (Ti <= 32 ? 32 : (Ti <= 64 ? 64 : 128));
+                launch(lc, "moe_gather", 0, ly_moe_gather_kernel, dim3(E, std::min(Ti, 16)), dim3(256), 0, (const uint16_t*)hhi, (const uint16_t*)hlo, W,
+                       (const int*)y.grp_off.p, (const int*)y.pair_row.p, cap, y.gx_hi.p, y.gx_lo.p, y.grp_cnt.p);
+                int ks = dense_gemm_grouped(c, lc, "gemm_tc_moe_in", E, cap, GF, W, lw.tm_gu, y.gemm_out.p, y.gx_hi.p, y.gx_lo.p, y.grp_cnt.p);
+                FL_CHECK((size_t)ks * E * cap * GF <= y.gemm_out.n, FL_ERR_STATE, "internal: grouped GEMM scratch too small");
+                launch(lc, "glu_grouped", 0, ly_glu_grouped_kernel, dim3((F + 255) / 256, E * cap), dim3(256), 0, (const float*)y.gemm_out.p, ks,
+                       (size_t)E * cap * GF, F, d.limit, act, (const int*)y.grp_cnt.p, cap, y.ga_hi.p, y.ga_lo.p);
+                ks = dense_gemm_grouped(c, lc, "gemm_tc_moe_out", E, cap, W, F, lw.tm_down, y.gemm_out.p, y.ga_hi.p, y.ga_lo.p, y.grp_cnt.p);
+                FL_CHECK((size_t)ks * E * cap * W <= y.gemm_out.n, FL_ERR_STATE, "internal: grouped GEMM scratch too small");
+                launch(lc, "moe_combine", 0, ly_moe_combine_grouped_kernel, gw, dim3(256), 0, (const float*)y.gemm_out.p, ks, (size_t)E * cap * W,
+                       (const int*)y.route_sel.p, (const int*)y.pair_of.p, (const int*)y.grp_off.p, cap, (const float*)y.route_w.p, top, sh,
+                       sg, W, out);
+            } else {
+                LyGemm g1{sub_in, 0, W, y.pair_row.p, lw.w_gu, (long long)GF * W, GF, W, y.gu.p, 0, GF, y.grp_off.p, P};
+                gemm_groups(lc, "gemm_moe_in", g1, E, P);
+                launch_glu(lc, Slices{y.gu.p, 1, 0}, P, F, d.limit, act, nullptr, y.act.p, nullptr, nullptr);
+                LyGemm g2{y.act.p, 0, F, nullptr, lw.w_down, (long long)W * F, W, F, y.eo.p, 0, W, y.grp_off.p, P};
+                gemm_groups(lc, "gemm_moe_out", g2, E, P);
+                launch(lc, "moe_combine", 0, ly_moe_combine_kernel, gw, dim3(256), 0, (const float*)y.eo.p, (const int*)y.pair_of.p,
+                       (const float*)y.route_w.p, top, sh, sg, W, out);
+            }
+        }
     };
     const int n_runs = (int)m.runs.size();
     for (int run = 0; run < n_runs; ++run) {
@@ -1473,38 +1665,67 @@ static void enqueue_step(fl_cache& c, LaunchCtx& lc, const StepTab& st, const in
         sublayer_front(lw, run, 0);
         if (shifted) shift_front(lw, run);
         Slices in = gemm_slices(c, lc, "gemm_mix_in", shifted ? (const float*)y.hc.p : sub_in, hhi, hlo, lw.w_in, lw.tm_in, lw.tc_in, lw.n_in, W, y.proj.p, Ti);
-        if (in.n > 1 && !(d.mixer == FL_MIXER_LATENT_ATTN && d.q_rank > 0)) {        // only that mixer folds the slices itself
+        const bool folds = !lw.side && (d.mixer == FL_MIXER_ATTN || (d.mixer == FL_MIXER_LATENT_ATTN && d.q_rank > 0));     // mixers that fold the slices themselves
+        if (in.n > 1 && !folds) {
             launch(lc, "sum_slices", 0, ly_sum_slices_kernel, dim3((unsigned)std::min<size_t>(4 * kNumSMs, (in.stride + 255) / 256)), dim3(256), 0, in.p, in.n, in.stride,
                    in.stride, y.proj.p);
             in = Slices{y.proj.p, 1, 0};
         }
-        run_mixer(c, lc, st, lw, in, pass, slots, counts, n, h_row0, h_pos0);
-        Slices mix = gemm_slices(c, lc, "gemm_mix_out", y.u.p, uhi, ulo, lw.w_o, lw.tm_o, lw.tc_o, W, H * Dv, y.y.p, Ti), ff{y.y.p, 1, 0};
-        if (!post || sum_norm || lw.side) fold(mix);
-        if (lw.side) {
-            const LayeredLayerW& sw = *lw.side;
-            run_mixer(c, lc, st, sw, in, pass, slots, counts, n, h_row0, h_pos0);
-            gemm_tc_or_exact(c, lc, "gemm_mix_out", y.u.p, uhi, ulo, sw.w_o, sw.tm_o, sw.tc_o, W, sw.d.heads * sw.d.vdim, y.y2.p, Ti);
-        }
         const bool last = run + 1 == n_runs, has_ff = d.ffn != FL_FFN_NONE;
-        // whether the next sublayer (the feed-forward; the next run's mixer) takes its input as hi | lo halves only
-        const bool ff_halves = lw.tc_gu && d.ffn == FL_FFN_DENSE && !canon && !gated, mix_halves = !last && m.layers[m.runs[run + 1].layer].tc_in && !canon && !gated;
-        const float* next1 = (pre && !last) ? m.layers[m.runs[run + 1].layer].norm1 : nullptr;
+        const NormW next1 = (pre && !last) ? norm1_of(run + 1) : NormW{};
         const int more = last ? 0 : split_x;               // whether another sublayer reads x after this layer
         // what joins the stream between this layer and the next run when that one starts a pass of the loop
         const bool into_pass = !last && m.runs[run + 1].pass_start;
         const int next_pass = into_pass ? m.runs[run + 1].pass : 0;
         const float* again = (into_pass && next_pass > 0 && m.cfg.loop_reinject) ? (const float*)y.xs.p : (const float*)nullptr;
         const float* pstep = (into_pass && m.cfg.loop_step) ? (const float*)m.loop_step + (size_t)next_pass * W : (const float*)nullptr;
+        float* h_next = !last && halves_only(run + 1) ? nullptr : y.h.p;
+        // the layer's last join: behind it (or, with token vectors, behind theirs) the stream gains what a loop adds and the next norm follows
+        auto last_join = [&](const Slices& yv, const float* y2, const float* wa, const float* wb, const float* gate_bias) {
+            const int hist = depth ? li + 1 : -1;
+            if (!tside) { join(yv, y2, wa, wb, gate_bias, hist, lw.dwa, again, pstep, next1, more, h_next); return; }
+            join(yv, y2, wa, wb, gate_bias, -1, nullptr, nullptr, nullptr, NormW{}, lw.tc_tgate ? 1 : 0, nullptr);
+            const int S = m.cfg.token_side;
+            const Slices z = gemm_slices(c, lc, "gemm_side_gate", y.x.p, hhi, hlo, lw.side_gate, lw.tm_tgate, lw.tc_tgate, S, W, y.tz.p, Ti);
+            launch(lc, "token_side", 0, ly_token_side_kernel, dim3(Ti), dim3(std::min(256, (S + 31) / 32 * 32)), 0, z, st.tok,
+                   (const uint16_t*)m.side_embed + (size_t)li * S, (size_t)m.L * S, S, lw.tc_tproj ? (float*)nullptr : y.ta.p,
+                   lw.tc_tproj ? y.ta_hi.p : (uint16_t*)nullptr, y.ta_lo.p);
+            const Slices v = gemm_slices(c, lc, "gemm_side_proj", y.ta.p, y.ta_hi.p, y.ta_lo.p, lw.side_proj, lw.tm_tproj, lw.tc_tproj, W, S, y.y.p, Ti);
+            post_norm(v, nullptr, lw.side_norm, 1, next1, nullptr, again, pstep, more, h_next);
+        };
+        if (par) {          // mixer and feed-forward read the same h and join together
+            const int off = lw.u_ld - lw.fx;
+            if (lw.fx > 0)
+                launch_glu(lc, Slices{in.p + lw.off_ff, in.n, in.stride}, Ti, lw.fx, d.ffn == FL_FFN_MOE ? d.shared_limit : d.limit, d.ffn_act, nullptr,
+                           lw.tc_o ? (float*)nullptr : y.u.p + off, lw.tc_o ? uhi + off : (uint16_t*)nullptr, lw.tc_o ? ulo + off : (uint16_t*)nullptr, lw.n_in, lw.u_ld);
+            run_mixer(c, lc, st, lw, in, pass, slots, counts, n, h_row0, h_pos0);
+            if (d.ffn == FL_FFN_MOE) experts(lw, y.y2.p);
+            const Slices both = gemm_slices(c, lc, "gemm_mix_out", y.u.p, uhi, ulo, lw.w_o, lw.tm_o, lw.tc_o, W, lw.u_ld, y.y.p, Ti);
+            last_join(both, d.ffn == FL_FFN_MOE ? (const float*)y.y2.p : (const float*)nullptr, nullptr, nullptr, nullptr);
+            continue;
+        }
+        run_mixer(c, lc, st, lw, in, pass, slots, counts, n, h_row0, h_pos0);
+        Slices mix = gemm_slices(c, lc, "gemm_mix_out", y.u.p, uhi, ulo, lw.w_o, lw.tm_o, lw.tc_o, W, H * Dv, y.y.p, Ti), ff{y.y.p, 1, 0};
+        if (sum_norm || lw.side) fold(mix);
+        if (lw.side) {
+            const LayeredLayerW& sw = *lw.side;
+            run_mixer(c, lc, st, sw, in, pass, slots, counts, n, h_row0, h_pos0);
+            gemm_tc_or_exact(c, lc, "gemm_mix_out", y.u.p, uhi, ulo, sw.w_o, sw.tm_o, sw.tc_o, W, sw.d.heads * sw.d.vdim, y.y2.p, Ti);
+        }
+        // whether the feed-forward takes its input as hi | lo halves only
+        const bool ff_halves = lw.tc_gu && d.ffn == FL_FFN_DENSE && !canon && !gated;
+        const NormW norm2 = norm_of(lw.norm2, lw.norm2_bias, lw.norm2_alpha);
+        float* h_ff = ff_halves ? nullptr : y.h.p;
         if (sum_norm)
             sum_norm_join(nullptr, lw.side ? (const float*)y.y2.p : (const float*)nullptr, lw.side ? d.out_scale : 1.f, lw.side ? lw.side->d.out_scale : 0.f,
                           lw.norm1b, (has_ff || !shifted) ? (has_ff ? split_x : more) : 0);
         else if (post)
-            post_norm(mix, nullptr, lw.norm1b, has_ff ? (const float*)lw.norm2 : next1, lw.ls1, has_ff ? nullptr : again, has_ff ? nullptr : pstep, has_ff ? split_x : more,
-                      (has_ff ? ff_halves : mix_halves) ? nullptr : y.h.p);
+            post_norm(mix, nullptr, lw.norm1b, plain, has_ff ? norm2 : next1, lw.ls1, has_ff ? nullptr : again, has_ff ? nullptr : pstep, has_ff ? split_x : more,
+                      has_ff ? h_ff : h_next);
+        else if (has_ff)
+            join(mix, lw.side ? (const float*)y.y2.p : (const float*)nullptr, lw.pair_wa, lw.pair_wb, lw.rg1b, -1, nullptr, nullptr, nullptr, norm2, 0, h_ff);
         else
-            join(lw.side ? (const float*)y.y2.p : (const float*)nullptr, lw.pair_wa, lw.pair_wb, lw.rg1b, (depth && !has_ff) ? li + 1 : -1, lw.dwa,
-                 has_ff ? (const float*)lw.norm2 : next1);
+            last_join(mix, lw.side ? (const float*)y.y2.p : (const float*)nullptr, lw.pair_wa, lw.pair_wb, lw.rg1b);
         if (!has_ff) continue;
         sublayer_front(lw, run, 1);
         const int F = d.ff, act = d.ffn_act, GF = act == FL_ACT_RELU2 ? F : 2 * F;
@@ -1512,74 +1733,20 @@ static void enqueue_step(fl_cache& c, LaunchCtx& lc, const StepTab& st, const in
             const Slices gu = gemm_slices(c, lc, "gemm_ff_in", sub_in, hhi, hlo, lw.w_gu, lw.tm_gu, lw.tc_gu, GF, W, y.gu.p, Ti);
             launch_glu(lc, gu, Ti, F, d.limit, act, lw.b_gu, lw.tc_down ? (float*)nullptr : y.act.p, lw.tc_down ? ahi : (uint16_t*)nullptr, alo);
             ff = gemm_slices(c, lc, "gemm_ff_out", y.act.p, ahi, alo, lw.w_down, lw.tm_down, lw.tc_down, W, F, y.y.p, Ti);
-            if (!post || sum_norm) fold(ff);
+            if (sum_norm) fold(ff);
         } else {
-            const int E = d.experts, top = d.top, P = Ti * top;
-            if (d.router == FL_ROUTER_SIGMOID_GROUPS)
-                launch(lc, "moe_router", 0, ly_router_sigmoid_kernel, dim3(Ti), dim3(256), ((size_t)2 * E + d.route_groups) * 4, sub_in, W, (const float*)lw.router,
-                       E, top, (const float*)lw.route_corr, d.route_groups, d.route_keep, y.route_sel.p, y.route_w.p);
-            else
-                launch(lc, "moe_router", 0, ly_router_kernel, dim3(Ti), dim3(256), (size_t)E * 4, sub_in, W, (const float*)lw.router, (const float*)lw.router_b, E, top,
-                       (const float*)lw.shared_gate, y.route_sel.p, y.route_w.p, y.sgate.p);
-            const float* sg = lw.shared_gate ? (const float*)y.sgate.p : (const float*)nullptr;    // nullptr: the shared expert counts fully
-            const float* sh = nullptr;
-            if (d.shared_ff > 0) {          // the always-on expert first: its split-K scratch is free again before the routed experts run
-                const int Fs = d.shared_ff;
-                const Slices gu = gemm_slices(c, lc, "gemm_shared_in", sub_in, hhi, hlo, lw.s_gu, lw.tm_sgu, lw.tc_sgu, 2 * Fs, W, y.sh_gu.p, Ti);
-                launch_glu(lc, gu, Ti, Fs, d.shared_limit, 0, nullptr, lw.tc_sdown ? (float*)nullptr : y.sh_act.p, lw.tc_sdown ? ahi : (uint16_t*)nullptr, alo);
-                gemm_tc_or_exact(c, lc, "gemm_shared_out", y.sh_act.p, ahi, alo, lw.s_down, lw.tm_sdown, lw.tc_sdown, W, Fs, y.sh_o.p, Ti);
-                sh = y.sh_o.p;
-            }
-            const dim3 gw((W + 255) / 256, Ti);
-            if (lw.tc_moe && Ti > 128) {
-                // many rows: every expert over all rows on the tensor cores, kept where the row picked it (ascending expert order)
-                for (int e = 0; e < E; ++e) {
-                    dense_gemm(c, lc, "gemm_tc_moe_in", Ti, GF, W, lw.tm_egu[e], y.gu.p, hhi, hlo);
-                    launch_glu(lc, Slices{y.gu.p, 1, 0}, Ti, F, d.limit, act, nullptr, nullptr, ahi, alo);
-                    dense_gemm(c, lc, "gemm_tc_moe_out", Ti, W, F, lw.tm_edown[e], y.eo.p, ahi, alo);
-                    launch(lc, "moe_accum", 0, ly_moe_accum_kernel, gw, dim3(256), 0, (const float*)y.eo.p, (const int*)y.route_sel.p,
-                           (const float*)y.route_w.p, top, e, (const float*)nullptr, e == 0 ? 1 : 0, W, y.y.p);
-                }
-                if (sh != nullptr)
-                    launch(lc, "moe_accum", 0, ly_moe_accum_kernel, gw, dim3(256), 0, sh, (const int*)nullptr, (const float*)nullptr, 0, -1,
-                           sg, 0, W, y.y.p);
-            } else {
-                launch(lc, "moe_lists", 0, ly_moe_lists_kernel, dim3(E), dim3(32), 0, (const int*)y.route_sel.p, Ti, top, E, y.grp_off.p, y.pair_row.p,
-                       y.pair_of.p);
-                if (lw.tc_moe) {
-                    // few rows: ONE grouped GEMM pair over (expert, weight tile, k slice) items; an expert without rows costs nothing
-                    const int cap = Ti <= 16 ? 16 : (Ti <= 32 ? 32 : (Ti <= 64 ? 64 : 128));
-                    launch(lc, "moe_gather", 0, ly_moe_gather_kernel, dim3(E, std::min(Ti, 16)), dim3(256), 0, (const uint16_t*)hhi, (const uint16_t*)hlo, W,
-                           (const int*)y.grp_off.p, (const int*)y.pair_row.p, cap, y.gx_hi.p, y.gx_lo.p, y.grp_cnt.p);
-                    int ks = dense_gemm_grouped(c, lc, "gemm_tc_moe_in", E, cap, GF, W, lw.tm_gu, y.gemm_out.p, y.gx_hi.p, y.gx_lo.p, y.grp_cnt.p);
-                    FL_CHECK((size_t)ks * E * cap * GF <= y.gemm_out.n, FL_ERR_STATE, "internal: grouped GEMM scratch too small");
-                    launch(lc, "glu_grouped", 0, ly_glu_grouped_kernel, dim3((F + 255) / 256, E * cap), dim3(256), 0, (const float*)y.gemm_out.p, ks,
-                           (size_t)E * cap * GF, F, d.limit, act, (const int*)y.grp_cnt.p, cap, y.ga_hi.p, y.ga_lo.p);
-                    ks = dense_gemm_grouped(c, lc, "gemm_tc_moe_out", E, cap, W, F, lw.tm_down, y.gemm_out.p, y.ga_hi.p, y.ga_lo.p, y.grp_cnt.p);
-                    FL_CHECK((size_t)ks * E * cap * W <= y.gemm_out.n, FL_ERR_STATE, "internal: grouped GEMM scratch too small");
-                    launch(lc, "moe_combine", 0, ly_moe_combine_grouped_kernel, gw, dim3(256), 0, (const float*)y.gemm_out.p, ks, (size_t)E * cap * W,
-                           (const int*)y.route_sel.p, (const int*)y.pair_of.p, (const int*)y.grp_off.p, cap, (const float*)y.route_w.p, top, sh,
-                           sg, W, y.y.p);
-                } else {
-                    LyGemm g1{sub_in, 0, W, y.pair_row.p, lw.w_gu, (long long)GF * W, GF, W, y.gu.p, 0, GF, y.grp_off.p, P};
-                    gemm_groups(lc, "gemm_moe_in", g1, E, P);
-                    launch_glu(lc, Slices{y.gu.p, 1, 0}, P, F, d.limit, act, nullptr, y.act.p, nullptr, nullptr);
-                    LyGemm g2{y.act.p, 0, F, nullptr, lw.w_down, (long long)W * F, W, F, y.eo.p, 0, W, y.grp_off.p, P};
-                    gemm_groups(lc, "gemm_moe_out", g2, E, P);
-                    launch(lc, "moe_combine", 0, ly_moe_combine_kernel, gw, dim3(256), 0, (const float*)y.eo.p, (const int*)y.pair_of.p,
-                           (const float*)y.route_w.p, top, sh, sg, W, y.y.p);
-                }
-            }
+            experts(lw, y.y.p);
         }
         if (sum_norm)
             sum_norm_join(lw.b_down, nullptr, 1.f, 0.f, lw.norm2b, shifted ? 0 : more);
         else if (post)
-            post_norm(ff, lw.b_down, lw.norm2b, next1, lw.ls2, again, pstep, more, mix_halves ? nullptr : y.h.p);
+            post_norm(ff, lw.b_down, lw.norm2b, plain, next1, lw.ls2, again, pstep, more, h_next);
         else
-            join(nullptr, nullptr, nullptr, lw.rg2b, depth ? li + 1 : -1, lw.dwa, next1);
+            last_join(ff, nullptr, nullptr, nullptr, lw.rg2b);
     }
     if (n_want > 0) {
-        launch(lc, "final_norm", 0, ly_final_norm_kernel, dim3(n_want), dim3(nthr), 0, (const float*)y.x.p, st.want, (const float*)m.final_norm, eps, W, plain, y.hf.p,
+        launch(lc, "final_norm", 0, ly_final_norm_kernel, dim3(n_want), dim3(nthr), 0, (const float*)y.x.p, st.want, norm_of(m.final_norm, m.final_bias, m.final_alpha),
+               eps, W, m.cfg.logit_scale != 0.f ? m.cfg.logit_scale : 1.f, y.hf.p,
                m.tc_head ? y.hf_hi.p : (uint16_t*)nullptr, y.hf_lo.p);
         gemm_tc_or_exact(c, lc, "gemm_head", y.hf.p, m.tc_head ? y.hf_hi.p : nullptr, y.hf_lo.p, m.head, m.tm_head, m.tc_head, m.V, W, y.logits.p, n_want);
         if (m.cfg.logit_softcap > 0.f) {

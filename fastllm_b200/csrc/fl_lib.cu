@@ -1169,8 +1169,8 @@ int dense_gemm(fl_cache& c, LaunchCtx& lc, const char* tag, int R, int N, int K,
 // Block-diagonal GEMM with hi | lo output (see GemmArgs.blocks): tokens are the M dimension above 128 rows, else the weights are
 // (swap-AB, never split over K: the halves are those of the finished sum).
 void dense_gemm_blocks(fl_cache& c, LaunchCtx& lc, const char* tag, int R, int blocks, int N, int K, const CUtensorMap& tmW, const uint16_t* xhi,
-                       const uint16_t* xlo, uint16_t* ohi, uint16_t* olo, int ldo, int o_bs, const float* gate, int ldg) {
-    FL_CHECK(K % 8 == 0 && N % 8 == 0 && ldo % 8 == 0 && o_bs % 8 == 0 && ldg % 4 == 0, FL_ERR_STATE, "internal: block-diagonal GEMM alignment");
+                       const uint16_t* xlo, uint16_t* ohi, uint16_t* olo, int ldo, int o_bs, const float* gate, int ldg, bool gate_blk) {
+    FL_CHECK(K % 8 == 0 && N % 8 == 0 && ldo % 8 == 0 && o_bs % 8 == 0 && (gate_blk || ldg % 4 == 0), FL_ERR_STATE, "internal: block-diagonal GEMM alignment");
     const bool prof = g_prof.on && !lc.capturing;
     const bool pdl = lc.pdl && !prof;
     ProfEntry pe;
@@ -1183,7 +1183,7 @@ void dense_gemm_blocks(fl_cache& c, LaunchCtx& lc, const char* tag, int R, int b
     }
     const bool swap = R <= 128;
     GemmArgs g{swap ? N : R, swap ? R : N, K, nullptr, nullptr, 0, ohi, ldo, 1, 0, olo};
-    g.blocks = blocks; g.o_bs = o_bs; g.gate = gate; g.ldg = ldg;
+    g.blocks = blocks; g.o_bs = o_bs; g.gate = gate; g.ldg = ldg; g.gate_blk = gate != nullptr && gate_blk ? 1 : 0;
     const uint64_t KX = (uint64_t)blocks * K;
     if (swap) {
         const int bn = R <= 16 ? 16 : (R <= 32 ? 32 : (R <= 64 ? 64 : 128)), tiles = blocks * ((N + 127) / 128);

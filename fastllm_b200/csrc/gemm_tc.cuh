@@ -49,11 +49,12 @@ struct GemmArgs {
     // [b K, (b + 1) K) of the activations [tokens, blocks K]; the weight rows per block (N with DUAL_A, M with DUAL_B) and K are per
     // block.  Where a block's K ends inside a k-block the weights are zero-filled (their map is K wide), so the neighbour's
     // activations there count nothing.  Token t, block b, weight row n of the result goes to out[t * ldo + b * o_bs + n] as bf16 hi and
-    // out2 as lo, times sigmoid(gate[t * ldg + b * rows + n]) when there is a gate.
+    // out2 as lo, times sigmoid(gate[t * ldg + b * rows + n]) when there is a gate, or sigmoid(gate[t * ldg + b]) with gate_blk.
     int blocks = 0;
     int o_bs = 0;
     const float* gate = nullptr;
     int ldg = 0;
+    int gate_blk = 0;
 };
 
 // ---- PTX wrappers ------------------------------------------------------------------------------------------------------
@@ -527,7 +528,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
                     } else if (EPI == GEPI_HL) {
                         const size_t o = (size_t)row * g.ldo + (size_t)grp * g.o_bs + col;
                         uint16_t *oh = reinterpret_cast<uint16_t*>(g.out) + o, *ol = reinterpret_cast<uint16_t*>(g.out2) + o;
-                        const float* gt = g.gate != nullptr ? g.gate + (size_t)row * g.ldg + (size_t)grp * g.N + col : nullptr;
+                        const float* gt = g.gate != nullptr ? g.gate + (size_t)row * g.ldg + (g.gate_blk ? (size_t)grp : (size_t)grp * g.N + col) : nullptr;
+                        const float gs = gt != nullptr && g.gate_blk ? 1.f / (1.f + expf(-gt[0])) : 1.f;
                         const bool wide = ((g.ldo | g.o_bs | g.N) & 15) == 0 && ((reinterpret_cast<uintptr_t>(g.out) | reinterpret_cast<uintptr_t>(g.out2)) & 31) == 0;
 #pragma unroll
                         for (int j = 0; j < 32; j += 16) {
@@ -539,7 +541,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
                                     float v[8];
 #pragma unroll
                                     for (int e = 0; e < 8; ++e) v[e] = __uint_as_float(r[j + 8 * q8 + e]);
-                                    if (gt != nullptr && (q8 == 0 || second)) {
+                                    if (g.gate_blk) {
+#pragma unroll
+                                        for (int e = 0; e < 8; ++e) v[e] *= gs;
+                                    } else if (gt != nullptr && (q8 == 0 || second)) {
                                         const float4 z0 = *reinterpret_cast<const float4*>(gt + j + 8 * q8), z1 = *reinterpret_cast<const float4*>(gt + j + 8 * q8 + 4);
                                         const float z[8] = {z0.x, z0.y, z0.z, z0.w, z1.x, z1.y, z1.z, z1.w};
 #pragma unroll
@@ -569,7 +574,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
                         // for a fixed token the 32 lanes of the warp write 32 consecutive halves
                         const size_t o = (size_t)grp * g.o_bs + row;
                         uint16_t *oh = reinterpret_cast<uint16_t*>(g.out) + o, *ol = reinterpret_cast<uint16_t*>(g.out2) + o;
-                        const float* gt = g.gate != nullptr ? g.gate + (size_t)grp * g.M + row : nullptr;
+                        const float* gt = g.gate != nullptr ? g.gate + (g.gate_blk ? (size_t)grp : (size_t)grp * g.M + row) : nullptr;
 #pragma unroll
                         for (int j = 0; j < 32; ++j)
                             if (col + j < g.N) {

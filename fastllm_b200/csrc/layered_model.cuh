@@ -1,8 +1,9 @@
-// Layered decoders (FL_ARCH_NIFUNEX, FL_ARCH_ROFETAR, FL_ARCH_TOZARAX, FL_ARCH_MEDULORN, FL_ARCH_LATODRA): model / cache objects shared by
+// Layered decoders (FL_ARCH_NIFUNEX, FL_ARCH_ROFETAR, FL_ARCH_TOZARAX, FL_ARCH_MEDULORN, FL_ARCH_LATODRA, FL_ARCH_TUFAZEN): model / cache objects shared by
 // fl_layered.cu and fl_lib.cu.  A layer = one mixer (gated linear attention | latent attention | grouped-query attention | Mamba-2 | gated delta rule |
 // lightning attention), or two of them side by side, + an optional feed-forward (dense | MoE), each wrapped by a norm before and
 // after, after only (fl_stack_config.no_pre_norm), before only (no_post_norm), or a norm of the sum of stream and sublayer result
-// (post_sum_norm); optionally a learned position table, an input convolution in front of every sublayer, a token shift in front of
+// (post_sum_norm), or both reading one norm and joining together (parallel_sub); optionally hashed bigram rows in the embedding, a vector
+// per layer and token id behind every layer, a learned position table, an input convolution in front of every sublayer, a token shift in front of
 // every mixer, a gate on every sublayer's contribution, an average over all earlier layers' outputs, a scale per channel on every
 // sublayer's normed result, and a span of layers that runs several times with the same weights.  Sizes and constants come from fl_layer_desc / fl_stack_config; nothing is fixed per model.
 #pragma once
@@ -23,12 +24,16 @@ namespace fl {
 struct LayeredLayerW {
     fl_layer_desc d{};
     float *norm1 = nullptr, *norm1b = nullptr, *norm2 = nullptr, *norm2b = nullptr;     // [W] f32
+    float *norm1_bias = nullptr, *norm1_alpha = nullptr, *norm2_bias = nullptr, *norm2_alpha = nullptr;     // tanh norms: [W], [1]
     // mixer input projections stacked into ONE matrix [n_in, W] (one GEMM per layer):
     //   GLA:     q | k | v | g | a1        latent attention:  q (or dq, with a query latent) | dkv (not when kv_from >= 0) | g (with a gate)
-    //   attention:  q | k | v  (no k, v rows when kv_from >= 0)      Mamba-2:  z | x | B | C | dt      delta rule:  q | k | v | g | b | a
+    //   attention:  q | k | v | g  (no k, v rows when kv_from >= 0, no v rows with v_from_k, g with a gate)      Mamba-2:  z | x | B | C | dt      delta rule:  q | k | v | g | b | a
     // (rows padded with zeros to a multiple of 8 for the three newer mixers, so that the tensor-core GEMM's tiles fit)
+    // Sublayers that run in parallel: the always-on feed-forward (the dense one, or the shared expert) reads the same input and joins the
+    // same sum, so its gate | up rows follow at off_ff and its down matrix is the last fx columns of w_o: u = [heads | activation].
     uint16_t* w_in = nullptr;
     int n_in = 0;
+    int off_ff = -1, fx = 0, u_ld = 0;  // u_ld: columns of w_o = row stride of u (heads * vdim + fx)
     int off_q = 0, off_k = 0, off_v = 0, off_g = 0, off_a = 0, off_dkv = 0;             // row (= output column) offsets inside w_in
     int off_b = 0, off_dt = 0;          // delta rule: write strengths; Mamba-2: step sizes
     int conv_off = 0, conv_ch = 0;      // recurrent mixers with a short convolution: the convolved columns of w_in's output
@@ -41,7 +46,7 @@ struct LayeredLayerW {
     float* shift = nullptr;                                                             // token shift: [W]
     float* router_b = nullptr;                                                          // biased router: [experts]
     float *b_gu = nullptr, *b_down = nullptr;                                           // biased dense feed-forward: [2 ff], [W]
-    uint16_t* w_o = nullptr;            // [W, heads * vdim]
+    uint16_t* w_o = nullptr;            // [W, u_ld]
     // GLA
     uint16_t* a2 = nullptr;             // [heads*dim, rank]
     float *a2b = nullptr, *hnorm = nullptr;                                              // [heads*dim], [vdim]
@@ -80,6 +85,10 @@ struct LayeredLayerW {
     float *ls1 = nullptr, *ls2 = nullptr;              // [W] scales of the two sublayers' normed results
     CUtensorMap tm_rg1{}, tm_rg2{};
     bool tc_rg1 = false, tc_rg2 = false;
+    uint16_t *side_gate = nullptr, *side_proj = nullptr;        // token vectors: [token_side, W], [W, token_side]
+    float* side_norm = nullptr;                                 // [W]
+    CUtensorMap tm_tgate{}, tm_tproj{};
+    bool tc_tgate = false, tc_tproj = false;
 };
 
 struct RopeSpec {                       // one distinct rotary configuration (tables are built per cache: they depend on max_seq)
@@ -112,7 +121,8 @@ struct LayeredModel {
     DevBuf<uint8_t> slab;
     float *embed_norm = nullptr, *loop_step = nullptr;             // [W]; [loop_times, W]
     uint16_t *embed = nullptr, *head = nullptr, *pos = nullptr;    // head: the same table as embed when tied; pos: [max_positions, W] learned position vectors (or nullptr)
-    float* final_norm = nullptr;
+    uint16_t *bigram = nullptr, *side_embed = nullptr;             // [buckets + 1, W]; [V, L * token_side]
+    float *final_norm = nullptr, *final_bias = nullptr, *final_alpha = nullptr;
     CUtensorMap tm_head{};
     bool tc_head = false;
     std::set<std::string> have;
@@ -121,7 +131,7 @@ struct LayeredModel {
     bool finalized = false;
     uint64_t weight_bytes = 0;
     // widest sizes over the layers (workspace planning)
-    int max_in = 0, max_hv = 0, max_hd = 0, max_hc = 0, max_ff = 0, max_top = 0, max_experts = 0, max_cv = 0, max_heads = 0, max_av = 0, max_qr = 0, max_q = 0, max_hp = 0, max_hq = 0, max_c = 0;    // max_av: widest value head of a grouped-query attention layer; max_qr / max_q: widest query latent / queries
+    int max_in = 0, max_hv = 0, max_hd = 0, max_hc = 0, max_ff = 0, max_top = 0, max_experts = 0, max_cv = 0, max_heads = 0, max_av = 0, max_qr = 0, max_q = 0, max_hp = 0, max_hq = 0, max_c = 0, max_u = 0;    // max_u: widest u row; max_av: widest value head of a grouped-query attention layer; max_qr / max_q: widest query latent / queries
                                         // expanded from one; tensor-core latent attention: max_hp / max_hq widest plain query parts / query operand, max_c latent
     std::mutex mu;
 };
@@ -135,6 +145,7 @@ struct LayeredCache {
     std::vector<DevBuf<float>> gla_state;          // per recurrent layer: [slots][heads][dim | state][vdim]
     std::vector<DevBuf<float>> conv_state;         // per recurrent layer: [slots][taps - 1][conv_ch] (empty without a convolution)
     std::vector<DevBuf<float>> canon_state;        // input convolutions: per layer run [2 sublayers][slots][taps - 1][W]
+    std::vector<int> slot_last;         // the slot's last token (bigram embedding; -1: none yet)
     std::vector<DevBuf<float>> shift_state;        // token shift: per layer run [slots][W], the mixer input of the slot's last position
     std::vector<DevBuf<float>> rope_cos, rope_sin; // per RopeSpec: [max_seq][dims/2]
     DevBuf<int> page_table;             // [slots][pages_per_slot]
@@ -147,6 +158,8 @@ struct LayeredCache {
     DevBuf<float> hc, gz, y2, xs;       // convolved sublayer input; gate pre-activations; the second mixer's projected output;
                                         // xs [L + 1][rows][W]: the embedding output and every layer's own result (depth average); a
                                         // loop that adds the embedding output again keeps just that, [rows][W]
+    DevBuf<float> tz, ta;               // token vectors: [rows, token_side] before / behind the activation
+    DevBuf<uint16_t> ta_hi, ta_lo;
     DevBuf<float> cq, qx;               // query latents [rows, max_qr], the queries expanded from them [rows, max_q]
     DevBuf<float> cv, rs;               // recurrent mixers: convolved + activated columns [rows, max_cv]; per-head (decay, strength) [rows, 2 heads]
     DevBuf<int> route_sel, pair_row, pair_of, grp_off;

@@ -6,7 +6,8 @@
 // routers (softmax top-k; sigmoid scores with a choice correction and group-limited choice) / row lists / combine, and the pieces of
 // stacks whose sublayer results join the stream un-normed (learned positions, input convolution, gated contribution, two mixers
 // side by side, depth average).  Every mechanism takes its sizes and constants as
-// arguments.  Residual stream, norms, softmax, routers, decays and the recurrent state are f32 throughout; a row's result never
+// arguments.  Stacks whose mixer and feed-forward read one normed input and join together, element-wise tanh norms, hashed bigram rows and
+// a per-layer vector looked up by token id have their pieces here too.  Residual stream, norms, softmax, routers, decays and the recurrent state are f32 throughout; a row's result never
 // depends on which other rows share the launch (fixed summation order per output element).
 #pragma once
 #include <math.h>
@@ -25,6 +26,7 @@ struct StepTab {
     const int* seq_slot;    // [n] cache slot
     const int* seq_pos0;    // [n] tokens the slot held before this step
     const int* want;        // [n_want] rows whose logits are asked for
+    const int* prev;        // [T] token id before every row's (-1: the row is its sequence's first)
     int T, n, n_want;
 };
 
@@ -140,16 +142,39 @@ static __global__ void ly_sum_slices_kernel(const float* __restrict__ y, int nsl
 // A norm weight w scales by (1 + w), or by w itself when `plain`.
 __device__ __forceinline__ float norm_scale(const float* __restrict__ w, int c, int plain) { return plain ? w[c] : 1.f + w[c]; }
 
-// x[row] = embed[tok[row]] (times escale when that is not 0) (+ pos_tab[row_pos[row]], a learned position vector);  h[row] = x / sqrt(mean x^2 + eps) * scale(w).
-// nw == nullptr (the first sublayer reads the stream itself): h is not written and the hi | lo halves are those of x.
+// A norm in front of a sublayer: the RMS norm above, or (alpha != nullptr) channel by channel tanh(alpha x) * w + b, which needs no sum
+// over the row.  w == nullptr: none.
+struct NormW {
+    const float *w, *b, *alpha;     // [W], [W], [1]
+    int plain;
+};
+// Rows of a table of token pairs: row (prev * mul_prev + tok * mul_cur) mod buckets, row `buckets` for a sequence's first token
+struct BigramTab {
+    const uint16_t* tab;            // [buckets + 1, W] or nullptr
+    const int* prev;                // [T] previous token or -1
+    int buckets;
+    long long mul_prev, mul_cur;
+};
+
+// x[row] = embed[tok[row]] (times escale when that is not 0) (+ pos_tab[row_pos[row]], a learned position vector) (+ the bigram row);
+// h[row] = norm(x).
+// nw.w == nullptr (the first sublayer reads the stream itself): h is not written and the hi | lo halves are those of x.  h may be nullptr
+// (only the halves are read).
 // en (optional): the embedding row is RMS-normed first, scale(en).  x0 (optional): a second copy of x, the first entry of the depth
 // average's history or what a loop adds again; step (optional): a vector added to x behind that copy (a loop that starts with layer 0).
-static __global__ void ly_embed_norm_kernel(const uint16_t* __restrict__ embed, const int* __restrict__ tok, int W, const float* __restrict__ nw,
-                                            float eps, int plain, const uint16_t* __restrict__ pos_tab, const int* __restrict__ row_pos,
-                                            float escale, const float* __restrict__ en, const float* __restrict__ step, float* __restrict__ x,
+static __global__ void ly_embed_norm_kernel(const uint16_t* __restrict__ embed, const int* __restrict__ tok, int W, NormW nw, float eps, int plain,
+                                            const uint16_t* __restrict__ pos_tab, const int* __restrict__ row_pos, float escale,
+                                            const float* __restrict__ en, BigramTab bg, const float* __restrict__ step, float* __restrict__ x,
                                             float* __restrict__ x0, float* __restrict__ h, uint16_t* __restrict__ hhi, uint16_t* __restrict__ hlo) {
     __shared__ float red[33];
     const int row = blockIdx.x;
+    const uint16_t* be = nullptr;
+    if (bg.tab != nullptr) {
+        const int prev = bg.prev[row];
+        const long long r = prev < 0 ? bg.buckets : (prev * bg.mul_prev + tok[row] * bg.mul_cur) % bg.buckets;
+        be = bg.tab + (size_t)r * W;
+    }
+    const float alpha = nw.alpha != nullptr ? *nw.alpha : 0.f;
     const uint16_t* e = embed + (size_t)tok[row] * W;
     const uint16_t* pe = pos_tab ? pos_tab + (size_t)row_pos[row] * W : nullptr;
     float* xr = x + (size_t)row * W;
@@ -164,23 +189,38 @@ static __global__ void ly_embed_norm_kernel(const uint16_t* __restrict__ embed, 
         if (en != nullptr) v *= er * norm_scale(en, c, plain);
         if (escale != 0.f) v *= escale;
         if (pe) v += __uint_as_float((uint32_t)pe[c] << 16);
+        if (be) v += __uint_as_float((uint32_t)be[c] << 16);
         if (x0) x0[(size_t)row * W + c] = v;
         if (step) v += step[c];
         xr[c] = v;
         ss += v * v;
-        if (nw == nullptr) split_store(hhi, hlo, (size_t)row * W + c, v);
+        if (nw.w == nullptr) split_store(hhi, hlo, (size_t)row * W + c, v);
+        if (nw.alpha != nullptr) {
+            v = tanhf(alpha * v) * nw.w[c] + nw.b[c];
+            if (h) h[(size_t)row * W + c] = v;
+            split_store(hhi, hlo, (size_t)row * W + c, v);
+        }
     }
-    if (nw == nullptr) return;
+    if (nw.w == nullptr || nw.alpha != nullptr) return;
     const float r = 1.f / sqrtf(block_sum(ss, red) / (float)W + eps);
-    float* hr = h + (size_t)row * W;
     for (int c = threadIdx.x; c < W; c += blockDim.x) {
-        const float v = xr[c] * r * norm_scale(nw, c, plain);
-        hr[c] = v;
+        const float v = xr[c] * r * norm_scale(nw.w, c, nw.plain);
+        if (h) h[(size_t)row * W + c] = v;
         split_store(hhi, hlo, (size_t)row * W + c, v);
     }
 }
+// V channels of tanh(alpha v) * w + b at channel c of a row starting at rb, to h (optional) and its hi | lo halves
+template <int V>
+__device__ __forceinline__ void tanh_norm_store(const NormW& n, float alpha, float (&v)[V], int c, size_t rb, float* h, uint16_t* hhi, uint16_t* hlo) {
+    float w[V], b[V];
+    ld_vec<V>(n.w + c, w); ld_vec<V>(n.b + c, b);
+#pragma unroll
+    for (int i = 0; i < V; ++i) v[i] = tanhf(alpha * v[i]) * w[i] + b[i];
+    if (h != nullptr) st_vec<V>(h + rb + c, v);
+    split_store_vec<V>(hhi, hlo, rb + c, v);
+}
 
-// x[row] += norm(y[row] + yb; wb);  then, if wnext, h[row] = norm(x[row]; wnext); else, if split_x, the hi | lo halves of x[row]
+// x[row] += norm(y[row] + yb; wb);  then, if next.w, h[row] = norm(x[row]; next); else, if split_x, the hi | lo halves of x[row]
 // itself (the next sublayer reads the stream un-normed).  yb: optional bias of the projection that produced y.  ls (optional) [W] scales
 // the normed result per channel.  Between two passes of a loop the stream then gains x0[row] (optional: the embedding output once
 // more) and step (optional [W]: the next pass's vector), in this order, before the next norm.
@@ -188,7 +228,7 @@ static __global__ void ly_embed_norm_kernel(const uint16_t* __restrict__ embed, 
 // ([W] floats) between the passes (a thread reads back what it wrote itself).
 template <int V>
 static __global__ void __launch_bounds__(1024) ly_post_norm_kernel(float* __restrict__ x, Slices y, const float* __restrict__ yb, const float* __restrict__ wb,
-                                           const float* __restrict__ wnext, const float* __restrict__ ls, const float* __restrict__ x0, const float* __restrict__ step,
+                                           NormW next, const float* __restrict__ ls, const float* __restrict__ x0, const float* __restrict__ step,
                                            float eps, int W, int plain, int split_x, float* __restrict__ h, uint16_t* __restrict__ hhi, uint16_t* __restrict__ hlo) {
     extern __shared__ __align__(16) float srow[];
     __shared__ float red[33];
@@ -208,7 +248,7 @@ static __global__ void __launch_bounds__(1024) ly_post_norm_kernel(float* __rest
         for (int i = 0; i < V; ++i) ss += v[i] * v[i];
         st_vec<V>(srow + c, v);
     }
-    const float r = 1.f / sqrtf(block_sum(ss, red) / (float)W + eps);
+    const float r = 1.f / sqrtf(block_sum(ss, red) / (float)W + eps), alpha = next.alpha != nullptr ? *next.alpha : 0.f;
     float s2 = 0.f;
     auto add = [&](float (&v)[V], const float* p) {
         float t[V];
@@ -231,46 +271,50 @@ static __global__ void __launch_bounds__(1024) ly_post_norm_kernel(float* __rest
         if (x0 != nullptr) add(v, x0 + rb + c);
         if (step != nullptr) add(v, step + c);
         st_vec<V>(x + rb + c, v);
+        if (next.alpha != nullptr) { tanh_norm_store<V>(next, alpha, v, c, rb, h, hhi, hlo); continue; }
 #pragma unroll
         for (int i = 0; i < V; ++i) s2 += v[i] * v[i];
-        if (wnext != nullptr) st_vec<V>(srow + c, v);
+        if (next.w != nullptr) st_vec<V>(srow + c, v);
         else if (split_x) split_store_vec<V>(hhi, hlo, rb + c, v);
     }
-    if (wnext == nullptr) return;
+    if (next.w == nullptr || next.alpha != nullptr) return;
     const float r2 = 1.f / sqrtf(block_sum(s2, red) / (float)W + eps);
     for (int c = threadIdx.x * V; c < W; c += stride) {
         float v[V], w[V];
-        ld_vec<V>(srow + c, v); ld_vec<V>(wnext + c, w);
+        ld_vec<V>(srow + c, v); ld_vec<V>(next.w + c, w);
 #pragma unroll
-        for (int i = 0; i < V; ++i) v[i] = v[i] * r2 * (plain ? w[i] : 1.f + w[i]);
+        for (int i = 0; i < V; ++i) v[i] = v[i] * r2 * (next.plain ? w[i] : 1.f + w[i]);
         if (h != nullptr) st_vec<V>(h + rb + c, v);
         split_store_vec<V>(hhi, hlo, rb + c, v);
     }
 }
 
 // A sublayer's result joins the stream un-normed:  x[row] += gate * v,  where
-//   v = y[row], or with two mixers side by side (y2 != nullptr) v = (unit(y) * wa + unit(y2) * wb) / 2, unit(.) = . / sqrt(mean .^2 + eps);
+//   v = y[row] (perhaps still in split-K slices), or with two mixers side by side (wa != nullptr) v = (unit(y) * wa + unit(y2) * wb) / 2,
+//   unit(.) = . / sqrt(mean .^2 + eps), or (y2 without wa) v = y + y2;
 //   gate = sigmoid(gz[row] + gb) per channel (gz == nullptr: 1).
 // slot >= 0 (the layer's last sublayer, stacks with a depth average): hist[slot][row] = x[row], the layer's own result, and then
 //   x[row] = sum_{j <= slot} dw[j] * hist[j][row]  (hist[0] = the embedding output), in ascending j.
-// Then, if wnext, h[row] = norm(x[row]; wnext) with its hi | lo halves.
+// Between two passes of a loop the stream then gains x0[row] and step (both optional, see ly_post_norm_kernel).
+// Then, if next.w, h[row] (optional) = norm(x[row]; next) with its hi | lo halves; else, if split_x, the halves of x[row] itself.
 // One block per row; a thread takes V consecutive channels at a time (V = 4: 16-byte accesses, W a multiple of 4).
 template <int V>
-static __global__ void ly_join_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ y2, const float* __restrict__ wa,
+static __global__ void __launch_bounds__(1024) ly_join_kernel(float* __restrict__ x, Slices y, const float* __restrict__ y2, const float* __restrict__ wa,
                                       const float* __restrict__ wb, const float* __restrict__ gz, const float* __restrict__ gb,
                                       float* __restrict__ hist, size_t hist_stride, int slot, const float* __restrict__ dw,
-                                      const float* __restrict__ wnext, float eps, int W, int plain, float* __restrict__ h,
-                                      uint16_t* __restrict__ hhi, uint16_t* __restrict__ hlo) {
+                                      const float* __restrict__ x0, const float* __restrict__ pstep, NormW next, float eps, int W, int split_x,
+                                      float* __restrict__ h, uint16_t* __restrict__ hhi, uint16_t* __restrict__ hlo) {
     __shared__ float red[33];
     const int row = blockIdx.x;
     const size_t rb = (size_t)row * W;
     const int step = blockDim.x * V;
     float ra = 1.f, rb2 = 1.f;
-    if (y2 != nullptr) {
+    const float alpha = next.alpha != nullptr ? *next.alpha : 0.f;
+    if (wa != nullptr) {
         float sa = 0.f, sb = 0.f;
         for (int c = threadIdx.x * V; c < W; c += step) {
             float p[V], q[V];
-            ld_vec<V>(y + rb + c, p); ld_vec<V>(y2 + rb + c, q);
+            ld_slices<V>(y, rb + c, p); ld_vec<V>(y2 + rb + c, q);
 #pragma unroll
             for (int i = 0; i < V; ++i) { sa += p[i] * p[i]; sb += q[i] * q[i]; }
         }
@@ -280,8 +324,13 @@ static __global__ void ly_join_kernel(float* __restrict__ x, const float* __rest
     float s2 = 0.f;
     for (int c = threadIdx.x * V; c < W; c += step) {
         float v[V], t[V];
-        ld_vec<V>(y + rb + c, v);
-        if (y2 != nullptr) {
+        ld_slices<V>(y, rb + c, v);
+        if (y2 != nullptr && wa == nullptr) {
+            float q[V];
+            ld_vec<V>(y2 + rb + c, q);
+#pragma unroll
+            for (int i = 0; i < V; ++i) v[i] += q[i];
+        } else if (wa != nullptr) {
             float q[V], fa[V], fb[V];
             ld_vec<V>(y2 + rb + c, q); ld_vec<V>(wa + c, fa); ld_vec<V>(wb + c, fb);
 #pragma unroll
@@ -312,18 +361,30 @@ static __global__ void ly_join_kernel(float* __restrict__ x, const float* __rest
 #pragma unroll
             for (int i = 0; i < V; ++i) t[i] = fmaf(ds, t[i], acc[i]);
         }
+        if (x0 != nullptr) {
+            ld_vec<V>(x0 + rb + c, v);
+#pragma unroll
+            for (int i = 0; i < V; ++i) t[i] += v[i];
+        }
+        if (pstep != nullptr) {
+            ld_vec<V>(pstep + c, v);
+#pragma unroll
+            for (int i = 0; i < V; ++i) t[i] += v[i];
+        }
         st_vec<V>(x + rb + c, t);
+        if (next.alpha != nullptr) tanh_norm_store<V>(next, alpha, t, c, rb, h, hhi, hlo);
+        else if (next.w == nullptr && split_x) split_store_vec<V>(hhi, hlo, rb + c, t);
 #pragma unroll
         for (int i = 0; i < V; ++i) s2 += t[i] * t[i];
     }
-    if (wnext == nullptr) return;
+    if (next.w == nullptr || next.alpha != nullptr) return;
     const float r2 = 1.f / sqrtf(block_sum(s2, red) / (float)W + eps);
     for (int c = threadIdx.x * V; c < W; c += step) {
         float t[V], wn[V];
-        ld_vec<V>(x + rb + c, t); ld_vec<V>(wnext + c, wn);
+        ld_vec<V>(x + rb + c, t); ld_vec<V>(next.w + c, wn);
 #pragma unroll
-        for (int i = 0; i < V; ++i) t[i] = t[i] * r2 * (plain ? wn[i] : 1.f + wn[i]);
-        st_vec<V>(h + rb + c, t);
+        for (int i = 0; i < V; ++i) t[i] = t[i] * r2 * (next.plain ? wn[i] : 1.f + wn[i]);
+        if (h != nullptr) st_vec<V>(h + rb + c, t);
         split_store_vec<V>(hhi, hlo, rb + c, t);
     }
 }
@@ -379,17 +440,19 @@ static __global__ void ly_softcap_kernel(float* __restrict__ z, size_t n, float 
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) z[i] = cap * tanhf(z[i] * inv);
 }
 
-// hf[i] = norm(x[want[i]]; w): the rows that go on to the vocabulary projection
-static __global__ void ly_final_norm_kernel(const float* __restrict__ x, const int* __restrict__ want, const float* __restrict__ w, float eps, int W,
-                                            int plain, float* __restrict__ hf, uint16_t* __restrict__ hhi, uint16_t* __restrict__ hlo) {
+// hf[i] = norm(x[want[i]]; w) * scale: the rows that go on to the vocabulary projection (scale: what the logits are multiplied by)
+static __global__ void ly_final_norm_kernel(const float* __restrict__ x, const int* __restrict__ want, NormW nw, float eps, int W,
+                                            float scale, float* __restrict__ hf, uint16_t* __restrict__ hhi, uint16_t* __restrict__ hlo) {
     __shared__ float red[33];
     const float* xr = x + (size_t)want[blockIdx.x] * W;
     float ss = 0.f;
-    for (int c = threadIdx.x; c < W; c += blockDim.x) ss += xr[c] * xr[c];
-    const float r = 1.f / sqrtf(block_sum(ss, red) / (float)W + eps);
+    const bool tn = nw.alpha != nullptr;
+    if (!tn)
+        for (int c = threadIdx.x; c < W; c += blockDim.x) ss += xr[c] * xr[c];
+    const float r = tn ? *nw.alpha : 1.f / sqrtf(block_sum(ss, red) / (float)W + eps);
     float* hr = hf + (size_t)blockIdx.x * W;
     for (int c = threadIdx.x; c < W; c += blockDim.x) {
-        const float v = xr[c] * r * norm_scale(w, c, plain);
+        const float v = (tn ? tanhf(r * xr[c]) * nw.w[c] + nw.b[c] : xr[c] * r * norm_scale(nw.w, c, nw.plain)) * scale;
         hr[c] = v;
         split_store(hhi, hlo, (size_t)blockIdx.x * W + c, v);
     }
@@ -562,7 +625,7 @@ static __global__ void __launch_bounds__(kGlaVS * kGlaDG) ly_gla_scan_kernel(Gla
 
 // u[row, h, :] = o[row, h, :] / sqrt(mean o^2 + eps) * w[:] * silu(g[row, h, :])     (one warp per (row, head))
 static __global__ void ly_gla_out_kernel(const float* __restrict__ o, const float* __restrict__ proj, int ldp, int off_g, const float* __restrict__ w,
-                                         float eps, int T, int H, int Dv, float* __restrict__ u, uint16_t* __restrict__ uhi, uint16_t* __restrict__ ulo) {
+                                         float eps, int T, int H, int Dv, int ldo, float* __restrict__ u, uint16_t* __restrict__ uhi, uint16_t* __restrict__ ulo) {
     const int item = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (item >= T * H) return;
     const int row = item / H, hd = item % H;
@@ -571,12 +634,13 @@ static __global__ void ly_gla_out_kernel(const float* __restrict__ o, const floa
     for (int c = lane; c < Dv; c += 32) ss += op[c] * op[c];
     const float r = 1.f / sqrtf(warp_sum(ss) / (float)Dv + eps);
     const float* gp = proj + (size_t)row * ldp + off_g + hd * Dv;
-    float* up = u + (size_t)row * H * Dv + hd * Dv;
+    const size_t ub = (size_t)row * ldo + hd * Dv;
+    float* up = u + ub;
     for (int c = lane; c < Dv; c += 32) {
         const float g = gp[c];
         const float v = op[c] * r * w[c] * (g * sigmoidf_(g));
         up[c] = v;
-        split_store(uhi, ulo, (size_t)row * H * Dv + hd * Dv + c, v);
+        split_store(uhi, ulo, ub + c, v);
     }
 }
 
@@ -1221,15 +1285,25 @@ static __global__ void ly_attn_softmax_kernel(const float* __restrict__ S, const
     }
 }
 
-// u[row, c] *= sigmoid(proj[row, off_g + c]): a gate on the concatenated heads, with the hi | lo halves of the product
-static __global__ void ly_out_gate_kernel(float* __restrict__ u, const float* __restrict__ proj, int ldp, int off_g, int n, int T,
-                                          uint16_t* __restrict__ uhi, uint16_t* __restrict__ ulo) {
+// A sigmoid gate on an attention's output: channel c of head hd of a row is multiplied by sigmoid(g[row * ld + hd * hs + c * cs]) --
+// (hs, cs) = (Dv, 1): one gate per channel of the concatenated heads; (1, 0): one per head.  g == nullptr: none.
+struct OutGate {
+    const float* g;
+    int ld, hs, cs;
+    __device__ __forceinline__ float at(int row, int hd, int c) const { return sigmoidf_(g[(size_t)row * ld + hd * hs + c * cs]); }
+};
+// u[row, hd * Dv + c] *= gate (rows of u are ldo apart), with the hi | lo halves of the product
+static __global__ void ly_out_gate_kernel(float* __restrict__ u, int ldo, OutGate gate, int H, int Dv, int T, uint16_t* __restrict__ uhi,
+                                          uint16_t* __restrict__ ulo) {
+    const int n = H * Dv;
     const size_t total = (size_t)T * n;
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
         const size_t row = i / n;
-        const float v = u[i] * sigmoidf_(proj[row * ldp + off_g + (i - row * n)]);
-        u[i] = v;
-        split_store(uhi, ulo, i, v);
+        const int j = (int)(i - row * n), hd = j / Dv;
+        const size_t o = row * ldo + j;
+        float v = u[o];
+        if (gate.g != nullptr) u[o] = v = v * gate.at((int)row, hd, j - hd * Dv);
+        split_store(uhi, ulo, o, v);
     }
 }
 
@@ -1281,7 +1355,13 @@ static __global__ void __launch_bounds__(256) ly_attn_softmax_warp_kernel(const 
 }
 
 // ---- grouped-query attention over a paged key | value cache ---------------------------------------------------------------------
-// Cache row of a token: [kv_heads][dim] keys (normed, rotated) then [kv_heads][vdim] values.
+// Where a cache row of a token (E elements) keeps its heads: head g's key at g * ks, its value at vo + g * vs.  Keys and values apart: ks = D,
+// vo = G * D, vs = Dv.  Values that are the keys as projected, before their first rdims channels turn: [turned part | channels
+// rdims .. D | channels 0 .. rdims] per head (ks = vs = D + rdims, vo = rdims) -- the channels that do not turn are stored once, the key is
+// the first D elements and the value the last D, starting at channel `roll` = rdims: element i is channel (i + roll) mod Dv.
+struct KvLayout {
+    int E, ks, vo, vs, roll;
+};
 struct AttnPrepArgs {
     float* proj; int ldp, off_q, off_k, off_v;  // off_k < 0: the layer reads another layer's cache (queries are still prepared)
     const float *qnorm, *knorm; float eps;       // [dim] each ([H * dim], [G * dim] when `whole`)
@@ -1291,6 +1371,9 @@ struct AttnPrepArgs {
     int H, G, D, Dv, rdims, halves;
     const float *bq, *bk, *bv;                   // projection biases [H * dim], [G * dim], [G * vdim] (nullptr: none)
     int whole;                                   // 1: q (and k) are normed over all heads' channels at once
+    KvLayout kv;                                 // off_v < 0: the values are the keys (see there)
+    Slices in;                                   // what the columns are read from (proj itself, or the GEMM's slices)
+    int off_gate, n_gate;                        // gate columns to fold into proj when there are slices
 };
 // Per row: every query head and (when the layer owns its cache) every key head is RMS-normed over dim with a weight shared by the
 // heads (qnorm == nullptr: they are used as projected), then its first rdims channels are turned by the row's position: pairs (i, i + rdims/2) when `halves`, else (2i, 2i+1).
@@ -1303,16 +1386,18 @@ static __global__ void __launch_bounds__(256) ly_attn_prep_kernel(AttnPrepArgs a
     extern __shared__ float sm[];               // [warps][D]
     __shared__ float red[33];
     const int row = blockIdx.x, pos = a.row_pos[row], lane = threadIdx.x & 31, wid = threadIdx.x >> 5, nw = blockDim.x >> 5;
-    float* pr = a.proj + (size_t)row * a.ldp;
-    const bool own = a.off_k >= 0;
+    const size_t rb = (size_t)row * a.ldp;
+    float* pr = a.proj + rb;
+    auto in = [&](int c) { float v[1]; ld_slices<1>(a.in, rb + c, v); return v[0]; };
+    const bool own = a.off_k >= 0, shared_v = a.off_v < 0;
     float rq = 0.f, rk = 0.f;
     if (a.whole && a.qnorm != nullptr) {
         float ss = 0.f;
-        for (int c = threadIdx.x; c < a.H * a.D; c += blockDim.x) { const float v = pr[a.off_q + c] + (a.bq ? a.bq[c] : 0.f); ss += v * v; }
+        for (int c = threadIdx.x; c < a.H * a.D; c += blockDim.x) { const float v = in(a.off_q + c) + (a.bq ? a.bq[c] : 0.f); ss += v * v; }
         rq = 1.f / sqrtf(block_sum(ss, red) / (float)(a.H * a.D) + a.eps);
         if (own) {
             ss = 0.f;
-            for (int c = threadIdx.x; c < a.G * a.D; c += blockDim.x) { const float v = pr[a.off_k + c] + (a.bk ? a.bk[c] : 0.f); ss += v * v; }
+            for (int c = threadIdx.x; c < a.G * a.D; c += blockDim.x) { const float v = in(a.off_k + c) + (a.bk ? a.bk[c] : 0.f); ss += v * v; }
             rk = 1.f / sqrtf(block_sum(ss, red) / (float)(a.G * a.D) + a.eps);
         }
     }
@@ -1324,17 +1409,17 @@ static __global__ void __launch_bounds__(256) ly_attn_prep_kernel(AttnPrepArgs a
     if (own) {
         const int slot = a.seq_slot[a.row_seq[row]];
         const int page = a.page_table[(size_t)slot * a.pps + pos / kKvPage];
-        dst = (CT*)a.pool + ((size_t)page * kKvPage + pos % kKvPage) * ((size_t)a.G * (a.D + a.Dv));
+        dst = (CT*)a.pool + ((size_t)page * kKvPage + pos % kKvPage) * (size_t)a.kv.E;
     }
     const int items = a.H + (own ? a.G : 0);
     for (int it = blockIdx.y * nw + wid; it < items; it += gridDim.y * nw) {
         const bool isq = it < a.H;
         const int hd = isq ? it : it - a.H;
-        float* src = isq ? pr + a.off_q + hd * a.D : pr + a.off_k + hd * a.D;
+        const int src = (isq ? a.off_q : a.off_k) + hd * a.D;
         const float* bias = isq ? a.bq : a.bk;
         if (bias != nullptr) bias += (size_t)hd * a.D;
         const float* w = isq ? a.qnorm : a.knorm;
-        for (int c = lane; c < a.D; c += 32) buf[c] = src[c] + (bias ? bias[c] : 0.f);
+        for (int c = lane; c < a.D; c += 32) buf[c] = in(src + c) + (bias ? bias[c] : 0.f);
         __syncwarp();
         if (w != nullptr) {
             float r;
@@ -1359,22 +1444,27 @@ static __global__ void __launch_bounds__(256) ly_attn_prep_kernel(AttnPrepArgs a
                 const float u = buf[cu], v = buf[cv];
                 val = second ? v * cs[pi] + u * sn[pi] : u * cs[pi] - v * sn[pi];
             }
-            if (isq) src[c] = val; else st_c(dst + (size_t)hd * a.D + c, val);
+            if (isq) { pr[src + c] = val; continue; }
+            CT* kd = dst + (size_t)hd * a.kv.ks;
+            st_c(kd + c, val);
+            if (shared_v && c < a.rdims) st_c(kd + a.D + c, buf[c]);
         }
         __syncwarp();
     }
-    if (own && blockIdx.y == 0) {
-        const float* v = pr + a.off_v;
+    if (blockIdx.y != 0) return;
+    if (own && !shared_v) {
         CT* vd = dst + (size_t)a.G * a.D;
-        for (int c = threadIdx.x; c < a.G * a.Dv; c += blockDim.x) st_c(vd + c, v[c] + (a.bv ? a.bv[c] : 0.f));
+        for (int c = threadIdx.x; c < a.G * a.Dv; c += blockDim.x) st_c(vd + c, in(a.off_v + c) + (a.bv ? a.bv[c] : 0.f));
     }
+    if (a.in.n > 1)
+        for (int c = threadIdx.x; c < a.n_gate; c += blockDim.x) pr[a.off_gate + c] = in(a.off_gate + c);
 }
 
 struct GqaAttnArgs {
     const float* proj; int ldp, off_q;          // prepared queries at proj[row, off_q + h * D ...]
     const void* pool; const int* page_table; int pps;
     const int *row_seq, *row_pos, *seq_slot;
-    float* out;                 // [T, H * Dv]
+    float* out;                 // [T, ldo]: channel c of head h in column h * Dv + c
     uint16_t *ohi, *olo;        // its hi | lo halves (nullptr: not wanted)
     int H, G, D, Dv, window;
     float scale, softcap;       // softcap 0 = scores are used as they are
@@ -1383,6 +1473,9 @@ struct GqaAttnArgs {
     float* part;                // key splits (gridDim.z > 1): [T][H][splits][2 + Dv] partial (max, sum, weighted values)
     int keep_first, chunk;      // masks beside the window (see key_span)
     const float* sinkv;         // [H] or nullptr
+    KvLayout kv;
+    int ldo;
+    OutGate gate;
 };
 constexpr int kGqaWarps = 8;
 // One block per (row, RB query heads of one key/value head, key split).  score_j = cap(q . k_j * scale) over the keys the position
@@ -1398,7 +1491,7 @@ static __global__ void __launch_bounds__(kGqaWarps * 32) ly_gqa_attn_kernel(GqaA
     const int row = a.row_base + blockIdx.x, hd0 = blockIdx.y * RB, split = blockIdx.z, S = gridDim.z;
     const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
     const int D = a.D, Dv = a.Dv, g = hd0 / (a.H / a.G);
-    const size_t E = (size_t)a.G * (D + Dv);
+    const size_t E = a.kv.E;
     const int pos = a.row_pos[row], slot = a.seq_slot[a.row_seq[row]];
     const KeySpan ks = key_span(pos, a.window, a.keep_first, a.chunk);
     const int n_st = ks.s_hi - ks.s_lo, n_vis = n_st + pos - ks.j0 + 1;        // kept first keys, then the contiguous range
@@ -1424,8 +1517,8 @@ static __global__ void __launch_bounds__(kGqaWarps * 32) ly_gqa_attn_kernel(GqaA
             if (ji < n_vis) {
                 const CT* kp = (const CT*)a.pool + ((size_t)pt[jj / kKvPage] * kKvPage + jj % kKvPage) * E;
                 float kk[CPL];
-                load_chunk<CPL>(kp + (size_t)g * D, lane * CPL, D, kk);
-                load_chunk<CPL>(kp + (size_t)a.G * D + (size_t)g * Dv, lane * CPL, Dv, val[u]);
+                load_chunk<CPL>(kp + (size_t)g * a.kv.ks, lane * CPL, D, kk);
+                load_chunk<CPL>(kp + a.kv.vo + (size_t)g * a.kv.vs, lane * CPL, Dv, val[u]);
 #pragma unroll
                 for (int r = 0; r < RB; ++r)
 #pragma unroll
@@ -1477,12 +1570,14 @@ static __global__ void __launch_bounds__(kGqaWarps * 32) ly_gqa_attn_kernel(GqaA
         }
         if (S == 1) {
             const float inv = 1.f / Lsum;
-            const size_t ob = ((size_t)row * a.H + hd0 + r) * Dv;
-            for (int c = threadIdx.x; c < Dv; c += blockDim.x) {
+            const size_t ob = (size_t)row * a.ldo + (size_t)(hd0 + r) * Dv;
+            for (int i = threadIdx.x; i < Dv; i += blockDim.x) {
                 float t = 0.f;
 #pragma unroll
-                for (int w = 0; w < kGqaWarps; ++w) t += sacc[(w * RB + r) * Dv + c] * f[w];
+                for (int w = 0; w < kGqaWarps; ++w) t += sacc[(w * RB + r) * Dv + i] * f[w];
                 t *= inv;
+                const int c = i + a.kv.roll < Dv ? i + a.kv.roll : i + a.kv.roll - Dv;
+                if (a.gate.g != nullptr) t *= a.gate.at(row, hd0 + r, c);
                 a.out[ob + c] = t;
                 split_store(a.ohi, a.olo, ob + c, t);
             }
@@ -1499,9 +1594,9 @@ static __global__ void __launch_bounds__(kGqaWarps * 32) ly_gqa_attn_kernel(GqaA
     }
 }
 // Folds the key splits of ly_gqa_attn_kernel (or ly_latent_mma_kernel) in split order (and the sink): one block per (row, head).
-// out == nullptr: only the halves are wanted.
+// out == nullptr: only the halves are wanted.  roll: element i of a partial is channel (i + roll) mod Dv (see KvLayout).
 static __global__ void ly_gqa_merge_kernel(const float* __restrict__ part, int S, int H, int Dv, int sink, const float* __restrict__ sinkv, int row_base,
-                                           float* __restrict__ out, uint16_t* __restrict__ ohi, uint16_t* __restrict__ olo) {
+                                           int ldo, int roll, OutGate gate, float* __restrict__ out, uint16_t* __restrict__ ohi, uint16_t* __restrict__ olo) {
     const int row = row_base + blockIdx.x, hd = blockIdx.y;
     const float* pp = part + ((size_t)blockIdx.x * H + hd) * S * (Dv + 2);
     const float sv = sinkv ? sinkv[hd] : 0.f;
@@ -1513,14 +1608,16 @@ static __global__ void ly_gqa_merge_kernel(const float* __restrict__ part, int S
         L += ms == -INFINITY ? 0.f : pp[(size_t)s * (Dv + 2) + 1] * expf(ms - M);
     }
     const float inv = 1.f / L;
-    const size_t ob = ((size_t)row * H + hd) * Dv;
-    for (int c = threadIdx.x; c < Dv; c += blockDim.x) {
+    const size_t ob = (size_t)row * ldo + (size_t)hd * Dv;
+    for (int i = threadIdx.x; i < Dv; i += blockDim.x) {
         float t = 0.f;
         for (int s = 0; s < S; ++s) {
             const float ms = pp[(size_t)s * (Dv + 2)];
-            if (ms != -INFINITY) t += pp[(size_t)s * (Dv + 2) + 2 + c] * expf(ms - M);
+            if (ms != -INFINITY) t += pp[(size_t)s * (Dv + 2) + 2 + i] * expf(ms - M);
         }
         t *= inv;
+        const int c = i + roll < Dv ? i + roll : i + roll - Dv;
+        if (gate.g != nullptr) t *= gate.at(row, hd, c);
         if (out != nullptr) out[ob + c] = t;
         split_store(ohi, olo, ob + c, t);
     }
@@ -1532,7 +1629,7 @@ static __global__ void ly_gqa_merge_kernel(const float* __restrict__ part, int S
 // the group) pairs -- all of them meet the same keys --, S = Q . Kc^T, P = masked softmax(S) (cap, sink), O = P . V.
 // Rows r < n_first hold keys 0 .. n_first - 1 (kept first keys before k_lo), rows n_first + i key k_lo + i, i < nk.
 static __global__ void ly_gqa_gather_kv_kernel(const uint16_t* __restrict__ pool, const int* __restrict__ page_row, int k_lo, int n_first, int nk, int nkp,
-                                               int E, int koff, int D, int Dp, int voff, int Dv, uint16_t* __restrict__ kc, uint16_t* __restrict__ vt) {
+                                               int E, int koff, int D, int Dp, int voff, int Dv, int roll, uint16_t* __restrict__ kc, uint16_t* __restrict__ vt) {
     const int r = blockIdx.x;
     const uint16_t* src = nullptr;
     if (r < n_first + nk) {
@@ -1540,7 +1637,10 @@ static __global__ void ly_gqa_gather_kv_kernel(const uint16_t* __restrict__ pool
         src = pool + ((size_t)page_row[j / kKvPage] * kKvPage + j % kKvPage) * E;
     }
     for (int c = threadIdx.x; c < Dp; c += blockDim.x) kc[(size_t)r * Dp + c] = (src != nullptr && c < D) ? src[koff + c] : (uint16_t)0;
-    for (int c = threadIdx.x; c < Dv; c += blockDim.x) vt[(size_t)c * nkp + r] = src != nullptr ? src[voff + c] : (uint16_t)0;
+    for (int c = threadIdx.x; c < Dv; c += blockDim.x) {
+        const int ch = c + roll < Dv ? c + roll : c + roll - Dv;
+        vt[(size_t)ch * nkp + r] = src != nullptr ? src[voff + c] : (uint16_t)0;
+    }
 }
 // Q operand rows (token t, head hq of group g): the prepared query times `scale`, zero padded to Dp, as hi | lo halves.  grid (nq, rep)
 static __global__ void ly_gqa_build_q_kernel(const float* __restrict__ proj, int ldp, int off_q, int row0, int rep, int g, int D, int Dp, float scale,
@@ -1550,8 +1650,9 @@ static __global__ void ly_gqa_build_q_kernel(const float* __restrict__ proj, int
     const size_t base = ((size_t)t * rep + hq) * Dp;
     for (int c = threadIdx.x; c < Dp; c += blockDim.x) split_store(qhi, qlo, base + c, c < D ? qp[c] * scale : 0.f);
 }
-// o [G][nq * rep][Dv] (the value GEMMs' outputs, one slab per key/value head) -> u[row0 + t, (g rep + hq) Dv + c] and its hi | lo halves
-static __global__ void ly_gqa_scatter_kernel(const float* __restrict__ o, int nq, int G, int rep, int Dv, int row0, float* __restrict__ u,
+// o [G][nq * rep][Dv] (the value GEMMs' outputs, one slab per key/value head) -> u[row0 + t, (g rep + hq) Dv + c] (rows ldo
+// apart, times the gate) and its hi | lo halves
+static __global__ void ly_gqa_scatter_kernel(const float* __restrict__ o, int nq, int G, int rep, int Dv, int row0, int ldo, OutGate gate, float* __restrict__ u,
                                              uint16_t* __restrict__ uhi, uint16_t* __restrict__ ulo) {
     const size_t total = (size_t)nq * G * rep * Dv;
     const int H = G * rep;
@@ -1559,8 +1660,9 @@ static __global__ void ly_gqa_scatter_kernel(const float* __restrict__ o, int nq
         const int c = (int)(i % Dv);
         const int hd = (int)((i / Dv) % H), t = (int)(i / ((size_t)Dv * H));
         const int g = hd / rep, hq = hd % rep;
-        const float v = o[(((size_t)g * nq + t) * rep + hq) * Dv + c];
-        const size_t dst = ((size_t)(row0 + t) * H + hd) * Dv + c;
+        float v = o[(((size_t)g * nq + t) * rep + hq) * Dv + c];
+        if (gate.g != nullptr) v *= gate.at(row0 + t, hd, c);
+        const size_t dst = (size_t)(row0 + t) * ldo + (size_t)hd * Dv + c;
         u[dst] = v;
         split_store(uhi, ulo, dst, v);
     }
@@ -1861,13 +1963,14 @@ static __global__ void __launch_bounds__(128) ly_rec_scan_kernel(RecArgs a) {
 // sig_after: u[row, part] = y / sqrt(mean_part y^2 + eps) * w * sigmoid(z) instead -- the norm sees the scan's output itself and the
 // gate follows it (lightning attention, parts = 1).
 static __global__ void ly_gated_group_norm_kernel(const float* __restrict__ y, const float* __restrict__ proj, int ldp, int off_z,
-                                                  const float* __restrict__ w, float eps, int inner, int parts, int sig_after, float* __restrict__ u,
+                                                  const float* __restrict__ w, float eps, int inner, int parts, int sig_after, int ldo, float* __restrict__ u,
                                                   uint16_t* __restrict__ uhi, uint16_t* __restrict__ ulo) {
     __shared__ float red[33];
     const int row = blockIdx.x, n = inner / parts, c0 = blockIdx.y * n;
     const float* yr = y + (size_t)row * inner + c0;
     const float* zr = proj + (size_t)row * ldp + off_z + c0;
-    if (((inner | n | ldp | off_z) & 3) == 0) {         // 16-byte rows and parts: four channels per thread
+    const size_t ub = (size_t)row * ldo + c0;
+    if (((inner | n | ldp | off_z | ldo) & 3) == 0) {         // 16-byte rows and parts: four channels per thread
         float ss = 0.f;
         for (int c = threadIdx.x * 4; c < n; c += blockDim.x * 4) {
             float a[4], z[4];
@@ -1886,8 +1989,8 @@ static __global__ void ly_gated_group_norm_kernel(const float* __restrict__ y, c
             ld_vec<4>(yr + c, a); ld_vec<4>(zr + c, z); ld_vec<4>(w + c0 + c, ww);
 #pragma unroll
             for (int i = 0; i < 4; ++i) a[i] = sig_after ? a[i] * r * ww[i] * sigmoidf_(z[i]) : a[i] * siluf_(z[i]) * r * ww[i];
-            st_vec<4>(u + (size_t)row * inner + c0 + c, a);
-            split_store_vec<4>(uhi, ulo, (size_t)row * inner + c0 + c, a);
+            st_vec<4>(u + ub + c, a);
+            split_store_vec<4>(uhi, ulo, ub + c, a);
         }
         return;
     }
@@ -1896,8 +1999,8 @@ static __global__ void ly_gated_group_norm_kernel(const float* __restrict__ y, c
     const float r = 1.f / sqrtf(block_sum(ss, red) / (float)n + eps);
     for (int c = threadIdx.x; c < n; c += blockDim.x) {
         const float v = sig_after ? yr[c] * r * w[c0 + c] * sigmoidf_(zr[c]) : yr[c] * siluf_(zr[c]) * r * w[c0 + c];
-        u[(size_t)row * inner + c0 + c] = v;
-        split_store(uhi, ulo, (size_t)row * inner + c0 + c, v);
+        u[ub + c] = v;
+        split_store(uhi, ulo, ub + c, v);
     }
 }
 
@@ -1905,21 +2008,25 @@ static __global__ void ly_gated_group_norm_kernel(const float* __restrict__ y, c
 // act 0: act[p, f] = g * sigmoid(1.702 g) * (u + 1),  g = min(gu[p, f], limit),  u = clamp(gu[p, F + f], -limit, limit);
 // act 1: act[p, f] = gelu_tanh(g) * u,  gelu_tanh(z) = z/2 (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))).  bias [2F] (optional) is added
 // to gate | up first.  act 2: act[p, f] = relu(gu[p, f])^2 -- no gate matrix, gu has F columns.  act 3: act[p, f] = relu(g) * u.
+// act 4: act[p, f] = silu(g) * u.
+__device__ __forceinline__ float gelu_tanhf_(float g) { return 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))); }
 __device__ __forceinline__ float glu_value(float g, float u, int act, float limit) {
     if (act == 2) { g = fmaxf(g, 0.f); return g * g; }
     if (act == 3) return fmaxf(g, 0.f) * u;
-    if (act == 1) return 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
+    if (act == 4) return g * sigmoidf_(g) * u;
+    if (act == 1) return gelu_tanhf_(g) * u;
     g = fminf(g, limit);
     u = fminf(fmaxf(u, -limit), limit);
     return g * sigmoidf_(1.702f * g) * (u + 1.f);
 }
-// One block per (row p, chunk of 256 V channels); V consecutive channels per thread (V = 4: F a multiple of 4).
+// One block per (row p, chunk of 256 V channels); V consecutive channels per thread (V = 4: F, the row strides ldg of gu and ldo of the
+// output, and the addresses in multiples of 4).
 template <int V>
-static __global__ void __launch_bounds__(256) ly_glu_kernel(Slices gu, int F, float limit, int act_kind, const float* __restrict__ bias, float* __restrict__ act,
+static __global__ void __launch_bounds__(256) ly_glu_kernel(Slices gu, int ldg, int ldo, int F, float limit, int act_kind, const float* __restrict__ bias, float* __restrict__ act,
                                                             uint16_t* __restrict__ ahi, uint16_t* __restrict__ alo) {
     const int f = (blockIdx.y * 256 + threadIdx.x) * V;
     if (f >= F) return;
-    const size_t p = blockIdx.x, base = p * (act_kind == 2 ? (size_t)F : (size_t)2 * F) + f;
+    const size_t p = blockIdx.x, base = p * (size_t)ldg + f;
     float g[V], u[V] = {}, b[V];
     ld_slices<V>(gu, base, g);
     if (act_kind != 2) ld_slices<V>(gu, base + F, u);
@@ -1935,8 +2042,23 @@ static __global__ void __launch_bounds__(256) ly_glu_kernel(Slices gu, int F, fl
     }
 #pragma unroll
     for (int i = 0; i < V; ++i) g[i] = glu_value(g[i], u[i], act_kind, limit);
-    if (act != nullptr) st_vec<V>(act + p * F + f, g);          // nullptr: only the hi | lo halves are consumed (a tensor-core GEMM follows)
-    split_store_vec<V>(ahi, alo, p * F + f, g);
+    if (act != nullptr) st_vec<V>(act + p * ldo + f, g);          // nullptr: only the hi | lo halves are consumed (a tensor-core GEMM follows)
+    split_store_vec<V>(ahi, alo, p * ldo + f, g);
+}
+
+// Token vectors, between the two projections: a[row, j] = gelu_tanh(z[row, j]) * e[tok[row]][j], e = rows of a table (row stride lde, the
+// layer's columns first), z [rows, D] perhaps still in split-K slices.  a == nullptr: only the halves are read.
+static __global__ void ly_token_side_kernel(Slices z, const int* __restrict__ tok, const uint16_t* __restrict__ e, size_t lde, int D, float* __restrict__ a,
+                                            uint16_t* __restrict__ ahi, uint16_t* __restrict__ alo) {
+    const int row = blockIdx.x;
+    const uint16_t* er = e + (size_t)tok[row] * lde;
+    for (int j = threadIdx.x; j < D; j += blockDim.x) {
+        float v[1];
+        ld_slices<1>(z, (size_t)row * D + j, v);
+        v[0] = gelu_tanhf_(v[0]) * __uint_as_float((uint32_t)er[j] << 16);
+        if (a != nullptr) a[(size_t)row * D + j] = v[0];
+        split_store(ahi, alo, (size_t)row * D + j, v[0]);
+    }
 }
 
 // Router: z = Wr h (f32), s = softmax(z) over all experts, the `top` largest (lower index first among equals), weights s / (sum + 1e-20).
@@ -1989,14 +2111,15 @@ static __global__ void ly_router_kernel(const float* __restrict__ h, int W, cons
     }
 }
 
-// Router with independent scores: z = Wr h (f32), s = sigmoid(z); the choice runs on c = s + corr.  The experts form `groups` equal
-// groups of neighbours; a group's mark is the sum of its two largest c (its only one, for groups of one); the `keep` groups with the
-// largest marks stay eligible, the others' experts cannot be chosen whatever their c (c may be negative); the `top` eligible experts
-// with the largest c are used with the weights s, as they are.  Lower index first among equals, everywhere.
+// Router with group-limited choice: z = Wr h (f32), scores s = sigmoid(z), or (softmax) the softmax of z over all experts; the choice runs on
+// c = s + corr (corr == nullptr: c = s).  The experts form `groups` equal groups of neighbours; a group's mark is the sum of its two
+// largest c (mark2; its only one, for groups of one) or its largest; the `keep` groups with the largest marks stay eligible, the others'
+// experts cannot be chosen whatever their c (c may be negative); the `top` eligible experts with the largest c are used with the
+// weights s, as they are or (renorm) divided by their sum.  Lower index first among equals, everywhere.
 // One block per row, one warp per expert in turn; shared memory: 2 E + groups floats.
-static __global__ void ly_router_sigmoid_kernel(const float* __restrict__ h, int W, const float* __restrict__ wr, int E, int top,
-                                                const float* __restrict__ corr, int groups, int keep, int* __restrict__ sel,
-                                                float* __restrict__ wt) {
+static __global__ void ly_router_groups_kernel(const float* __restrict__ h, int W, const float* __restrict__ wr, int E, int top, int softmax,
+                                               const float* __restrict__ corr, int groups, int keep, int mark2, int renorm, int* __restrict__ sel,
+                                               float* __restrict__ wt) {
     extern __shared__ float z[];                 // [E] scores s, [E] choice scores c, [groups] marks
     float* cc = z + E;
     float* mark = cc + E;
@@ -2016,10 +2139,24 @@ static __global__ void ly_router_sigmoid_kernel(const float* __restrict__ h, int
             for (int c = lane; c < W; c += 32) d = fmaf(w[c], hr[c], d);
         }
         d = warp_sum(d);
-        if (lane == 0) { const float s = sigmoidf_(d); z[e] = s; cc[e] = s + corr[e]; }
+        if (lane == 0) z[e] = d;
     }
     __syncthreads();
-    if (threadIdx.x != 0) return;
+    if (wid != 0) return;                        // one warp finishes the row
+    float mx = -INFINITY, sum = 0.f;
+    if (softmax) {
+        for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
+        mx = warp_max(mx);
+        for (int e = lane; e < E; e += 32) sum += expf(z[e] - mx);
+        sum = warp_sum(sum);
+    }
+    for (int e = lane; e < E; e += 32) {
+        const float s = softmax ? expf(z[e] - mx) / sum : sigmoidf_(z[e]);
+        z[e] = s;
+        cc[e] = corr ? s + corr[e] : s;
+    }
+    __syncwarp();
+    if (lane != 0) return;
     const int per = E / groups;
     for (int g = 0; g < groups; ++g) {
         float b1 = -INFINITY, b2 = -INFINITY;
@@ -2027,7 +2164,7 @@ static __global__ void ly_router_sigmoid_kernel(const float* __restrict__ h, int
             const float v = cc[e];
             if (v > b1) { b2 = b1; b1 = v; } else if (v > b2) b2 = v;
         }
-        mark[g] = per > 1 ? b1 + b2 : b1;
+        mark[g] = per > 1 && mark2 ? b1 + b2 : b1;
     }
     // drop the groups.count - keep groups with the smallest marks (higher index first among equals): what stays is the `keep` best
     for (int k = 0; k < groups - keep; ++k) {
@@ -2038,6 +2175,7 @@ static __global__ void ly_router_sigmoid_kernel(const float* __restrict__ h, int
         mark[worst] = INFINITY;                  // a dropped group
         for (int e = worst * per; e < (worst + 1) * per; ++e) cc[e] = -INFINITY;
     }
+    float psum = 0.f;
     for (int k = 0; k < top; ++k) {
         int best = -1;
         float bv = -INFINITY;
@@ -2046,7 +2184,12 @@ static __global__ void ly_router_sigmoid_kernel(const float* __restrict__ h, int
         if (best < 0) best = 0;                  // only with scores that are not numbers
         sel[row * top + k] = best;
         wt[row * top + k] = z[best];
+        psum += z[best];
         cc[best] = -INFINITY;
+    }
+    if (renorm) {
+        const float inv = 1.f / (psum + 1e-20f);
+        for (int k = 0; k < top; ++k) wt[row * top + k] *= inv;
     }
 }
 

@@ -174,8 +174,9 @@ int dense_gemm(fl_cache& c, LaunchCtx& lc, const char* tag, int R, int N, int K,
 int dense_gemm_grouped(fl_cache& c, LaunchCtx& lc, const char* tag, int groups, int cap, int Ne, int K, const CUtensorMap& tmWall,
                        float* out, const uint16_t* xhi, const uint16_t* xlo, const int* cnt);
 // Block-diagonal GEMM (one matrix per head, say): out[t * ldo + b * o_bs + n] = sum_k x[t, b K + k] W_b[n, k] for b < blocks, n < N,
-// optionally times sigmoid(gate[t * ldg + b N + n]), as bf16 hi | lo halves; x = xhi + xlo [R, blocks * K], tmW covers the stacked
+// optionally times sigmoid(gate[t * ldg + b N + n]) (gate_blk: sigmoid(gate[t * ldg + b])), as bf16 hi | lo halves; x = xhi + xlo [R, blocks * K], tmW covers the stacked
 // [blocks * N, K] weights.  K, N, ldo and o_bs are multiples of 8, ldg of 4 (gate 16-byte aligned).
 void dense_gemm_blocks(fl_cache& c, LaunchCtx& lc, const char* tag, int R, int blocks, int N, int K, const CUtensorMap& tmW, const uint16_t* xhi,
-                       const uint16_t* xlo, uint16_t* ohi, uint16_t* olo, int ldo, int o_bs, const float* gate = nullptr, int ldg = 0);
+                       const uint16_t* xlo, uint16_t* ohi, uint16_t* olo, int ldo, int o_bs, const float* gate = nullptr, int ldg = 0,
+                       bool gate_blk = false);
 }  // namespace fl

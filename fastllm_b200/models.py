@@ -517,10 +517,10 @@ def _ffn_desc(d, i: int, mlp, act: str = "swish_clamp", bias: bool = False):
     elif mlp["kind"] == "dense":
         d.ffn, d.ff, d.limit = _lib.FL_FFN["dense"], int(mlp["ff"]), float(mlp.get("limit", 0.0))
     elif mlp["kind"] == "moe":
-        d.ffn, d.ff, d.limit = _lib.FL_FFN["moe"], int(mlp["expert"]["ff"]), float(mlp["expert"]["limit"])
+        d.ffn, d.ff, d.limit = _lib.FL_FFN["moe"], int(mlp["expert"]["ff"]), float(mlp["expert"].get("limit") or 0.0)
         d.experts, d.top = int(mlp["router"]["experts"]), int(mlp["router"]["top"])
         if mlp.get("shared"):
-            d.shared_ff, d.shared_limit = int(mlp["shared"]["ff"]), float(mlp["shared"]["limit"])
+            d.shared_ff, d.shared_limit = int(mlp["shared"]["ff"]), float(mlp["shared"].get("limit") or 0.0)
     else:
         raise FastllmError(-1, f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
 
@@ -841,6 +841,14 @@ def _query_latent_desc(d, m: dict):
     d.scale = float(m["scale"])
 
 
+def _loop_options(config: dict, sc, reinject: bool) -> None:
+    """fills the loop fields of a FlStackConfig from config.json's optional 'loop' entry"""
+    loop = config.get("loop")
+    if loop:
+        sc.loop_start, sc.loop_stop, sc.loop_times = int(loop["start"]), int(loop["stop"]), int(loop["times"])
+        sc.loop_reinject, sc.loop_step = int(reinject), 1
+
+
 def latodra_layer_descs(config: dict):
     """config.json of the Latodra decoder -> ctypes array of FlLayerDesc (every size and constant comes from the file)."""
     layers = config["layers"]
@@ -872,20 +880,69 @@ class LatodraWithConfig(_LayeredBase):
     @classmethod
     def stack_options(cls, config: dict, sc) -> None:
         sc.embed_norm, sc.layer_scale, sc.tied_head = 1, 1, 1
-        loop = config.get("loop")
-        if loop:
-            sc.loop_start, sc.loop_stop, sc.loop_times = int(loop["start"]), int(loop["stop"]), int(loop["times"])
-            sc.loop_reinject, sc.loop_step = 1, 1
+        _loop_options(config, sc, reinject=True)
 
     @classmethod
     def layer_descs(cls, config: dict, tensor_shapes: dict):
         return latodra_layer_descs(config)
 
 
+def tufazen_layer_descs(config: dict):
+    """config.json of the Tufazen decoder -> ctypes array of FlLayerDesc (every size and constant comes from the file)."""
+    layers = config["layers"]
+    arr = (_lib.FlLayerDesc * len(layers))()
+    for i, l in enumerate(layers):
+        d, m, kind, mlp = arr[i], l["mixer"], l["type"], l.get("mlp")
+        if kind == "latent_attention":          # a query latent, a key part turned in halves, one gate per head
+            _query_latent_desc(d, m)
+            d.rot_dim, d.rot_halves, d.out_gate = int(m["rot_dim"]), 1, 2
+            _rotary_desc(d, m.get("rot") or {}, d.rot_dim)
+        elif kind == "attention":               # values = un-turned keys, neighbours turn, capped scores, learned sink, a gate per channel
+            d.mixer, d.kv_from = _lib.FL_MIXER["attention"], -1
+            d.heads, d.kv_heads, d.dim = int(m["heads"]), int(m.get("kv_heads") or m["heads"]), int(m["dim"])
+            d.vdim = int(m.get("vdim") or d.dim)
+            d.scale, d.softcap = float(m["scale"]), float(m.get("softcap") or 0.0)
+            d.no_qk_norm, d.v_from_k, d.sink, d.out_gate = 1, 1, 2, 1
+            _rotary_desc(d, m.get("rot") or {"dims": 0}, 0)
+        else:
+            raise FastllmError(-1, f"layer {i}: unknown mixer type {kind!r}")
+        _ffn_desc(d, i, mlp, act="silu" if mlp and mlp["kind"] == "moe" else "swish_clamp")
+        if d.ffn == _lib.FL_FFN["moe"]:
+            g = mlp["router"].get("groups") or {}
+            d.router, d.route_best, d.shared_plain = _lib.FL_ROUTER["softmax_groups"], 1, 1
+            d.route_groups = int(g.get("count") or 1)
+            d.route_keep = int(g.get("keep") or d.route_groups)
+    return arr
+
+
+class TufazenWithConfig(_LayeredBase):
+    """The Tufazen decoder (no reference path): x += mixer(n) + ff(n) with one element-wise tanh norm n per layer, then a vector looked
+    up by token id and layer; latent attention (query latent, one gate per head) and grouped-query attention whose values are its
+    un-rotated keys; clamped-swish or silu-expert feed-forwards (best groups by softmax scores, weights as scored, a shared expert);
+    a hashed bigram table beside the embedding, a span of layers that runs several times with the same weights, scaled logits."""
+    arch, family, architectures = "tufazen", "Tufazen", ("Tufazen",)
+    norm_plain, no_post_norm = True, True
+
+    @classmethod
+    def stack_options(cls, config: dict, sc) -> None:
+        sc.norm_tanh, sc.parallel_sub = 1, 1
+        sc.token_side = int((config.get("token_side") or {}).get("dim") or 0)
+        bigram = (config.get("embedding") or {}).get("bigram")
+        if bigram:
+            sc.bigram_buckets = int(bigram["buckets"])
+            sc.bigram_mul_prev, sc.bigram_mul_cur = int(bigram["mul_prev"]), int(bigram["mul_cur"])
+        sc.logit_scale = float(config.get("logit_scale") or 0.0)
+        _loop_options(config, sc, reinject=False)
+
+    @classmethod
+    def layer_descs(cls, config: dict, tensor_shapes: dict):
+        return tufazen_layer_descs(config)
+
+
 # every adapter, in the order the registry tries them (model_registry.rs:169-182 keeps the same kind of list)
 def registered_models():
     return (LlamaWithConfig, MistralWithConfig, QwenWithConfig, MixtralWithConfig, NifunexWithConfig, RofetarWithConfig, TozaraxWithConfig,
-            MedulornWithConfig, LatodraWithConfig)
+            MedulornWithConfig, LatodraWithConfig, TufazenWithConfig)
 
 
 def model_class_for(config: dict):

@@ -79,10 +79,15 @@ typedef enum fl_arch {
                               (fl_stack_config.post_sum_norm); mixers read x through a token shift; chunk-masked attention with biased
                               projections | sliding-window attention with kept first tokens and a learned sink beside lightning attention;
                               relu-gated dense feed-forward or clamped-swish experts with a biased router; scaled embedding, capped logits */
-    FL_ARCH_LATODRA = 9    /* layered decoder (no reference path): latent attentions whose queries go through a latent of their own (one kind
+    FL_ARCH_LATODRA = 9,   /* layered decoder (no reference path): latent attentions whose queries go through a latent of their own (one kind
                               with a rotated shared key part and a learned softmax sink, one without positions and with a sigmoid gate on
                               the heads); a scale per channel on every sublayer's normed result; a span of layers that runs several times
                               with the same weights; a normed embedding that is also the output projection */
+    FL_ARCH_TUFAZEN = 10   /* layered decoder (no reference path): mixer and feed-forward read one element-wise tanh norm of the stream and join
+                              it together (fl_stack_config.parallel_sub, norm_tanh); latent attention with a query latent, halves rotation and one
+                              gate per head | grouped-query attention whose values are its un-rotated keys, capped, with a learned sink and a
+                              gate per channel; clamped-swish dense feed-forward | silu experts chosen from the best groups by softmax scores,
+                              beside a shared expert; hashed bigram rows in the embedding, per-layer token vectors, looped layers */
 } fl_arch;
 
 typedef enum fl_dtype { FL_DTYPE_F32 = 0, FL_DTYPE_BF16 = 1, FL_DTYPE_F16 = 2 } fl_dtype;
@@ -165,12 +170,19 @@ typedef struct fl_config {
  * logits.  shared_plain: the shared expert's output is added as it is (no "mlp.shared.sg").
  * Latent attention with q_rank > 0: q = W_uq c_q, c_q = RMS norm of W_dq h (tensors "dq" [q_rank, width], "dq.norm" [q_rank], "uq"
  * [heads * (dim + rot_dim), q_rank] instead of "q").  sink as for FL_MIXER_ATTN.  rot_dim = 0: no rotated part, only the latent is
- * cached.  out_gate: the concatenated heads are multiplied by sigmoid(W_g h) before W_o (tensor "g" [heads * vdim, width]). */
+ * cached.  out_gate = 1: the concatenated heads are multiplied by sigmoid(W_g h) before W_o (tensor "g" [heads * vdim, width]);
+ * out_gate = 2: every head by one number (tensor "g" [heads, width]); both for FL_MIXER_ATTN too.  rot_halves counts for latent
+ * attention as for FL_MIXER_ATTN (its queries' and its shared key part's rotated channels).
+ * FL_MIXER_ATTN with v_from_k: a head's values are its keys as projected, before they turn (no tensor "v", vdim = dim); the cache keeps
+ * the channels that do not turn once.
+ * Feed-forward (ffn_act = FL_ACT_SILU): y = W_down (silu(W_gate h) * (W_up h)).  A shared expert uses the experts' activation.
+ * router = FL_ROUTER_SOFTMAX_GROUPS: as FL_ROUTER_SIGMOID_GROUPS with scores s = softmax(W_r h) over all experts and no correction.
+ * route_best: a group is marked by its largest choice score alone.  route_renorm: the chosen experts' weights are divided by their sum. */
 typedef enum fl_mixer_kind { FL_MIXER_GLA = 0, FL_MIXER_LATENT_ATTN = 1, FL_MIXER_ATTN = 2, FL_MIXER_MAMBA2 = 3, FL_MIXER_DELTA = 4, FL_MIXER_LIGHTNING = 5 } fl_mixer_kind;
 typedef enum fl_ffn_kind { FL_FFN_NONE = 0, FL_FFN_DENSE = 1, FL_FFN_MOE = 2 } fl_ffn_kind;
-typedef enum fl_ffn_act { FL_ACT_SWISH_CLAMP = 0, FL_ACT_GELU_TANH = 1, FL_ACT_RELU2 = 2, FL_ACT_RELU = 3 } fl_ffn_act;
+typedef enum fl_ffn_act { FL_ACT_SWISH_CLAMP = 0, FL_ACT_GELU_TANH = 1, FL_ACT_RELU2 = 2, FL_ACT_RELU = 3, FL_ACT_SILU = 4 } fl_ffn_act;
 typedef enum fl_rot_scaling { FL_ROT_SCALE_YARN = 0, FL_ROT_SCALE_BANDS = 1 } fl_rot_scaling;
-typedef enum fl_router_kind { FL_ROUTER_SOFTMAX = 0, FL_ROUTER_SIGMOID_GROUPS = 1 } fl_router_kind;
+typedef enum fl_router_kind { FL_ROUTER_SOFTMAX = 0, FL_ROUTER_SIGMOID_GROUPS = 1, FL_ROUTER_SOFTMAX_GROUPS = 2 } fl_router_kind;
 
 typedef struct fl_layer_desc {
     int32_t mixer;                     /* fl_mixer_kind */
@@ -196,7 +208,7 @@ typedef struct fl_layer_desc {
     int32_t state, groups, norm_groups;/* Mamba-2: state size per head, B / C groups, parts of the gated output norm */
     float softcap;                     /* attention: score <- softcap * tanh(score / softcap); 0 = none */
     int32_t sink;                      /* attention, latent attention: 1 = one is added to the softmax denominator; 2 = exp(sink_h), a learned number per head */
-    int32_t rot_halves;                /* attention: 1 = rotary pairs are (i, i + rot_dims / 2), 0 = (2i, 2i + 1) */
+    int32_t rot_halves;                /* attention, latent attention: 1 = rotary pairs are (i, i + rot_dims / 2), 0 = (2i, 2i + 1) */
     int32_t ffn_act, ffn_bias;         /* feed-forward: fl_ffn_act; dense: 1 = gate / up / down carry biases */
     int32_t no_qk_norm;                /* attention: 1 = queries and keys are used as projected (no per-head norm, no norm tensors) */
     int32_t beside;                    /* 1 = the NEXT descriptor of the array describes a second mixer of this layer (its mixer fields only;
@@ -213,8 +225,10 @@ typedef struct fl_layer_desc {
     int32_t router_bias;               /* MoE, FL_ROUTER_SOFTMAX: 1 = the router logits carry a bias */
     int32_t shared_plain;              /* MoE: 1 = the shared expert is not gated */
     int32_t q_rank;                    /* latent attention: > 0 = queries go through a normed latent of this width */
-    int32_t out_gate;                  /* latent attention: 1 = the concatenated heads are gated by sigmoid(W_g h) */
-    int32_t reserved[2];
+    int32_t out_gate;                  /* attention, latent attention: the concatenated heads are gated by sigmoid(W_g h), 1 = per channel, 2 = per head */
+    int32_t v_from_k;                  /* attention: 1 = the values are the keys as projected, before rotation (needs no_qk_norm and vdim = dim) */
+    int32_t route_best, route_renorm;  /* routers with groups: 1 = a group's mark is its best score / weights are renormalised */
+    int32_t reserved[1];
 } fl_layer_desc;
 
 typedef struct fl_stack_config {
@@ -251,7 +265,17 @@ typedef struct fl_stack_config {
     int32_t loop_times;                /*   each pass with its own cache / state; 0 = no loop */
     int32_t loop_reinject;             /* 1: the embedding output is added to the stream before every pass but the first */
     int32_t loop_step;                 /* 1: row t of "loop.step" [loop_times, width] is added to the stream before pass t (after loop_reinject's sum) */
-    int32_t reserved[3];
+    int32_t norm_tanh;                 /* 1: the norms in front of sublayers and the final norm are tanh(alpha x) * w + b, channel by channel
+                                          ("<norm>" [width], "<norm>.b" [width], "<norm>.alpha" one number; needs no_post_norm) */
+    int32_t parallel_sub;              /* 1: x += mixer(norm1(x)) + ffn(norm1(x)) -- one norm and one join per layer (needs no_post_norm) */
+    int32_t token_side;                /* > 0: behind every layer x += rms_norm(P (gelu_tanh(G x) * e)) with this many inner channels, e = the layer's
+                                          part of the token's row of "side.embed" [vocab, n_layers * token_side] ("l<i>.side.gate" [token_side, width],
+                                          ".side.proj" [width, token_side], ".side.norm" [width], plain; needs no_post_norm) */
+    int32_t bigram_buckets;            /* > 0: row (previous token * mul_prev + token * mul_cur) mod buckets of "bigram" [buckets + 1, width] is added to
+                                          the embedding, the last row for a sequence's first token; the previous token is kept per slot */
+    float logit_scale;                 /* != 0: logits are multiplied by this (before a cap) */
+    int64_t bigram_mul_prev, bigram_mul_cur;
+    int32_t reserved[2];
 } fl_stack_config;
 
 /* ---- process / device -------------------------------------------------------------------------- */

@@ -64,7 +64,7 @@ def test_descriptor_layout_matches_header():
     assert _lib.FlLayerDesc.qkv_bias.offset == 104 + 15 * 4 and _lib.FlLayerDesc.shared_plain.offset == 104 + 23 * 4
     assert _lib.FlLayerDesc.out_scale.offset == 104 + 20 * 4
     assert _lib.FlStackConfig.post_sum_norm.offset == 13 * 4 and _lib.FlStackConfig.token_shift.offset == 18 * 4
-    assert ctypes.sizeof(_lib.FlLayerDesc) == 216 and ctypes.sizeof(_lib.FlStackConfig) == 120
+    assert ctypes.sizeof(_lib.FlLayerDesc) == 224 and ctypes.sizeof(_lib.FlStackConfig) == 152
 
 
 def test_registry_picks_by_architecture():

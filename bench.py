@@ -68,6 +68,10 @@ WORKLOADS = {
                            "positions and gated, layer scales, looped middle layers, dense gelu feed-forward) beside Nifunex with latent attention in "
                            "every layer and a dense feed-forward at equal width / ff / layers: 2048-token prefill and batch-8 decode at 2k context, "
                            "random weights"),
+    "tufazen_vs_latodra": ("tufazen", 8, 2048, "layered decoder (Tufazen: mixer and feed-forward in parallel on one tanh norm, token vectors behind every "
+                           "layer; latent attention with a dense feed-forward alternating with grouped-query attention on un-rotated values with "
+                           "silu experts) beside Latodra (latent attention, dense feed-forward) and Medulorn (grouped-query attention, experts with a "
+                           "shared one) at equal width / layers: 2048-token prefill and batch-8 decode at 2k context, random weights"),
 }
 QWEN_PREFILL_TFLOP_4K = 56.83         # 53.46 linear + 3.37 causal attention
 MINILM_FLOP_PER_TOKEN = 22.41e6      # 2 x 10.617 M linear + 4 T H 6 attention at T = 128
@@ -362,7 +366,7 @@ def run_reference(args, rank):
         return
     arch, batch, ctx, desc = WORKLOADS[args.workload]
     if args.workload in ("mixtral8x7b_b32", "qwen25_7b_prefill4k", "nifunex_vs_mixtral", "rofetar_vs_nifunex", "tozarax_vs_rofetar", "medulorn_vs_tozarax",
-                         "latodra_vs_nifunex"):
+                         "latodra_vs_nifunex", "tufazen_vs_latodra"):
         print(json.dumps({"impl": "reference", "unavailable": f"no CPU leg for workload {args.workload}: the reference does not wire Mixtral "
                           "and a 4096-token f32 prefill of a 7B model does not fit a bounded CPU sample; the decode workloads carry the CPU baseline"}),
               flush=True)
@@ -1268,6 +1272,69 @@ def run_latodra_compare(args, local_rank):
                       "clocks": clk.summary(t_wall0, t_wall1), "sizes": results}), flush=True)
 
 
+def _tufazen_config(width, ff, layers, vocab, times):
+    """A Tufazen config at the sizes of a real model's layers: even layers a latent attention (heads of 128 unrotated and 64 rotated
+    channels, values of 128, latents of 512, query latents of 3/8 of the width) with a dense feed-forward, odd layers a grouped-query
+    attention (4 query heads of 128 channels per key head, half of them turned) with 8 experts of half the dense width, top 2 of the best 2
+    of 4 groups, and a shared one; token vectors of 128 channels; the middle layers run `times` times."""
+    H = width // 128
+    ly = []
+    for i in range(layers):
+        if i % 2 == 0:
+            ly.append({"type": "latent_attention", "mlp": {"kind": "dense", "ff": ff, "limit": 7.0},
+                       "mixer": {"heads": H, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "q_rank": width * 3 // 8, "scale": 192 ** -0.5,
+                                 "rot": {"base": 10000.0, "dims": 64}}})
+        else:
+            ly.append({"type": "attention", "mlp": {"kind": "moe", "expert": {"ff": ff // 2}, "shared": {"ff": ff // 2},
+                                                    "router": {"experts": 8, "top": 2, "groups": {"count": 4, "keep": 2}}},
+                       "mixer": {"heads": H, "kv_heads": max(1, H // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 30.0,
+                                 "rot": {"base": 500000.0, "dims": 64, "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}})
+    return {"architecture": "Tufazen", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_scale": 1.0, "token_side": {"dim": 128},
+            "embedding": {"bigram": {"buckets": 4 * vocab - 3, "mul_prev": 1000003, "mul_cur": 31}},
+            "loop": {"start": 1, "stop": layers - 1, "times": times}, "layers": ly}
+
+
+def _medulorn_attention_config(width, ff, layers, vocab):
+    """Medulorn with its chunk-masked grouped-query attention in every layer (one chunk holds the whole context), experts of hidden width
+    ff and a shared one"""
+    cfg = _medulorn_config(width, ff, 2 * layers, vocab)
+    return dict(cfg, layers=cfg["layers"][1::2])
+
+
+def run_tufazen_compare(args, local_rank):
+    """--workload tufazen_vs_latodra (one GPU): Tufazen (each layer once, and with its middle layers run twice) beside the closest existing
+    design of either of its layer kinds -- Latodra (latent attention, dense feed-forward) and Medulorn (grouped-query attention, experts)
+    -- at the same width / layer count, random weights: one 2048-token prefill and batch-8 decode steps at a 2k context."""
+    from fastllm_b200 import models
+    batch, T, steps, warm = 8, 2048, max(4, min(args.steps, 32)), 3
+    sizes = [("w1024", 1024, 2816, 4), ("w2048", 2048, 5632, 4), ("w4096", 4096, 14336, 4)]
+    vocab = 32000
+    results = {}
+
+    def layered(cls, cfg, **hints):
+        return _layered_record(cls, cfg, local_rank, batch, T, steps, warm, vocab, **hints)
+
+    with ClockSampler(local_rank) as clk:
+        t_wall0 = time.time()
+        for name, width, ff, layers in sizes:
+            rec = {"width": width, "ff": ff, "expert_ff": ff // 2, "layers": layers}
+            rec["tufazen"] = layered(models.TufazenWithConfig, _tufazen_config(width, ff, layers, vocab, 1))
+            rec["tufazen_twice"] = layered(models.TufazenWithConfig, _tufazen_config(width, ff, layers, vocab, 2))
+            rec["latodra"] = layered(models.LatodraWithConfig, _latodra_config(width, ff, layers, vocab, 1))
+            rec["medulorn"] = layered(models.MedulornWithConfig, _medulorn_attention_config(width, ff // 2, layers, vocab))
+            results[name] = rec
+        t_wall1 = time.time()
+        time.sleep(0.12)
+    big = results[sizes[-1][0]]
+    print(json.dumps({"metric": "decode_tokens_per_s", "value": big["tufazen"]["decode_tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": steps, "warmup": warm,
+                      "ms_per_step": big["tufazen"]["decode_ms_per_step"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16",
+                      "data": "synthetic",
+                      "config": {"workload": WORKLOADS[args.workload][3], "batch": batch, "context": T, "timing": "wall clock around the public call "
+                                 "(host ids in, f32 logits out) with a device synchronise on both sides; per-kernel figures are CUDA events",
+                                 "l2": "weights of a step exceed L2 at the two larger sizes"},
+                      "clocks": clk.summary(t_wall0, t_wall1), "sizes": results}), flush=True)
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1310,6 +1377,9 @@ def main():
     elif args.workload == "latodra_vs_nifunex":
         if rank == 0:
             run_latodra_compare(args, local_rank)
+    elif args.workload == "tufazen_vs_latodra":
+        if rank == 0:
+            run_tufazen_compare(args, local_rank)
     elif args.workload == "rofetar_vs_nifunex":
         if rank == 0:
             run_rofetar_compare(args, local_rank)

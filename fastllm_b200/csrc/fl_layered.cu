@@ -916,10 +916,15 @@ static Slices gemm_slices(fl_cache& c, LaunchCtx& lc, const char* tag, const flo
     if (R <= 0) return Slices{Y, 1, 0};
     if (!tc || ahi == nullptr) { gemm(lc, tag, A, K, Wt, N, K, Y, N, R); return Slices{Y, 1, 0}; }
     LayeredCache& y = *c.ly;
-    const int ks_plan = R <= 128 ? pick_ksplit((N + 127) / 128, (K + 63) / 64, R) : 1;
+    int ks_plan = R <= 128 ? pick_ksplit((N + 127) / 128, (K + 63) / 64, R) : 1;
+    if (R > 128) {              // many rows but few output tiles (a narrow matrix): cut K as long as the slices fit the scratch
+        const int tiles = ((R + 127) / 128) * ((N + 255) / 256), nk = (K + 63) / 64;
+        // (up to eight slices of at least eight k blocks: none of them is empty)
+        while (ks_plan < 8 && 2 * ks_plan * tiles <= kNumSMs && nk / (2 * ks_plan) >= 8 && (size_t)(2 * ks_plan) * R * N <= y.gemm_out.n) ks_plan *= 2;
+    }
     float* out = ks_plan == 1 ? Y : y.gemm_out.p;
     FL_CHECK(ks_plan == 1 || (size_t)ks_plan * R * N <= y.gemm_out.n, FL_ERR_STATE, "internal: split-K scratch too small");
-    const int ks = dense_gemm(c, lc, tag, R, N, K, tm, out, ahi, alo);
+    const int ks = dense_gemm(c, lc, tag, R, N, K, tm, out, ahi, alo, nullptr, nullptr, R > 128 ? ks_plan : 1);
     FL_CHECK(ks == ks_plan, FL_ERR_STATE, "internal: split-K plan mismatch");
     return Slices{out, ks, (size_t)R * N};
 }
@@ -1320,10 +1325,10 @@ static void run_mixer(fl_cache& c, LaunchCtx& lc, const StepTab& st, const Layer
         AttnPrepArgs pa{y.proj.p, lw.n_in, lw.off_q, lw.off_k, lw.off_v, lw.qnorm, lw.knorm, eps, y.kv_pool[kv_index], y.page_table.p,
                         c.pages_per_seq, st.row_seq, st.row_pos, st.seq_slot, y.rope_cos[lw.rope_index].p, y.rope_sin[lw.rope_index].p,
                         H, G, D, Dv, d.rot_dims, d.rot_halves, lw.bq, lw.bk, lw.bv, d.qk_norm_whole, kv, in, lw.off_g, n_gate};
-        // eight warps per block take the heads in turn; steps of few rows spread a row's heads over up to four blocks (not with a
+        // eight warps per block take the heads in turn; steps of few rows spread a row's heads and gate columns over up to eight blocks (not with a
         // norm over the whole projection: its sums read every head before any is rewritten in place, which one block orders)
         const size_t psm = (size_t)8 * D * 4;
-        const int heads_all = H + (lw.off_k >= 0 ? G : 0), py = (Ti <= 64 && !d.qk_norm_whole) ? std::max(1, std::min(4, (heads_all + 7) / 8)) : 1;
+        const int heads_all = H + (lw.off_k >= 0 ? G : 0), py = (Ti <= 64 && !d.qk_norm_whole) ? std::max(1, std::min(8, std::max((heads_all + 7) / 8, n_gate / 512))) : 1;
         if (m.f32) launch(lc, "attn_prep", 0, ly_attn_prep_kernel<float>, dim3(Ti, py), dim3(256), psm, pa);
         else launch(lc, "attn_prep", 0, ly_attn_prep_kernel<uint16_t>, dim3(Ti, py), dim3(256), psm, pa);
         GqaAttnArgs at{y.proj.p, lw.n_in, lw.off_q, y.kv_pool[kv_index], y.page_table.p, c.pages_per_seq, st.row_seq, st.row_pos, st.seq_slot,
@@ -1599,10 +1604,15 @@ static void enqueue_step(fl_cache& c, LaunchCtx& lc, const StepTab& st, const in
         const fl_layer_desc& d = lw.d;
         const int F = d.ff, act = d.ffn_act, GF = act == FL_ACT_RELU2 ? F : 2 * F;
         const int E = d.experts, top = d.top, P = Ti * top;
-        if (d.router != FL_ROUTER_SOFTMAX)
-            launch(lc, "moe_router", 0, ly_router_groups_kernel, dim3(Ti), dim3(256), ((size_t)2 * E + d.route_groups) * 4, sub_in, W, (const float*)lw.router,
-                   E, top, d.router == FL_ROUTER_SOFTMAX_GROUPS ? 1 : 0, (const float*)lw.route_corr, d.route_groups, d.route_keep, d.route_best ? 0 : 1,
-                   d.route_renorm, y.route_sel.p, y.route_w.p);
+        if (d.router != FL_ROUTER_SOFTMAX) {
+            auto route = [&](auto kern, int rb) {
+                launch(lc, "moe_router", 0, kern, dim3((Ti + rb - 1) / rb), dim3(256), (size_t)rb * (2 * E + d.route_groups) * 4, sub_in, W, (const float*)lw.router, E, top,
+                       d.router == FL_ROUTER_SOFTMAX_GROUPS ? 1 : 0, (const float*)lw.route_corr, d.route_groups, d.route_keep, d.route_best ? 0 : 1, d.route_renorm, Ti,
+                       y.route_sel.p, y.route_w.p);
+            };
+            if (Ti >= 1024) route(ly_router_groups_kernel<4>, 4);       // (at most 48 KB of shared memory: E <= 1024)
+            else route(ly_router_groups_kernel<1>, 1);
+        }
         else
             launch(lc, "moe_router", 0, ly_router_kernel, dim3(Ti), dim3(256), (size_t)E * 4, sub_in, W, (const float*)lw.router, (const float*)lw.router_b, E, top,
                    (const float*)lw.shared_gate, y.route_sel.p, y.route_w.p, y.sgate.p);

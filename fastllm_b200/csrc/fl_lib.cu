@@ -1114,7 +1114,7 @@ int pick_ksplit(int tiles, int nk, int R) {
 //             N = R tile, the result is stored transposed; the only large shared-memory traffic is the weight stream.
 //   R  > 128 (prefill): tokens are the M dimension, 128 x 128 output tiles.
 int dense_gemm(fl_cache& c, LaunchCtx& lc, const char* tag, int R, int N, int K, const CUtensorMap& tmW, float* out,
-               const uint16_t* xhi, const uint16_t* xlo, uint16_t* silu_hi, uint16_t* silu_lo) {
+               const uint16_t* xhi, const uint16_t* xlo, uint16_t* silu_hi, uint16_t* silu_lo, int prefill_ks) {
     if (!xhi) { xhi = c.dw.xhi.p; xlo = c.dw.xlo.p; }
     const int nk = (K + kGemmBK - 1) / kGemmBK;
     const bool swap = R <= 128;
@@ -1123,7 +1123,7 @@ int dense_gemm(fl_cache& c, LaunchCtx& lc, const char* tag, int R, int N, int K,
     // 64 KB per 2 x 128 x 256 x 64 MACs where the 128-row one is 48 KB per half of that -- 1.5x the arithmetic per staged byte.
     static const int prefill_bn = env_flag("FL_PREFILL_BN128") ? 128 : 256;      // dev knob: the 128-row tile of round 1
     const int tiles = swap ? (N + 127) / 128 : ((R + kGemmBM - 1) / kGemmBM) * ((N + prefill_bn - 1) / prefill_bn);
-    const int ks = swap ? pick_ksplit(tiles, nk, R) : 1;
+    const int ks = swap ? pick_ksplit(tiles, nk, R) : (silu_hi != nullptr ? 1 : prefill_ks);
     ProfEntry pe;
     const bool prof = g_prof.on && !lc.capturing;
     const bool pdl = lc.pdl && !prof;
@@ -1153,9 +1153,9 @@ int dense_gemm(fl_cache& c, LaunchCtx& lc, const char* tag, int R, int N, int K,
             if (prefill_bn == 256) launch_gemm_tc<256, GEPI_SILU_HL, DUAL_A>(lc.stream, pdl, tiles, hi, lo, tmW, g);
             else launch_gemm_tc<128, GEPI_SILU_HL, DUAL_A>(lc.stream, pdl, tiles, hi, lo, tmW, g);
         } else {
-            GemmArgs g{R, N, K, nullptr, nullptr, 0, out, N, 1, (long long)R * N};
-            if (prefill_bn == 256) launch_gemm_tc<256, GEPI_F32, DUAL_A>(lc.stream, pdl, tiles, hi, lo, tmW, g);
-            else launch_gemm_tc<128, GEPI_F32, DUAL_A>(lc.stream, pdl, tiles, hi, lo, tmW, g);
+            GemmArgs g{R, N, K, nullptr, nullptr, 0, out, N, ks, (long long)R * N};
+            if (prefill_bn == 256) launch_gemm_tc<256, GEPI_F32, DUAL_A>(lc.stream, pdl, tiles * ks, hi, lo, tmW, g);
+            else launch_gemm_tc<128, GEPI_F32, DUAL_A>(lc.stream, pdl, tiles * ks, hi, lo, tmW, g);
         }
     }
     if (prof) {

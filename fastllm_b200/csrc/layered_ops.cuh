@@ -1451,13 +1451,13 @@ static __global__ void __launch_bounds__(256) ly_attn_prep_kernel(AttnPrepArgs a
         }
         __syncwarp();
     }
-    if (blockIdx.y != 0) return;
+    const int c0 = blockIdx.y * blockDim.x + threadIdx.x, cn = gridDim.y * blockDim.x;
     if (own && !shared_v) {
         CT* vd = dst + (size_t)a.G * a.D;
-        for (int c = threadIdx.x; c < a.G * a.Dv; c += blockDim.x) st_c(vd + c, in(a.off_v + c) + (a.bv ? a.bv[c] : 0.f));
+        for (int c = c0; c < a.G * a.Dv; c += cn) st_c(vd + c, in(a.off_v + c) + (a.bv ? a.bv[c] : 0.f));
     }
     if (a.in.n > 1)
-        for (int c = threadIdx.x; c < a.n_gate; c += blockDim.x) pr[a.off_gate + c] = in(a.off_gate + c);
+        for (int c = c0; c < a.n_gate; c += cn) pr[a.off_gate + c] = in(a.off_gate + c);
 }
 
 struct GqaAttnArgs {
@@ -2116,33 +2116,49 @@ static __global__ void ly_router_kernel(const float* __restrict__ h, int W, cons
 // largest c (mark2; its only one, for groups of one) or its largest; the `keep` groups with the largest marks stay eligible, the others'
 // experts cannot be chosen whatever their c (c may be negative); the `top` eligible experts with the largest c are used with the
 // weights s, as they are or (renorm) divided by their sum.  Lower index first among equals, everywhere.
-// One block per row, one warp per expert in turn; shared memory: 2 E + groups floats.
-static __global__ void ly_router_groups_kernel(const float* __restrict__ h, int W, const float* __restrict__ wr, int E, int top, int softmax,
-                                               const float* __restrict__ corr, int groups, int keep, int mark2, int renorm, int* __restrict__ sel,
+// One block per RB rows (many rows: an expert's weights are read once per RB of them), one warp per expert in turn, then one warp per row;
+// shared memory: RB (2 E + groups) floats.  A row's sums are taken in the same order whatever RB.
+template <int RB>
+static __global__ void __launch_bounds__(256) ly_router_groups_kernel(const float* __restrict__ h, int W, const float* __restrict__ wr, int E, int top, int softmax,
+                                               const float* __restrict__ corr, int groups, int keep, int mark2, int renorm, int T, int* __restrict__ sel,
                                                float* __restrict__ wt) {
-    extern __shared__ float z[];                 // [E] scores s, [E] choice scores c, [groups] marks
-    float* cc = z + E;
-    float* mark = cc + E;
-    const int row = blockIdx.x, lane = threadIdx.x & 31, wid = threadIdx.x >> 5, nw = blockDim.x >> 5;
-    const float* hr = h + (size_t)row * W;
+    extern __shared__ float zs[];                // per row: [E] scores s, [E] choice scores c, [groups] marks
+    const int row0 = blockIdx.x * RB, lane = threadIdx.x & 31, wid = threadIdx.x >> 5, nw = blockDim.x >> 5, per_row = 2 * E + groups;
+    const int nr = min(RB, T - row0);
+    const float* hr = h + (size_t)row0 * W;
     for (int e = wid; e < E; e += nw) {
         const float* w = wr + (size_t)e * W;
-        float d = 0.f;
+        float d[RB];
+#pragma unroll
+        for (int r = 0; r < RB; ++r) d[r] = 0.f;
         if ((W & 3) == 0) {
             const float4* w4 = reinterpret_cast<const float4*>(w);
-            const float4* h4 = reinterpret_cast<const float4*>(hr);
+#pragma unroll 2
             for (int c = lane; c < W / 4; c += 32) {
-                const float4 a = w4[c], b = h4[c];
-                d = fmaf(a.x, b.x, d); d = fmaf(a.y, b.y, d); d = fmaf(a.z, b.z, d); d = fmaf(a.w, b.w, d);
+                const float4 a = w4[c];
+#pragma unroll
+                for (int r = 0; r < RB; ++r)
+                    if (r < nr) {
+                        const float4 b = reinterpret_cast<const float4*>(hr + (size_t)r * W)[c];
+                        d[r] = fmaf(a.x, b.x, d[r]); d[r] = fmaf(a.y, b.y, d[r]); d[r] = fmaf(a.z, b.z, d[r]); d[r] = fmaf(a.w, b.w, d[r]);
+                    }
             }
         } else {
-            for (int c = lane; c < W; c += 32) d = fmaf(w[c], hr[c], d);
+            for (int c = lane; c < W; c += 32)
+#pragma unroll
+                for (int r = 0; r < RB; ++r)
+                    if (r < nr) d[r] = fmaf(w[c], hr[(size_t)r * W + c], d[r]);
         }
-        d = warp_sum(d);
-        if (lane == 0) z[e] = d;
+#pragma unroll
+        for (int r = 0; r < RB; ++r) {
+            d[r] = warp_sum(d[r]);
+            if (lane == 0) zs[r * per_row + e] = d[r];
+        }
     }
     __syncthreads();
-    if (wid != 0) return;                        // one warp finishes the row
+    if (wid >= nr) return;                       // (nr <= RB <= 8 warps)
+    const int row = row0 + wid;
+    float *z = zs + wid * per_row, *cc = z + E, *mark = cc + E;
     float mx = -INFINITY, sum = 0.f;
     if (softmax) {
         for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
@@ -2156,9 +2172,8 @@ static __global__ void ly_router_groups_kernel(const float* __restrict__ h, int 
         cc[e] = corr ? s + corr[e] : s;
     }
     __syncwarp();
-    if (lane != 0) return;
     const int per = E / groups;
-    for (int g = 0; g < groups; ++g) {
+    for (int g = lane; g < groups; g += 32) {
         float b1 = -INFINITY, b2 = -INFINITY;
         for (int e = g * per; e < (g + 1) * per; ++e) {
             const float v = cc[e];
@@ -2166,28 +2181,38 @@ static __global__ void ly_router_groups_kernel(const float* __restrict__ h, int 
         }
         mark[g] = per > 1 && mark2 ? b1 + b2 : b1;
     }
-    // drop the groups.count - keep groups with the smallest marks (higher index first among equals): what stays is the `keep` best
-    for (int k = 0; k < groups - keep; ++k) {
-        int worst = -1;
-        float wv = INFINITY;
-        for (int g = 0; g < groups; ++g)
-            if (mark[g] != INFINITY && (worst < 0 || mark[g] <= wv)) { wv = mark[g]; worst = g; }
-        mark[worst] = INFINITY;                  // a dropped group
-        for (int e = worst * per; e < (worst + 1) * per; ++e) cc[e] = -INFINITY;
+    __syncwarp();
+    // a group stays when fewer than `keep` others come before it (a larger mark, or an equal one and a lower index)
+    for (int g = lane; g < groups; g += 32) {
+        const float mg = mark[g];
+        int before = 0;
+        for (int o = 0; o < groups; ++o) before += mark[o] > mg || (mark[o] == mg && o < g);
+        if (before >= keep)
+            for (int e = g * per; e < (g + 1) * per; ++e) cc[e] = -INFINITY;
     }
+    __syncwarp();
     float psum = 0.f;
     for (int k = 0; k < top; ++k) {
-        int best = -1;
+        int best = E;
         float bv = -INFINITY;
-        for (int e = 0; e < E; ++e)
+        for (int e = lane; e < E; e += 32)
             if (cc[e] > bv) { bv = cc[e]; best = e; }
-        if (best < 0) best = 0;                  // only with scores that are not numbers
-        sel[row * top + k] = best;
-        wt[row * top + k] = z[best];
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ov = __shfl_xor_sync(0xFFFFFFFFu, bv, o);
+            const int oe = __shfl_xor_sync(0xFFFFFFFFu, best, o);
+            if (ov > bv || (ov == bv && oe < best)) { bv = ov; best = oe; }
+        }
+        if (best >= E) best = 0;                 // only with scores that are not numbers
         psum += z[best];
-        cc[best] = -INFINITY;
+        if (lane == 0) {
+            sel[row * top + k] = best;
+            wt[row * top + k] = z[best];
+            cc[best] = -INFINITY;
+        }
+        __syncwarp();
     }
-    if (renorm) {
+    if (renorm && lane == 0) {
         const float inv = 1.f / (psum + 1e-20f);
         for (int k = 0; k < top; ++k) wt[row * top + k] *= inv;
     }

@@ -167,10 +167,11 @@ struct fl_cache {
 namespace fl {
 // The dense tensor-core GEMM of fl_lib.cu (tcgen05 / TMEM / TMA, hi|lo activation halves), shared with the layered decoder:
 // out[ks][R, N] (f32, row stride N, slice stride R * N) = (xhi + xlo)[R, K] . W[N, K]^T; returns the number of split-K slices
-// (R <= 128: pick_ksplit of the weight tiles; R > 128: always 1), which the consumer sums in a fixed order.
+// (R <= 128: pick_ksplit of the weight tiles; R > 128: prefill_ks, one unless the caller asks for more), which the consumer sums in a fixed order.
 int pick_ksplit(int tiles, int nk, int R);
 int dense_gemm(fl_cache& c, LaunchCtx& lc, const char* tag, int R, int N, int K, const CUtensorMap& tmW, float* out,
-               const uint16_t* xhi = nullptr, const uint16_t* xlo = nullptr, uint16_t* silu_hi = nullptr, uint16_t* silu_lo = nullptr);
+               const uint16_t* xhi = nullptr, const uint16_t* xlo = nullptr, uint16_t* silu_hi = nullptr, uint16_t* silu_lo = nullptr,
+               int prefill_ks = 1);
 int dense_gemm_grouped(fl_cache& c, LaunchCtx& lc, const char* tag, int groups, int cap, int Ne, int K, const CUtensorMap& tmWall,
                        float* out, const uint16_t* xhi, const uint16_t* xlo, const int* cnt);
 // Block-diagonal GEMM (one matrix per head, say): out[t * ldo + b * o_bs + n] = sum_k x[t, b K + k] W_b[n, k] for b < blocks, n < N,

@@ -1016,10 +1016,17 @@ static void launch_gqa_attn_rb(LaunchCtx& lc, const GqaAttnArgs& a, int T, int s
     const int cpl = (std::max(a.D, a.Dv) + 31) / 32;
     const size_t smem = ((size_t)kGqaWarps * RB * (a.Dv + 2)) * 4;
     const dim3 g(T, a.H / RB, splits), b(kGqaWarps * 32);
-    if (cpl <= 1) launch(lc, "gqa_attn", 0, ly_gqa_attn_kernel<CT, 1, RB>, g, b, smem, a);
-    else if (cpl <= 2) launch(lc, "gqa_attn", 0, ly_gqa_attn_kernel<CT, 2, RB>, g, b, smem, a);
-    else if (cpl <= 4) launch(lc, "gqa_attn", 0, ly_gqa_attn_kernel<CT, 4, RB>, g, b, smem, a);
-    else launch(lc, "gqa_attn", 0, ly_gqa_attn_kernel<CT, 8, RB>, g, b, smem, a);
+    auto go = [&](auto c) {
+        constexpr int CPL = decltype(c)::value;
+        const size_t al = std::min<size_t>(16, CPL * sizeof(CT)) - 1, es = sizeof(CT);
+        const bool vec = a.D % CPL == 0 && a.Dv % CPL == 0 && (((size_t)a.kv.E * es | (size_t)a.kv.ks * es | (size_t)a.kv.vo * es | (size_t)a.kv.vs * es) & al) == 0;
+        if (vec) launch(lc, "gqa_attn", 0, ly_gqa_attn_kernel<CT, CPL, RB, true>, g, b, smem, a);
+        else launch(lc, "gqa_attn", 0, ly_gqa_attn_kernel<CT, CPL, RB, false>, g, b, smem, a);
+    };
+    if (cpl <= 1) go(std::integral_constant<int, 1>{});
+    else if (cpl <= 2) go(std::integral_constant<int, 2>{});
+    else if (cpl <= 4) go(std::integral_constant<int, 4>{});
+    else go(std::integral_constant<int, 8>{});
 }
 // max_keys: the most keys a row of the launch can see (bounds the useful number of key splits).  The exact mode never splits: there
 // a position's result is bitwise the same whatever else the launch holds.

@@ -765,6 +765,39 @@ __device__ __forceinline__ void load_chunk(const uint16_t* kp, int c0, int C, fl
     }
 }
 
+// the same for chunks that are whole and aligned to their size (at most 16 bytes): one or two loads, no branch
+template <int CPL>
+__device__ __forceinline__ void load_whole(const float* p, float (&o)[CPL]) {
+    if constexpr (CPL % 4 == 0) {
+#pragma unroll
+        for (int i = 0; i < CPL / 4; ++i) {
+            const float4 v = reinterpret_cast<const float4*>(p)[i];
+            o[4 * i] = v.x; o[4 * i + 1] = v.y; o[4 * i + 2] = v.z; o[4 * i + 3] = v.w;
+        }
+    } else if constexpr (CPL == 2) {
+        const float2 v = *reinterpret_cast<const float2*>(p);
+        o[0] = v.x; o[1] = v.y;
+    } else {
+        o[0] = *p;
+    }
+}
+template <int CPL>
+__device__ __forceinline__ void load_whole(const uint16_t* p, float (&o)[CPL]) {
+    if constexpr (CPL == 8) {
+        const uint4 v = *reinterpret_cast<const uint4*>(p);
+        o[0] = bf16lo(v.x); o[1] = bf16hi(v.x); o[2] = bf16lo(v.y); o[3] = bf16hi(v.y);
+        o[4] = bf16lo(v.z); o[5] = bf16hi(v.z); o[6] = bf16lo(v.w); o[7] = bf16hi(v.w);
+    } else if constexpr (CPL == 4) {
+        const uint2 v = *reinterpret_cast<const uint2*>(p);
+        o[0] = bf16lo(v.x); o[1] = bf16hi(v.x); o[2] = bf16lo(v.y); o[3] = bf16hi(v.y);
+    } else if constexpr (CPL == 2) {
+        const uint32_t v = *reinterpret_cast<const uint32_t*>(p);
+        o[0] = bf16lo(v); o[1] = bf16hi(v);
+    } else {
+        o[0] = ld_c(p);
+    }
+}
+
 constexpr int kLatWarps = 8;
 // One block per (row, head).  score_j = (q~ . c_j + q_rot . k_rot_j) * scale over the keys j the window admits (0 <= pos - j <
 // window), softmax in f32 with the optional sink, out = sum_j p_j c_j.  Warp w of the eight folds keys j0 + w, j0 + w + 8, ... into an online softmax (lanes own
@@ -1478,6 +1511,24 @@ struct GqaAttnArgs {
     OutGate gate;
 };
 constexpr int kGqaWarps = 8;
+// N sums over the warp at once (N a power of two): halves of the values are exchanged instead of whole sums, so that lanes
+// j * 32 / N .. end with the sum of v[j] -- N + log2(32 / N) - 1 shuffles instead of 5 N, added in the same order as warp_sum's
+template <int N>
+__device__ __forceinline__ float warp_sum_scatter(float (&v)[N], int lane) {
+    int off = 16;
+#pragma unroll
+    for (int n = N; n > 1; n >>= 1, off >>= 1) {
+        const bool up = lane & off;
+#pragma unroll
+        for (int i = 0; i < n / 2; ++i) {
+            const float send = up ? v[i] : v[i + n / 2], keep = up ? v[i + n / 2] : v[i];
+            v[i] = keep + __shfl_xor_sync(0xFFFFFFFFu, send, off);
+        }
+    }
+#pragma unroll
+    for (; off > 0; off >>= 1) v[0] += __shfl_xor_sync(0xFFFFFFFFu, v[0], off);
+    return v[0];
+}
 // One block per (row, RB query heads of one key/value head, key split).  score_j = cap(q . k_j * scale) over the keys the position
 // admits (key_span: causal, window with kept first keys, chunk), softmax in f32 with the optional sink, out = sum_j p_j v_j.  The
 // 8 x splits warps of a (row, head group) take the visible keys round-robin in ascending order: warp v folds the v-th, (v + 8 splits)-th,
@@ -1485,7 +1536,9 @@ constexpr int kGqaWarps = 8;
 // CPL consecutive channels of the key and of the value; a key and its value are loaded once for the RB heads).  Partial results
 // are merged in warp order; with one split the block writes the output itself (which warp takes which key then depends on the
 // position alone), otherwise ly_gqa_merge_kernel folds the splits in order.
-template <typename CT, int CPL, int RB>
+// VEC: D and Dv are multiples of CPL and every chunk of a cache row is aligned to its size (16 bytes at most): the keys in flight are
+// loaded without a branch between them (lanes behind the head's end read its last chunk; their query is zero and their sums are not used).
+template <typename CT, int CPL, int RB, bool VEC>
 static __global__ void __launch_bounds__(kGqaWarps * 32) ly_gqa_attn_kernel(GqaAttnArgs a) {
     extern __shared__ float sm[];               // [warps][RB][Dv] accumulators, then [warps][RB][2] (max, sum)
     const int row = a.row_base + blockIdx.x, hd0 = blockIdx.y * RB, split = blockIdx.z, S = gridDim.z;
@@ -1505,46 +1558,60 @@ static __global__ void __launch_bounds__(kGqaWarps * 32) ly_gqa_attn_kernel(GqaA
     }
     const int* pt = a.page_table + (size_t)slot * a.pps;
     const float inv_cap = a.softcap > 0.f ? 1.f / a.softcap : 0.f;
-    constexpr int KU = 2;
+    constexpr int KU = CPL <= 4 ? 4 : 2;        // keys in flight per warp
+    const int ck = g * a.kv.ks + min(lane * CPL, D - CPL), cv = a.kv.vo + g * a.kv.vs + min(lane * CPL, Dv - CPL);
     const int stride = kGqaWarps * S;
     for (int j = split * kGqaWarps + wid; j < n_vis; j += stride * KU) {
-        float val[KU][CPL], dot[KU][RB];
+        float key[KU][CPL], val[KU][CPL], dot[KU * RB];
+        const CT* kp[KU];
+#pragma unroll
+        for (int u = 0; u < KU; ++u) {          // (behind the last visible key: that key once more, its score is dropped below)
+            const int ji = min(j + u * stride, n_vis - 1), jj = ji < n_st ? ks.s_lo + ji : ks.j0 + (ji - n_st);
+            kp[u] = (const CT*)a.pool + ((size_t)pt[jj / kKvPage] * kKvPage + jj % kKvPage) * E;
+        }
 #pragma unroll
         for (int u = 0; u < KU; ++u) {
-            const int ji = j + u * stride, jj = ji < n_st ? ks.s_lo + ji : ks.j0 + (ji - n_st);
-#pragma unroll
-            for (int r = 0; r < RB; ++r) dot[u][r] = 0.f;
-            if (ji < n_vis) {
-                const CT* kp = (const CT*)a.pool + ((size_t)pt[jj / kKvPage] * kKvPage + jj % kKvPage) * E;
-                float kk[CPL];
-                load_chunk<CPL>(kp + (size_t)g * a.kv.ks, lane * CPL, D, kk);
-                load_chunk<CPL>(kp + a.kv.vo + (size_t)g * a.kv.vs, lane * CPL, Dv, val[u]);
-#pragma unroll
-                for (int r = 0; r < RB; ++r)
-#pragma unroll
-                    for (int i = 0; i < CPL; ++i) dot[u][r] = fmaf(q[r][i], kk[i], dot[u][r]);
+            if constexpr (VEC) {
+                load_whole<CPL>(kp[u] + ck, key[u]);
+                load_whole<CPL>(kp[u] + cv, val[u]);
             } else {
-#pragma unroll
-                for (int i = 0; i < CPL; ++i) val[u][i] = 0.f;
+                load_chunk<CPL>(kp[u] + (size_t)g * a.kv.ks, lane * CPL, D, key[u]);
+                load_chunk<CPL>(kp[u] + a.kv.vo + (size_t)g * a.kv.vs, lane * CPL, Dv, val[u]);
             }
         }
 #pragma unroll
         for (int u = 0; u < KU; ++u)
 #pragma unroll
-            for (int r = 0; r < RB; ++r) dot[u][r] = warp_sum(dot[u][r]);
-#pragma unroll
-        for (int u = 0; u < KU; ++u) {
-            if (j + u * stride >= n_vis) break;
-#pragma unroll
             for (int r = 0; r < RB; ++r) {
-                float sc = dot[u][r];
-                if (a.softcap > 0.f) sc = a.softcap * tanhf(sc * inv_cap);
-                const float mn = fmaxf(m[r], sc), corr = expf(m[r] - mn), p = expf(sc - mn);
-                l[r] = l[r] * corr + p;
+                float t = 0.f;
 #pragma unroll
-                for (int i = 0; i < CPL; ++i) acc[r][i] = acc[r][i] * corr + p * val[u][i];
-                m[r] = mn;
+                for (int i = 0; i < CPL; ++i) t = fmaf(q[r][i], key[u][i], t);
+                dot[u * RB + r] = t;
             }
+        // each lane caps one of the scores, then all of them are handed round
+        float own = warp_sum_scatter<KU * RB>(dot, lane);
+        if (a.softcap > 0.f) own = a.softcap * tanhf(own * inv_cap);
+#pragma unroll
+        for (int r = 0; r < RB; ++r) {
+            float sc[KU], mn = m[r];
+#pragma unroll
+            for (int u = 0; u < KU; ++u) {
+                const float t = __shfl_sync(0xFFFFFFFFu, own, (u * RB + r) * (32 / (KU * RB)));
+                sc[u] = j + u * stride < n_vis ? t : -INFINITY;
+                mn = fmaxf(mn, sc[u]);
+            }
+            const float corr = expf(m[r] - mn);
+            l[r] *= corr;
+#pragma unroll
+            for (int i = 0; i < CPL; ++i) acc[r][i] *= corr;
+#pragma unroll
+            for (int u = 0; u < KU; ++u) {
+                const float p = expf(sc[u] - mn);
+                l[r] += p;
+#pragma unroll
+                for (int i = 0; i < CPL; ++i) acc[r][i] = fmaf(p, val[u][i], acc[r][i]);
+            }
+            m[r] = mn;
         }
     }
     float* sacc = sm;
